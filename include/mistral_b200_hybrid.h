@@ -13,7 +13,7 @@
 extern "C" {
 #endif
 
-#define MBH_ABI_VERSION 4
+#define MBH_ABI_VERSION 5
 
 int mbh_abi_version(void);
 const char* mbh_last_error(void);
@@ -21,10 +21,11 @@ const char* mbh_last_error(void);
 /* x32[t, :] = table[tokens[t], :] * scale.  tokens: int64 [T]; table [V, D]; x32: fp32 [T, D]. */
 int mbh_embed_scale(const void* tokens, const void* table, float scale, void* x32, int64_t T, int64_t D, int dt, void* stream);
 
-/* y[t, :] = x32[t, :] / sqrt(mean(x32[t]^2) + eps) * w.  x32 fp32 [T, D] (the residual stream); y, w: storage type. */
-int mbh_rmsnorm(const void* x32, const void* w, void* y, int64_t T, int64_t D, float eps, int dt, void* stream);
+/* y[t, :] = x32[t, :] / sqrt(mean(x32[t]^2) + eps) * (offset + w).  x32 fp32 [T, D] (the residual stream); y, w: storage type.  offset 0:
+ * w is the weight; 1: the weight is stored around zero.  w2, y2 (both or null): a second norm of the same rows with its own weight. */
+int mbh_rmsnorm(const void* x32, const void* w, const void* w2, void* y, void* y2, int64_t T, int64_t D, float eps, float offset, int dt, void* stream);
 
-/* Linear x[M, K] W[N, K]^T (+ bias[N]) with an epilogue:
+/* Linear x[M, K] W[N, K]^T (+ bias[N]); row m of x starts at x + m * ldx (ldx >= K: x may be some columns of a wider matrix); an epilogue:
  *   0  out[M, N] = act(.)      SiLU on columns < n_act, identity elsewhere
  *   1  out32[M, N] += .        in-place add into the fp32 residual stream
  *   2  out[M, N/2]             rows of W interleaved (2c gate, 2c+1 up): g = min(gate, limit), u = clamp(up, -limit, limit),
@@ -32,8 +33,12 @@ int mbh_rmsnorm(const void* x32, const void* w, void* y, int64_t T, int64_t D, f
  *   3  out32[M, N] = .         fp32 result (logits); with limit > 0: limit * tanh(. / limit)
  *   5  out32[M, N] += alpha * .  the residual add of epilogue 1 with a fixed weight
  * Any M, N, K.  M <= 8 runs the weight-streaming kernel, larger M the tiled one (tensor cores for bf16). */
-int mbh_linear(const void* x, const void* w, const void* bias, void* out, void* out32, int64_t M, int64_t N, int64_t K, int epi, int64_t n_act,
+int mbh_linear(const void* x, int64_t ldx, const void* w, const void* bias, void* out, void* out32, int64_t M, int64_t N, int64_t K, int epi, int64_t n_act,
                float limit, float alpha, int dt, void* stream);
+
+/* Decays of a gated recurrence: out32[M, N] = exp(-exp(a_log[n / group]) * softplus(x W^T + bias)), fp32 from the sum on; a_log [N / group]. */
+int mbh_linear_decay(const void* x, int64_t ldx, const void* w, const void* bias, const void* a_log, int64_t group, void* out32, int64_t M, int64_t N, int64_t K,
+                     int dt, void* stream);
 
 /* The epilogues of mbh_linear alone, applied to y[M, N] (storage type, N even) that another GEMM produced. */
 int mbh_linear_epilogue(const void* y, const void* bias, void* out, void* out32, int64_t M, int64_t N, int epi, int64_t n_act, float limit, float alpha,
@@ -73,56 +78,57 @@ int mbh_embed_add(const void* tokens, const void* table, float scale, void* x32,
  * Exactly one of y (storage type [T, D]: y = norm) and acc32 (fp32 [T, D]: acc32 += norm, in fp32) is given. */
 int mbh_layernorm(const void* x32, const void* w, const void* b, void* y, void* acc32, int64_t T, int64_t D, float eps, int dt, void* stream);
 
-/* Linear with interleaved gate/up rows (as epilogue 2 of mbh_linear) and out[M, N/2] = silu(gate) * up * rowscale[m, c / rs_group];
- * rowscale: fp32 [M, rs_pitch] or null (no scaling).  mbh_swiglu_epilogue applies the same to y[M, N] of another GEMM. */
+/* Linear with interleaved gate/up rows (as epilogue 2 of mbh_linear) and out[M, N/2] = act(gate) * up * rowscale[m, c / rs_group];
+ * act 0: SiLU, 1: the tanh form of gelu; rowscale: fp32 [M, rs_pitch] or null (no scaling).  mbh_swiglu_epilogue applies the same to y[M, N] of another GEMM. */
 int mbh_linear_swiglu(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, const void* rowscale, int64_t rs_pitch,
-                      int64_t rs_group, int dt, void* stream);
-int mbh_swiglu_epilogue(const void* y, void* out, int64_t M, int64_t N, const void* rowscale, int64_t rs_pitch, int64_t rs_group, int dt,
+                      int64_t rs_group, int act, int dt, void* stream);
+int mbh_swiglu_epilogue(const void* y, void* out, int64_t M, int64_t N, const void* rowscale, int64_t rs_pitch, int64_t rs_group, int act, int dt,
                         void* stream);
 
-/* Latent attention, input side.  y [T, pitch] = [query latent (q_rank) | key/value latent (kv_rank) | shared rotated key part
- * (rot_dim) | ...].  cq [T, q_rank] = rms_norm(query latent) * qnorm; ring row cache_rows[t] (-1: not cached) of ring
- * [rows, kv_rank + rot_dim] = [rms_norm(kv latent) * cnorm | rot(key part)].  rot: the pairs (2i, 2i+1), i < rot_dims / 2, turn by
- * positions[t] * freq[i] (freq: float64 [rot_dims / 2]), cos and sin times mag; entries from rot_dims on pass unchanged. */
+/* Latent attention, input side.  y [T, pitch] holds the query latent (q_rank entries from column 0; q_rank 0: none) and, from column kv_off,
+ * [key/value latent (kv_rank) | shared rotated key part (rot_dim)].  cq [T, q_rank] = rms_norm(query latent) * qnorm; the token's row
+ * [rms_norm(kv latent) * cnorm | rot(key part)] goes to ring row cache_rows[t] of ring [rows, kv_rank + rot_dim] (-1: not cached;
+ * cache_rows null: no ring write) and, when given, to own [T, kv_rank + rot_dim].  rot: the pairs (2i, 2i+1), or (i, i + rot_dims / 2) with
+ * halves = 1, i < rot_dims / 2, turn by positions[t] * freq[i] (freq: float64 [rot_dims / 2]), cos and sin times mag; entries from rot_dims
+ * on pass unchanged. */
 int mbh_latent_prep(const void* y, const void* qnorm, const void* cnorm, const void* freq, const void* positions, const void* cache_rows, void* cq,
-                    void* ring, int64_t T, int64_t pitch, int64_t q_rank, int64_t kv_rank, int64_t rot_dim, int64_t rot_dims, float eps, float mag,
-                    int dt, void* stream);
+                    void* ring, int64_t T, int64_t pitch, int64_t q_rank, int64_t kv_off, int64_t kv_rank, int64_t rot_dim, int64_t rot_dims, int halves,
+                    float eps, float mag, void* own, int dt, void* stream);
 
-/* q [T, H, dn + rot_dim] -> qa [T, H, kv_rank + rot_dim] = [W_uk[h]^T q[:dn] | rot(q[dn:])], w_uk [H * dn, kv_rank].
- * w_uk null: no folding, qa [T, H, dn + rot_dim] = [q[:dn] | rot(q[dn:])]. */
-int mbh_latent_absorb(const void* q, const void* w_uk, const void* freq, const void* positions, void* qa, int64_t T, int64_t H, int64_t dn,
-                      int64_t rot_dim, int64_t rot_dims, int64_t kv_rank, float mag, int dt, void* stream);
+/* q (rows of q_pitch elements, [H, dn + rot_dim] at the start of each) -> qa [T, H, kv_rank + rot_dim] = [W_uk[h]^T q[:dn] | rot(q[dn:])],
+ * w_uk [H * dn, kv_rank].  w_uk null: no folding, qa [T, H, dn + rot_dim] = [q[:dn] | rot(q[dn:])]. */
+int mbh_latent_absorb(const void* q, int64_t q_pitch, const void* w_uk, const void* freq, const void* positions, void* qa, int64_t T, int64_t H, int64_t dn,
+                      int64_t rot_dim, int64_t rot_dims, int halves, int64_t kv_rank, float mag, int dt, void* stream);
 
-/* Keys and values per head of whole prompts, for ordinary multi-head attention (mbh_attn_bias with bias_tab null): token t at
- * position p of sequence b goes to row b * Wt + p of kfull [B * Wt, H, dn + rot_dim] = [kn[t, h] | rotated key part of ring row
- * cache_rows[t]] and vfull [B * Wt, H, dv] = v[t, h].  kn [T, H * dn], v [T, H * dv]. */
-int mbh_latent_expand(const void* kn, const void* v, const void* ring, const void* positions, const void* cache_rows, const void* q_start, void* kfull,
-                      void* vfull, int64_t T, int64_t B, int64_t Wt, int64_t H, int64_t dn, int64_t rot_dim, int64_t dv, int64_t kv_rank, int dt,
-                      void* stream);
+/* Keys per head of R latent rows [R, kv_rank + rot_dim], for ordinary multi-head attention: kfull [R, H, dn + rot_dim] = [kn[r, h] | the row's
+ * rotated key part], kn [R, H * dn]. */
+int mbh_latent_expand(const void* kn, const void* rows, void* kfull, int64_t R, int64_t H, int64_t dn, int64_t rot_dim, int64_t kv_rank, int dt, void* stream);
 
 /* out [T, H, dv] *= sigmoid(gate[t * g_pitch + g_off + h]), in place. */
 int mbh_head_gate(void* out, const void* gate, int64_t g_pitch, int64_t g_off, int64_t T, int64_t H, int64_t dv, int dt, void* stream);
 
 /* Causal softmax attention of qa over latent rows: score = qa . ring row * scale, value = the row's first kv_rank entries;
- * o_lat [T, H, kv_rank].  Ring addressing, splits and scratch as mbh_attn_bias (exact fp32 kernel, one key/value head). */
+ * o_lat [T, H, kv_rank].  Ring addressing, splits and scratch as mbh_attn_bias (exact fp32 kernel, one key/value head); window, own (rows of
+ * this call's tokens) with seqpos, and sink as mbh_attn_window. */
 int mbh_attn_latent(const void* qa, const void* ring, const void* positions, const void* q_start, const void* slots, void* o_lat, int64_t T,
-                    int64_t B, int64_t W, int64_t H, int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int dt,
-                    void* stream);
+                    int64_t B, int64_t W, int64_t H, int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int64_t window,
+                    const void* own, const void* seqpos, const void* sink, int dt, void* stream);
 
 /* The same for one token per sequence (token b belongs to sequence b; qa [B, H, kv_rank + rot_dim]): each CTA reads a span of one
- * sequence's rows once for all heads.  H <= 32, kv_rank <= 512; scratch fp32 [B * H, splits, 2 + kv_rank], splits >= 1. */
+ * sequence's rows once for all heads.  H <= 32, kv_rank <= 512; scratch fp32 [B * H, splits, 2 + kv_rank], splits >= 1; window and
+ * sink as mbh_attn_window. */
 int mbh_attn_latent_decode(const void* qa, const void* ring, const void* positions, const void* slots, void* o_lat, int64_t B, int64_t W, int64_t H,
-                           int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int dt, void* stream);
+                           int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int64_t window, const void* sink, int dt, void* stream);
 
 /* out [T, H * dv] = (W_uv[h] o_lat[t, h]) * sigmoid(gate[t * g_pitch + g_off + h]); w_uv [H * dv, kv_rank]; gate null: no gate. */
 int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_t g_pitch, int64_t g_off, void* out, int64_t T, int64_t H,
                    int64_t dv, int64_t kv_rank, int dt, void* stream);
 
 /* Router of a mixture of experts, fp32: s = softmax(W_r h) over n outputs (score 0) or sigmoid of each output (score 1), choice = s + correction (null: none); the outputs form
- * `groups` equal groups of neighbours and only those of the `keep` groups with the largest choice stay eligible; the `top` largest
- * eligible choices are taken, weighted by s * scale.  dense: fp32 [T, n] (0 where not chosen); idx int32 / wsel fp32 [T, top]. */
+ * `groups` equal groups of neighbours and only those of the `keep` groups with the largest choice (group_two: the largest sum of the two largest
+ * choices) stay eligible; the `top` largest eligible choices are taken, weighted by s * scale (renorm: s / (sum of the chosen s + 1e-20) * scale).  dense: fp32 [T, n] (0 where not chosen); idx int32 / wsel fp32 [T, top]. */
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int dt, void* stream);
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, int dt, void* stream);
 
 /* The chosen experts of few tokens: y32 [T, width] = sum_k wsel[t, k] * expert(idx[t, k])(h[t]); an index >= E is an identity
  * expert (output = h[t]).  w13 [E * 2 * ff, width] (gate and up rows interleaved), w2 [width, E * ff]; act: scratch [T * top, ff].
@@ -143,11 +149,12 @@ int mbh_rows_axpy(void* y32, const void* h, const void* dense, int64_t T, int64_
  * chunk: keys per warp and step of the exact kernel, 1 .. 128 (0: 128); with `splits` CTAs of 4 warps per (token, head) a CTA takes
  * 4 * chunk keys per round, so a short ring read by few tokens is spread over splits = ceil(W / (4 * chunk)) CTAs.
  * weights 0: softmax over the visible keys.  weights 1: every visible key weighs sigmoid(score) and nothing is normalised (bias_tab with
- * n_tab = 1 is then a number per head inside the sigmoid). */
+ * n_tab = 1 is then a number per head inside the sigmoid).
+ * softcap > 0: score <- softcap * tanh(score / softcap).  sink (fp32 [H] or null): the softmax denominator of head h also holds exp(sink[h]). */
 int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, const void* bias_tab, int64_t n_tab, const void* positions,
                     const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
                     float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, const void* own_k, const void* own_v,
-                    const void* seqpos, int64_t chunk, int weights, int dt, void* stream);
+                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, int dt, void* stream);
 
 /* Linear with interleaved gate/up rows and the clamped gated unit of mbh_linear's epilogue 2; gate and up of column c are multiplied by
  * rowscale[m, c / rs_group] (fp32 [M, rs_pitch]; null: 1) BEFORE the clamps.  mbh_glu_epilogue applies the same to y[M, N] of another GEMM. */
@@ -160,12 +167,13 @@ int mbh_glu_epilogue(const void* y, void* out, int64_t M, int64_t N, float limit
 int mbh_embed_pos(const void* tokens, const void* positions, const void* table, const void* pos_table, float scale, void* x32, int64_t T, int64_t D,
                   int dt, void* stream);
 
-/* Splits qkv[T, H*d + G*d + G*e]; rotates the first rot_dims entries of every q and k head as interleaved pairs (2i, 2i + 1) by the angle
- * positions[t] * freq[i] (freq: float64 [rot_dims / 2]); with unit_norm divides every rotated head by sqrt(mean(x^2) + eps).  Writes
+/* Splits qkv[T, H*d + G*d + G*e]; rotates the first rot_dims entries of every q and k head as interleaved pairs (2i, 2i + 1), or as pairs
+ * (i, i + rot_dims / 2) with halves = 1, by the angle positions[t] * freq[i] (freq: float64 [rot_dims / 2]), cos and sin times mag; with unit_norm divides every rotated head by sqrt(mean(x^2) + eps).  Writes
  * q_out [T, H*d]; k_out [T, G*d] and v_out [T, G*e] (both or neither); and, when cache_rows is given, k and v of token t into ring row
  * cache_rows[t] (-1: not cached). */
 int mbh_rot_prep(const void* qkv, const void* freq, const void* positions, const void* cache_rows, void* q_out, void* k_out, void* v_out, void* ring_k,
-                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int unit_norm, float eps, int dt, void* stream);
+                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int halves, float mag, int unit_norm, float eps, int dt,
+                 void* stream);
 
 /* ring_k[cache_rows[t]] = k[t] (Nk entries), ring_v[cache_rows[t]] = v[t] (Nv entries) for every t with cache_rows[t] >= 0. */
 int mbh_kv_scatter(const void* k, const void* v, const void* cache_rows, void* ring_k, void* ring_v, int64_t T, int64_t Nk, int64_t Nv, int dt,
@@ -234,6 +242,27 @@ int mbh_linear_relu2(const void* x, const void* w, void* out, int64_t M, int64_t
                      int64_t rs_group, int dt, void* stream);
 int mbh_relu2_epilogue(const void* y, void* out, int64_t M, int64_t N, const void* rowscale, int64_t rs_pitch, int64_t rs_group, int dt,
                        void* stream);
+
+/* Gated delta rule, S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per head.  y [T, y_pitch] = q (G*d) | k (G*d) | v (H*e) | beta
+ * logits (H) | decay latent (ra) | gate latent (rg) | ...; head h uses q / k head h / (H / G).  q, k and v first pass a causal convolution over
+ * time per channel (conv [2*G*d + H*e, taps], last tap = the current token) and SiLU; cstate fp32 [slots, taps, 2*G*d + H*e] keeps the inputs of
+ * a sequence, position p in row p % taps.  mbh_delta_prep (prompts): qk fp32 [T, 2, G*d] = q / sqrt(sum q^2 + 1e-6) * d^(-1/2) | k / sqrt(sum k^2
+ * + 1e-6); kq [T, G] = k . q; v fp32 [T, H*e]; beta fp32 [T, H] = sigmoid; advances cstate. */
+int mbh_delta_prep(const void* y, int64_t y_pitch, const void* conv, int64_t taps, void* cstate, const void* positions, const void* q_start, const void* seqpos,
+                   const void* slots, void* qk, void* kq, void* v, void* beta, int64_t T, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, int dt,
+                   void* stream);
+
+/* The recurrence over whole prompts (portions): g fp32 [T, H*d]; state fp32 [slots, H, e, d] is read (unless seqpos[b] == 0: zero) and written back;
+ * o32 fp32 [T, H*e].  d <= 1024. */
+int mbh_delta_scan(const void* qk, const void* kq, const void* v, const void* beta, const void* g, void* state, const void* q_start, const void* seqpos,
+                   const void* slots, void* o32, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, void* stream);
+
+/* One token per sequence, everything between the input and the output projection in one launch: convolutions, unit norms, g = exp(-exp(a_log[h])
+ * softplus(w_a2 (decay latent) + dt_bias)) (w_a2 [H*d, ra], dt_bias [H*d], a_log [H]), the state step, every head's o / sqrt(mean(o^2) + eps) *
+ * norm[e] * sigmoid(w_g2 (gate latent)) (w_g2 [H*e, rg]).  out [B, H*e]. */
+int mbh_delta_step(const void* y, int64_t y_pitch, int64_t ra, int64_t rg, const void* conv, int64_t taps, void* cstate, void* state, const void* w_a2,
+                   const void* dt_bias, const void* a_log, const void* w_g2, const void* norm, const void* positions, const void* seqpos, const void* slots,
+                   void* out, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, float eps, int dt, void* stream);
 
 #ifdef __cplusplus
 }

@@ -13,7 +13,7 @@ import torch
 from . import _abi, build
 from ._abi import Mb200Error
 
-ABI_VERSION = 4
+ABI_VERSION = 5
 EPI_STORE, EPI_RESIDUAL, EPI_GLU, EPI_F32, EPI_RESIDUAL_SCALED = 0, 1, 2, 3, 5
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 _lib: Optional[ctypes.CDLL] = None
@@ -23,8 +23,9 @@ _SIGNATURES = {
     "mbh_abi_version": (c_int, []),
     "mbh_last_error": (c_char_p, []),
     "mbh_embed_scale": (c_int, [P, P, F, P, I, I, c_int, P]),
-    "mbh_rmsnorm": (c_int, [P, P, P, I, I, F, c_int, P]),
-    "mbh_linear": (c_int, [P, P, P, P, P, I, I, I, c_int, I, F, F, c_int, P]),
+    "mbh_rmsnorm": (c_int, [P, P, P, P, P, I, I, F, F, c_int, P]),
+    "mbh_linear_decay": (c_int, [P, I, P, P, P, I, P, I, I, I, c_int, P]),
+    "mbh_linear": (c_int, [P, I, P, P, P, P, I, I, I, c_int, I, F, F, c_int, P]),
     "mbh_linear_epilogue": (c_int, [P, P, P, P, I, I, c_int, I, F, F, c_int, P]),
     "mbh_attn_prep": (c_int, [P, P, P, P, P, P, P, P, P, P, c_int, I, I, I, I, I, F, F, I, c_int, P]),
     "mbh_attn_bias": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, c_int, P]),
@@ -32,22 +33,22 @@ _SIGNATURES = {
     "mbh_gated_headnorm": (c_int, [P, P, P, I, I, P, I, I, F, c_int, P]),
     "mbh_embed_add": (c_int, [P, P, F, P, I, I, c_int, P]),
     "mbh_layernorm": (c_int, [P, P, P, P, P, I, I, F, c_int, P]),
-    "mbh_linear_swiglu": (c_int, [P, P, P, I, I, I, P, I, I, c_int, P]),
-    "mbh_swiglu_epilogue": (c_int, [P, P, I, I, P, I, I, c_int, P]),
-    "mbh_latent_prep": (c_int, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, c_int, P]),
-    "mbh_latent_absorb": (c_int, [P, P, P, P, P, I, I, I, I, I, I, F, c_int, P]),
-    "mbh_latent_expand": (c_int, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, c_int, P]),
+    "mbh_linear_swiglu": (c_int, [P, P, P, I, I, I, P, I, I, c_int, c_int, P]),
+    "mbh_swiglu_epilogue": (c_int, [P, P, I, I, P, I, I, c_int, c_int, P]),
+    "mbh_latent_prep": (c_int, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, c_int, F, F, P, c_int, P]),
+    "mbh_latent_absorb": (c_int, [P, I, P, P, P, P, I, I, I, I, I, c_int, I, F, c_int, P]),
+    "mbh_latent_expand": (c_int, [P, P, P, I, I, I, I, I, c_int, P]),
     "mbh_head_gate": (c_int, [P, P, I, I, I, I, I, c_int, P]),
-    "mbh_attn_latent": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, c_int, P]),
-    "mbh_attn_latent_decode": (c_int, [P, P, P, P, P, I, I, I, I, I, F, I, P, c_int, P]),
+    "mbh_attn_latent": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, I, P, P, P, c_int, P]),
+    "mbh_attn_latent_decode": (c_int, [P, P, P, P, P, I, I, I, I, I, F, I, P, I, P, c_int, P]),
     "mbh_latent_vup": (c_int, [P, P, P, I, I, P, I, I, I, I, c_int, P]),
-    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, P]),
+    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, c_int, P]),
     "mbh_moe_sparse": (c_int, [P, P, P, P, P, P, P, I, I, I, I, I, c_int, F, F, c_int, c_int, P]),
-    "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, I, c_int, c_int, P]),
+    "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, I, c_int, F, P, c_int, P]),
     "mbh_linear_glu": (c_int, [P, P, P, I, I, I, F, F, P, I, I, c_int, P]),
     "mbh_glu_epilogue": (c_int, [P, P, I, I, F, F, P, I, I, c_int, P]),
     "mbh_embed_pos": (c_int, [P, P, P, P, F, P, I, I, c_int, P]),
-    "mbh_rot_prep": (c_int, [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, P]),
+    "mbh_rot_prep": (c_int, [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, F, c_int, P]),
     "mbh_kv_scatter": (c_int, [P, P, P, P, P, I, I, I, c_int, P]),
     "mbh_gated_scan": (c_int, [P, P, I, I, P, I, P, P, P, P, P, I, I, I, I, I, c_int, I, I, P, c_int, P]),
     "mbh_hgrn2_gates": (c_int, [P, P, P, I, I, I, c_int, P]),
@@ -61,6 +62,9 @@ _SIGNATURES = {
     "mbh_whole_norm_prep": (c_int, [P, P, P, P, P, P, P, P, P, I, I, I, I, F, c_int, P]),
     "mbh_linear_relu2": (c_int, [P, P, P, I, I, I, P, I, I, c_int, P]),
     "mbh_relu2_epilogue": (c_int, [P, P, I, I, P, I, I, c_int, P]),
+    "mbh_delta_prep": (c_int, [P, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, c_int, P]),
+    "mbh_delta_scan": (c_int, [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P]),
+    "mbh_delta_step": (c_int, [P, I, I, I, P, I, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, F, c_int, P]),
     "mbh_rows_axpy": (c_int, [P, P, P, I, I, I, I, c_int, P]),
 }
 
@@ -92,6 +96,12 @@ def _ptr(t: Optional[torch.Tensor]) -> Optional[int]:
     return t.data_ptr()
 
 
+def _rows(x: torch.Tensor):
+    """(pointer, elements between rows) of a matrix whose rows are contiguous: columns of a wider one are taken as they are."""
+    assert x.is_cuda and x.dim() == 2 and x.stride(1) == 1, "rows of contiguous elements"
+    return x.data_ptr(), max(x.stride(0), x.shape[1])
+
+
 def _stream() -> int:
     return torch.cuda.current_stream().cuda_stream
 
@@ -110,12 +120,22 @@ def embed_scale(tokens: torch.Tensor, table: torch.Tensor, scale: float, out: Op
     return out
 
 
-def rmsnorm(x32: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+def rmsnorm(x32: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0) -> torch.Tensor:
+    """offset 1: the weight is stored around zero."""
     T, D = x32.shape
     assert x32.dtype == torch.float32
     y = torch.empty(T, D, dtype=w.dtype, device=x32.device)
-    _check(lib().mbh_rmsnorm(_ptr(x32), _ptr(w), _ptr(y), T, D, eps, dt_of(w.dtype), _stream()), "mbh_rmsnorm")
+    _check(lib().mbh_rmsnorm(_ptr(x32), _ptr(w), None, _ptr(y), None, T, D, eps, offset, dt_of(w.dtype), _stream()), "mbh_rmsnorm")
     return y
+
+
+def rmsnorm_pair(x32: torch.Tensor, w: torch.Tensor, w2: torch.Tensor, eps: float, offset: float = 0.0):
+    """Two norms of the same rows, each with its own weight, in one pass."""
+    T, D = x32.shape
+    assert x32.dtype == torch.float32 and w.dtype == w2.dtype and w2.shape == w.shape
+    y, y2 = torch.empty(T, D, dtype=w.dtype, device=x32.device), torch.empty(T, D, dtype=w.dtype, device=x32.device)
+    _check(lib().mbh_rmsnorm(_ptr(x32), _ptr(w), _ptr(w2), _ptr(y), _ptr(y2), T, D, eps, offset, dt_of(w.dtype), _stream()), "mbh_rmsnorm")
+    return y, y2
 
 
 _ws: dict = {}
@@ -139,7 +159,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
            residual: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """x [M, K] @ w [N, K]^T with the epilogues of include/mistral_b200_hybrid.h.  EPI_RESIDUAL adds into `residual` (fp32, in
     place; EPI_RESIDUAL_SCALED: times `alpha`) and returns it; EPI_F32 returns fp32 [M, N] (soft-capped at `limit` when positive);
-    EPI_GLU returns [M, N/2]."""
+    EPI_GLU returns [M, N/2].  x may be columns of a wider matrix."""
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and x.dtype == w.dtype
@@ -154,13 +174,25 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     if _prompt_gemm_ok(x, M, N, K):
         # the framework's tcgen05 GEMM (bf16 out), then this library's epilogue over its result
         y = torch.empty(M, N, dtype=x.dtype, device=x.device)
-        _abi.linear_residual(x, w, None, y, _workspace(x.device))
+        _abi.linear_residual(x.contiguous(), w, None, y, _workspace(x.device))
         _check(lib().mbh_linear_epilogue(_ptr(y), _ptr(bias), _ptr(out), _ptr(out32), M, N, epi, n_act, limit, alpha, dt_of(x.dtype), _stream()),
                "mbh_linear_epilogue")
         return out if out is not None else out32
-    _check(lib().mbh_linear(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), _ptr(out32), M, N, K, epi, n_act, limit, alpha, dt_of(x.dtype), _stream()),
+    xp, ldx = _rows(x)
+    _check(lib().mbh_linear(xp, ldx, _ptr(w), _ptr(bias), _ptr(out), _ptr(out32), M, N, K, epi, n_act, limit, alpha, dt_of(x.dtype), _stream()),
            "mbh_linear")
     return out if out is not None else out32
+
+
+def linear_decay(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], a_log: torch.Tensor, group: int) -> torch.Tensor:
+    """fp32 [M, N] decays exp(-exp(a_log[n // group]) * softplus(x W^T + bias)); the sum is never rounded below fp32."""
+    M, K = x.shape
+    N = w.shape[0]
+    assert w.shape[1] == K and x.dtype == w.dtype and a_log.dtype == w.dtype and a_log.numel() * group == N
+    out = torch.empty(M, N, dtype=torch.float32, device=x.device)
+    xp, ldx = _rows(x)
+    _check(lib().mbh_linear_decay(xp, ldx, _ptr(w), _ptr(bias), _ptr(a_log), group, _ptr(out), M, N, K, dt_of(x.dtype), _stream()), "mbh_linear_decay")
+    return out
 
 
 def attn_prep(qkv, qnorm, knorm, positions, cache_rows, q_out, cache_k, cache_v, v_first, vmix, vmix_mode: int, H: int, G: int, d: int, e: int,
@@ -221,8 +253,8 @@ def layernorm(x32: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps
 
 
 # ------------------------------------------------------------------------------------------------ gated feed-forward, experts
-def linear_swiglu(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Tensor] = None, group: int = 0) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) with gate/up rows interleaved in w [2F, K]; column c is multiplied by rowscale[m, c // group]."""
+def linear_swiglu(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Tensor] = None, group: int = 0, gelu: bool = False) -> torch.Tensor:
+    """silu(x Wg^T) * (x Wu^T) (gelu: the tanh form of gelu instead of SiLU) with gate/up rows interleaved in w [2F, K]; column c is multiplied by rowscale[m, c // group]."""
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and x.dtype == w.dtype and N % 2 == 0
@@ -234,23 +266,26 @@ def linear_swiglu(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Ten
     if _prompt_gemm_ok(x, M, N, K):
         y = torch.empty(M, N, dtype=x.dtype, device=x.device)
         _abi.linear_residual(x, w, None, y, _workspace(x.device))
-        _check(lib().mbh_swiglu_epilogue(_ptr(y), _ptr(out), M, N, _ptr(rowscale), pitch, group, dt_of(x.dtype), _stream()), "mbh_swiglu_epilogue")
+        _check(lib().mbh_swiglu_epilogue(_ptr(y), _ptr(out), M, N, _ptr(rowscale), pitch, group, int(gelu), dt_of(x.dtype), _stream()),
+               "mbh_swiglu_epilogue")
         return out
-    _check(lib().mbh_linear_swiglu(_ptr(x), _ptr(w), _ptr(out), M, N, K, _ptr(rowscale), pitch, group, dt_of(x.dtype), _stream()), "mbh_linear_swiglu")
+    _check(lib().mbh_linear_swiglu(_ptr(x), _ptr(w), _ptr(out), M, N, K, _ptr(rowscale), pitch, group, int(gelu), dt_of(x.dtype), _stream()),
+           "mbh_linear_swiglu")
     return out
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], groups: int, keep: int, top: int, score: int = 0,
-              scale: float = 1.0):
+              scale: float = 1.0, group_two: bool = False, renorm: bool = False):
     """(dense fp32 [T, n], idx int32 [T, top], wsel fp32 [T, top]) of the fp32 router; score 0: softmax, 1: sigmoid; the weights are the
-    chosen scores times `scale`."""
+    chosen scores times `scale` (renorm: first divided by their sum).  group_two: a group of outputs counts the sum of its two largest
+    choices instead of its largest."""
     T, D = h.shape
     n = w_router.shape[0]
     dense = torch.empty(T, n, dtype=torch.float32, device=h.device)
     idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
     wsel = torch.empty(T, top, dtype=torch.float32, device=h.device)
     _check(lib().mbh_moe_route(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(dense), _ptr(idx), _ptr(wsel), T, D, n, groups, keep, top, score,
-                               scale, dt_of(h.dtype), _stream()), "mbh_moe_route")
+                               scale, int(group_two), int(renorm), dt_of(h.dtype), _stream()), "mbh_moe_route")
     return dense, idx, wsel
 
 
@@ -279,16 +314,20 @@ def rows_axpy(y32: torch.Tensor, h: torch.Tensor, dense: torch.Tensor, first: in
 
 # ------------------------------------------------------------------------------------------------ latent attention
 def latent_prep(y, qnorm, cnorm, freq, positions, cache_rows, ring, q_rank: int, kv_rank: int, rot_dim: int, rot_dims: int, eps: float,
-                mag: float) -> torch.Tensor:
+                mag: float, kv_off: Optional[int] = None, halves: bool = False, own: bool = False):
+    """(cq [T, q_rank] or None without a query latent, own [T, kv_rank + rot_dim] or None).  kv_off: column of the key/value latent in y
+    (default: after the query latent).  own: the tokens' latent rows are returned token-major; cache_rows given: they go to the ring."""
     assert freq.dtype == torch.float64 and freq.numel() == rot_dims // 2
     T = y.shape[0]
-    cq = torch.empty(T, q_rank, dtype=y.dtype, device=y.device)
-    _check(lib().mbh_latent_prep(_ptr(y), _ptr(qnorm), _ptr(cnorm), _ptr(freq), _ptr(positions), _ptr(cache_rows), _ptr(cq), _ptr(ring), T,
-                                 y.shape[1], q_rank, kv_rank, rot_dim, rot_dims, eps, mag, dt_of(y.dtype), _stream()), "mbh_latent_prep")
-    return cq
+    cq = torch.empty(T, q_rank, dtype=y.dtype, device=y.device) if q_rank else None
+    rows = torch.empty(T, kv_rank + rot_dim, dtype=y.dtype, device=y.device) if own else None
+    _check(lib().mbh_latent_prep(_ptr(y), _ptr(qnorm), _ptr(cnorm), _ptr(freq), _ptr(positions), _ptr(cache_rows), _ptr(cq),
+                                 _ptr(ring) if cache_rows is not None else None, T, y.shape[1], q_rank, q_rank if kv_off is None else kv_off, kv_rank, rot_dim,
+                                 rot_dims, int(halves), eps, mag, _ptr(rows), dt_of(y.dtype), _stream()), "mbh_latent_prep")
+    return cq, rows
 
 
-FLASH_SIZES = {(32, 32), (64, 32), (64, 64), (128, 64), (64, 128), (128, 128), (96, 64), (192, 128)}  # (key, value) sizes of the tensor-core prompt kernel
+FLASH_SIZES = {(32, 32), (64, 32), (64, 64), (128, 64), (64, 128), (128, 128), (96, 64), (96, 96), (48, 32), (192, 128)}  # (key, value) sizes of the tensor-core prompt kernel
 _iota: dict = {}
 
 
@@ -299,33 +338,36 @@ def iota(n: int, device: torch.device) -> torch.Tensor:
     return _iota[(device, n)]
 
 
-def latent_expand(kn, v, ring, positions, cache_rows, q_start, B: int, Wt: int, H: int, dn: int, rot_dim: int, dv: int, kv_rank: int):
-    kfull = torch.empty(B * Wt, H, dn + rot_dim, dtype=kn.dtype, device=kn.device)
-    vfull = torch.empty(B * Wt, H, dv, dtype=kn.dtype, device=kn.device)
-    _check(lib().mbh_latent_expand(_ptr(kn), _ptr(v), _ptr(ring), _ptr(positions), _ptr(cache_rows), _ptr(q_start), _ptr(kfull), _ptr(vfull), kn.shape[0],
-                                   B, Wt, H, dn, rot_dim, dv, kv_rank, dt_of(kn.dtype), _stream()), "mbh_latent_expand")
-    return kfull, vfull
+def latent_expand(kn, rows, H: int, dn: int, rot_dim: int, kv_rank: int) -> torch.Tensor:
+    """Keys per head [R, H, dn + rot_dim] of latent rows [R, kv_rank + rot_dim] and their up-projections kn [R, H * dn]."""
+    kfull = torch.empty(kn.shape[0], H, dn + rot_dim, dtype=kn.dtype, device=kn.device)
+    _check(lib().mbh_latent_expand(_ptr(kn), _ptr(rows), _ptr(kfull), kn.shape[0], H, dn, rot_dim, kv_rank, dt_of(kn.dtype), _stream()), "mbh_latent_expand")
+    return kfull
 
 
 def head_gate(out, gate, g_pitch: int, g_off: int, H: int, dv: int) -> None:
     _check(lib().mbh_head_gate(_ptr(out), _ptr(gate), g_pitch, g_off, out.shape[0], H, dv, dt_of(out.dtype), _stream()), "mbh_head_gate")
 
 
-def latent_absorb(q, w_uk, freq, positions, H: int, dn: int, rot_dim: int, rot_dims: int, kv_rank: int, mag: float) -> torch.Tensor:
-    """w_uk None: the queries are only rotated ([T, H * (dn + rot_dim)])."""
+def latent_absorb(q, w_uk, freq, positions, H: int, dn: int, rot_dim: int, rot_dims: int, kv_rank: int, mag: float,
+                  halves: bool = False) -> torch.Tensor:
+    """w_uk None: the queries are only rotated ([T, H * (dn + rot_dim)]).  q may be the first columns of a wider matrix."""
     T = q.shape[0]
     qa = torch.empty(T, H * ((kv_rank if w_uk is not None else dn) + rot_dim), dtype=q.dtype, device=q.device)
-    _check(lib().mbh_latent_absorb(_ptr(q), _ptr(w_uk), _ptr(freq), _ptr(positions), _ptr(qa), T, H, dn, rot_dim, rot_dims, kv_rank, mag,
+    qp, q_pitch = _rows(q)
+    _check(lib().mbh_latent_absorb(qp, q_pitch, _ptr(w_uk), _ptr(freq), _ptr(positions), _ptr(qa), T, H, dn, rot_dim, rot_dims, int(halves), kv_rank, mag,
                                    dt_of(q.dtype), _stream()), "mbh_latent_absorb")
     return qa
 
 
-def attn_latent(qa, ring, positions, q_start, slots, B: int, W: int, H: int, kv_rank: int, rot_dim: int, scale: float, splits: int = 1) -> torch.Tensor:
+def attn_latent(qa, ring, positions, q_start, slots, B: int, W: int, H: int, kv_rank: int, rot_dim: int, scale: float, splits: int = 1,
+                window: int = 0, own=None, seqpos=None, sink=None) -> torch.Tensor:
+    """window, own (this call's latent rows, token-major, with seqpos) and sink (fp32 [H]) as in attn_window."""
     T = qa.shape[0]
     o = torch.empty(T, H * kv_rank, dtype=qa.dtype, device=qa.device)
     scratch = torch.empty(T * H * splits * (2 + kv_rank), dtype=torch.float32, device=qa.device) if splits > 1 else None
     _check(lib().mbh_attn_latent(_ptr(qa), _ptr(ring), _ptr(positions), _ptr(q_start), _ptr(slots), _ptr(o), T, B, W, H, kv_rank, rot_dim, scale,
-                                 splits, _ptr(scratch), dt_of(qa.dtype), _stream()), "mbh_attn_latent")
+                                 splits, _ptr(scratch), window, _ptr(own), _ptr(seqpos), _ptr(sink), dt_of(qa.dtype), _stream()), "mbh_attn_latent")
     return o
 
 
@@ -338,12 +380,12 @@ def latent_decode_splits(B: int, W: int, n_sm: int = 148) -> int:
     return int(max(1, min((2 * n_sm) // B, (W + 63) // 64, 64)))
 
 
-def attn_latent_decode(qa, ring, positions, slots, B: int, W: int, H: int, kv_rank: int, rot_dim: int, scale: float) -> torch.Tensor:
+def attn_latent_decode(qa, ring, positions, slots, B: int, W: int, H: int, kv_rank: int, rot_dim: int, scale: float, window: int = 0, sink=None) -> torch.Tensor:
     splits = latent_decode_splits(B, W)
     o = torch.empty(B, H * kv_rank, dtype=qa.dtype, device=qa.device)
     scratch = torch.empty(B * H * splits * (2 + kv_rank), dtype=torch.float32, device=qa.device)
     _check(lib().mbh_attn_latent_decode(_ptr(qa), _ptr(ring), _ptr(positions), _ptr(slots), _ptr(o), B, W, H, kv_rank, rot_dim, scale, splits,
-                                        _ptr(scratch), dt_of(qa.dtype), _stream()), "mbh_attn_latent_decode")
+                                        _ptr(scratch), window, _ptr(sink), dt_of(qa.dtype), _stream()), "mbh_attn_latent_decode")
     return o
 
 
@@ -366,16 +408,18 @@ def embed_pos(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor
     return out
 
 
-def rot_prep(qkv, freq, positions, cache_rows, ring_k, ring_v, H: int, G: int, d: int, e: int, rot_dims: int, unit_norm: bool, eps: float, own: bool):
+def rot_prep(qkv, freq, positions, cache_rows, ring_k, ring_v, H: int, G: int, d: int, e: int, rot_dims: int, unit_norm: bool, eps: float, own: bool,
+             halves: bool = False, mag: float = 1.0):
     """(q [T, H*d], k [T, G*d] or None, v [T, G*e] or None): rotated (and unit-normed) queries and keys.  `own`: k and v are
-    returned token-major; `cache_rows` given: they are written into the ring rows as well."""
+    returned token-major; `cache_rows` given: they are written into the ring rows as well.  halves: pairs (i, i + rot_dims / 2) instead of
+    neighbours; mag: factor on cos and sin.  G = 0: queries only."""
     assert freq.dtype == torch.float64 and freq.numel() == rot_dims // 2
     T = qkv.shape[0]
     q = torch.empty(T, H * d, dtype=qkv.dtype, device=qkv.device)
     k = torch.empty(T, G * d, dtype=qkv.dtype, device=qkv.device) if own else None
     v = torch.empty(T, G * e, dtype=qkv.dtype, device=qkv.device) if own else None
     _check(lib().mbh_rot_prep(_ptr(qkv), _ptr(freq), _ptr(positions), _ptr(cache_rows), _ptr(q), _ptr(k), _ptr(v), _ptr(ring_k), _ptr(ring_v), T, H, G,
-                              d, e, rot_dims, int(unit_norm), eps, dt_of(qkv.dtype), _stream()), "mbh_rot_prep")
+                              d, e, rot_dims, int(halves), mag, int(unit_norm), eps, dt_of(qkv.dtype), _stream()), "mbh_rot_prep")
     return q, k, v
 
 
@@ -385,15 +429,18 @@ def kv_scatter(k, v, cache_rows, ring_k, ring_v) -> None:
 
 
 def attn_window(q, cache_k, cache_v, positions, q_start, slots, out, B: int, W: int, H: int, G: int, d: int, e: int, scale: float, window: int,
-                own_k=None, own_v=None, seqpos=None, n_tiles: int = 0, splits: int = 1, chunk: int = 0, head_bias=None) -> None:
+                own_k=None, own_v=None, seqpos=None, n_tiles: int = 0, splits: int = 1, chunk: int = 0, head_bias=None,
+                softcap: float = 0.0, sink=None) -> None:
     """`attn_bias` without a bias, with a sliding window (0: none) and, for prompts, this call's own keys and values beside the ring.
     chunk: keys per warp and step of the exact kernel (0: 128), see `window_decode_plan`.  head_bias (fp32 [H]): sigmoid weights instead
-    of the softmax, every visible key weighing sigmoid(score + head_bias[h]), not normalised."""
+    of the softmax, every visible key weighing sigmoid(score + head_bias[h]), not normalised.  softcap > 0: scores softcap * tanh(. / softcap); sink
+    (fp32 [H]): one more term exp(sink[h]) in the softmax denominator."""
     scratch = torch.empty(q.shape[0] * H * splits * (2 + e), dtype=torch.float32, device=q.device) if splits > 1 and n_tiles == 0 else None
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     assert head_bias is None or (head_bias.dtype == torch.float32 and head_bias.numel() == H)
     _check(lib().mbh_attn_window(_ptr(q), _ptr(cache_k), _ptr(cache_v), _ptr(head_bias), int(head_bias is not None), _ptr(positions), _ptr(q_start),
                                  _ptr(slots), _ptr(out), q.shape[0], B, W, H, G, d, e, scale, n_tiles, splits, _ptr(scratch), window, _ptr(own_k),
-                                 _ptr(own_v), _ptr(seqpos), chunk, int(head_bias is not None), dt_of(q.dtype), _stream()), "mbh_attn_window")
+                                 _ptr(own_v), _ptr(seqpos), chunk, int(head_bias is not None), softcap, _ptr(sink), dt_of(q.dtype), _stream()), "mbh_attn_window")
 
 
 def window_decode_plan(T: int, H: int, W: int):
@@ -557,4 +604,40 @@ def linear_relu2(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Tens
         _check(lib().mbh_relu2_epilogue(_ptr(y), _ptr(out), M, N, _ptr(rowscale), pitch, group, dt_of(x.dtype), _stream()), "mbh_relu2_epilogue")
         return out
     _check(lib().mbh_linear_relu2(_ptr(x), _ptr(w), _ptr(out), M, N, K, _ptr(rowscale), pitch, group, dt_of(x.dtype), _stream()), "mbh_linear_relu2")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------ gated delta rule
+def delta_prep(y, conv, cstate, positions, q_start, seqpos, slots, B: int, H: int, G: int, d: int, e: int):
+    """(qk fp32 [T, 2, G*d] unit queries (scaled) and keys, kq fp32 [T, G], v fp32 [T, H*e], beta fp32 [T, H]) of a prompt's tokens from the packed
+    projections y = q | k | v | beta logits | ...; advances the convolutions' carried inputs `cstate` (fp32 [rows, taps, 2*G*d + H*e])."""
+    T = y.shape[0]
+    assert cstate.dtype == torch.float32 and cstate.shape[1:] == (conv.shape[1], 2 * G * d + H * e) and conv.dtype == y.dtype
+    f = dict(dtype=torch.float32, device=y.device)
+    qk, kq, v, beta = torch.empty(T, 2, G * d, **f), torch.empty(T, G, **f), torch.empty(T, H * e, **f), torch.empty(T, H, **f)
+    _check(lib().mbh_delta_prep(_ptr(y), y.shape[1], _ptr(conv), conv.shape[1], _ptr(cstate), _ptr(positions), _ptr(q_start), _ptr(seqpos), _ptr(slots), _ptr(qk),
+                                _ptr(kq), _ptr(v), _ptr(beta), T, B, H, G, d, e, dt_of(y.dtype), _stream()), "mbh_delta_prep")
+    return qk, kq, v, beta
+
+
+def delta_scan(qk, kq, v, beta, g, state, q_start, seqpos, slots, B: int, H: int, G: int, d: int, e: int) -> torch.Tensor:
+    """fp32 o [T, H*e] of S <- diag(g) S; S <- S + k (beta (v - S^T k))^T; o = S^T q; state fp32 [rows, H, e, d] (columns of S are rows there)."""
+    T = qk.shape[0]
+    assert all(t.dtype == torch.float32 for t in (qk, kq, v, beta, g, state)) and state.shape[1:] == (H, e, d) and g.shape == (T, H * d)
+    o = torch.empty(T, H * e, dtype=torch.float32, device=qk.device)
+    _check(lib().mbh_delta_scan(_ptr(qk), _ptr(kq), _ptr(v), _ptr(beta), _ptr(g), _ptr(state), _ptr(q_start), _ptr(seqpos), _ptr(slots), _ptr(o), B, H, G, d, e,
+                                _stream()), "mbh_delta_scan")
+    return o
+
+
+def delta_step(y, ra: int, rg: int, conv, cstate, state, w_a2, dt_bias, a_log, w_g2, norm, positions, seqpos, slots, H: int, G: int, d: int, e: int,
+               eps: float) -> torch.Tensor:
+    """[B, H*e]: one token per sequence through convolutions, decays, state step, head norm and output gate in one launch."""
+    B = y.shape[0]
+    assert cstate.dtype == torch.float32 and state.dtype == torch.float32 and state.shape[1:] == (H, e, d)
+    assert cstate.shape[1:] == (conv.shape[1], 2 * G * d + H * e) and w_a2.shape == (H * d, ra) and w_g2.shape == (H * e, rg)
+    out = torch.empty(B, H * e, dtype=y.dtype, device=y.device)
+    _check(lib().mbh_delta_step(_ptr(y), y.shape[1], ra, rg, _ptr(conv), conv.shape[1], _ptr(cstate), _ptr(state), _ptr(w_a2), _ptr(dt_bias), _ptr(a_log),
+                                _ptr(w_g2), _ptr(norm), _ptr(positions), _ptr(seqpos), _ptr(slots), _ptr(out), B, H, G, d, e, eps, dt_of(y.dtype), _stream()),
+           "mbh_delta_step")
     return out

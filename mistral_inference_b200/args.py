@@ -128,6 +128,10 @@ class RotScalingArgs:
     fast: float
     slow: float
 
+    @classmethod
+    def from_dict(cls, d: Optional[dict]) -> Optional["RotScalingArgs"]:
+        return cls(float(d["factor"]), float(d["original"]), float(d["fast"]), float(d["slow"])) if d else None
+
 
 @dataclass
 class LatentAttentionArgs:
@@ -138,21 +142,36 @@ class LatentAttentionArgs:
     dim: int
     rot_dim: int
     vdim: int
-    q_rank: int
+    q_rank: int              # 0: no query latent, the queries are one projection of the input
     kv_rank: int
     scale: float
     rot_base: float
     rot_dims: int
     rot_scaling: Optional[RotScalingArgs] = None
+    window: Optional[int] = None   # sliding window, the token itself included; None: the whole sequence
+    rot_halves: bool = False       # rotated pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)
+    sink: bool = False             # a learned term per head in the softmax denominator
+    head_gate: bool = True         # sigmoid gate per head on the output
 
     @classmethod
     def from_dict(cls, d: dict) -> "LatentAttentionArgs":
         rot = d["rot"]
-        sc = rot.get("scaling")
         a = cls(heads=int(d["heads"]), dim=int(d["dim"]), rot_dim=int(d["rot_dim"]), vdim=int(d["vdim"]), q_rank=int(d["q_rank"]),
                 kv_rank=int(d["kv_rank"]), scale=float(d["scale"]), rot_base=float(rot["base"]), rot_dims=int(rot.get("dims", d["rot_dim"])),
-                rot_scaling=RotScalingArgs(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])) if sc else None)
+                rot_scaling=RotScalingArgs.from_dict(rot.get("scaling")))
         assert a.rot_dims <= a.rot_dim and a.rot_dims % 2 == 0, "the rotation covers an even number of the rotated entries"
+        return a
+
+
+class SinkLatentAttentionArgs(LatentAttentionArgs):
+    """Latent attention without a query latent and without an output gate: rotated halves, a sliding window, a sink per head."""
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "SinkLatentAttentionArgs":
+        a = super().from_dict({**d, "q_rank": 0})
+        a.window = int(d["mask"]["size"]) if d.get("mask") else None
+        a.rot_halves, a.sink, a.head_gate = True, True, False
+        assert a.window is None or a.window >= 1
         return a
 
 
@@ -199,6 +218,12 @@ class RotaryAttentionArgs:
     rot_dims: int = 0          # 0: no rotation
     rot_factor: float = 1.0    # linear scaling: every frequency divided by it
     unit_norm: bool = True
+    rot_scaling: Optional[RotScalingArgs] = None
+    rot_halves: bool = False   # rotated pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)
+    qkv_bias: bool = False
+    softcap: float = 0.0       # > 0: score <- softcap * tanh(score / softcap)
+    sink: bool = False         # a learned term per head in the softmax denominator
+    kv_from: Optional[int] = None  # the layer has queries only and attends to the keys and values that this earlier layer cached
 
     @classmethod
     def from_dict(cls, d: dict) -> "RotaryAttentionArgs":
@@ -209,6 +234,40 @@ class RotaryAttentionArgs:
         assert a.heads % a.kv_heads == 0, "query heads must be a multiple of key/value heads"
         assert a.rot_dims <= a.dim and a.rot_dims % 2 == 0, "the rotation covers an even number of a head's entries"
         assert a.window is None or a.window >= 1
+        return a
+
+
+class CappedAttentionArgs(RotaryAttentionArgs):
+    """Rotary attention with biases on q, k and v, rotated halves under frequency scaling, soft-capped scores, a sink per head, no unit norm;
+    a layer may read the keys and values of an earlier one (`kv_from`)."""
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "CappedAttentionArgs":
+        rot = d.get("rot") or {}
+        a = super().from_dict({**d, "rot": {k: v for k, v in rot.items() if k != "scaling"}})
+        a.rot_scaling = RotScalingArgs.from_dict(rot.get("scaling"))
+        a.unit_norm, a.rot_halves, a.qkv_bias, a.sink = False, True, True, True
+        a.softcap = float(d.get("softcap") or 0.0)
+        a.kv_from = int(d["kv_from"]) if d.get("kv_from") is not None else None
+        return a
+
+
+@dataclass
+class DeltaArgs:
+    """Gated delta rule: S <- diag(g) S; S <- S + k (beta (v - S^T k))^T; o = S^T q, with a decay g per head and key channel, unit queries and
+    keys shared by heads / kv_heads value heads, and short causal convolutions (`conv` taps) on q, k and v.  fp32 state [heads, vdim, dim] and the
+    convolutions' last inputs per sequence."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "DeltaArgs":
+        a = cls(heads=int(d["heads"]), kv_heads=int(d["kv_heads"]), dim=int(d["dim"]), vdim=int(d["vdim"]), conv=int(d["conv"]))
+        assert a.heads % a.kv_heads == 0, "heads must be a multiple of key heads"
+        assert a.conv >= 1, "conv >= 1"
         return a
 
 
@@ -355,14 +414,48 @@ class Relu2MoeArgs:
         return a
 
 
+@dataclass
+class GeluGluArgs:
+    """Dense feed-forward W_down (gelu(W_gate h) * (W_up h)), the tanh form of gelu."""
+    ff: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GeluGluArgs":
+        return cls(ff=int(d["ff"]))
+
+
+@dataclass
+class GroupedMoeArgs:
+    """Mixture of gated (SiLU) experts with an fp32 sigmoid router: the choice adds a per-expert correction and is limited to the best `keep` of
+    `groups` groups of neighbouring experts (a group counts its two largest choices); the chosen scores are divided by their sum and
+    multiplied by router_scale.  An optional shared expert of size `shared_ff` runs for every token behind a sigmoid gate of one number."""
+    ff: int
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    router_scale: float = 1.0
+    shared_ff: int = 0
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "GroupedMoeArgs":
+        r, g, sh = d["router"], d["router"].get("groups") or {}, d.get("shared")
+        a = cls(ff=int(d["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=int(g.get("count", 1)),
+                keep=int(g.get("keep", g.get("count", 1))), router_scale=float(r.get("scale", 1.0)), shared_ff=int(sh["ff"]) if sh else 0)
+        assert a.experts % a.groups == 0 and 1 <= a.keep <= a.groups, "router groups must be equal and keep <= count"
+        assert 1 <= a.top <= a.experts // a.groups * a.keep, "more experts per token than the kept groups hold"
+        return a
+
+
 MLP_ARGS = {"dense": ClampedGluArgs, "moe": MoeFfArgs}
 
 
 @dataclass
 class LayerArgs:
     type: str                                             # a key of MIXER_ARGS
-    mixer: Union[BiasedAttentionArgs, LightningArgs, LatentAttentionArgs, SideBySideArgs, MlstmArgs, RetentionArgs, GlaArgs, SigmoidAttentionArgs]
-    mlp: Union[None, ClampedGluArgs, MoeFfArgs, ScaledInputMoeArgs, Relu2MoeArgs]
+    mixer: Union[BiasedAttentionArgs, LightningArgs, LatentAttentionArgs, SideBySideArgs, MlstmArgs, RetentionArgs, GlaArgs, SigmoidAttentionArgs,
+                 CappedAttentionArgs, SinkLatentAttentionArgs, DeltaArgs]
+    mlp: Union[None, ClampedGluArgs, MoeFfArgs, ScaledInputMoeArgs, Relu2MoeArgs, GeluGluArgs, GroupedMoeArgs]
 
 
 MIXER_ARGS = {"attention": BiasedAttentionArgs, "lightning": LightningArgs, "latent_attention": LatentAttentionArgs,
@@ -390,9 +483,11 @@ DESIGNS = {
     "Taruvik": {"norm": "layer", "post_norm": True},
     "Lotazen": {"norm": "rms_scalar", "post_norm": False, "parallel_block": True, "learned_positions": True},
     "Viladra": {"norm": "rms", "post_norm": True, "pre_norm": False, "canon": True, "depth_average": True, "tied_head": True},
+    "Dimorax": {"norm": "rms_around_one", "post_norm": False, "parallel_block": True, "parallel_norms": 2},
 }
-DESIGN_MLP_ARGS = {"Lotazen": {"moe": ScaledInputMoeArgs}, "Viladra": {"moe": Relu2MoeArgs}}
-DESIGN_MIXER_ARGS = {"Viladra": {"attention": SigmoidAttentionArgs, "retention": RetentionArgs, "gla": GlaArgs}}
+DESIGN_MLP_ARGS = {"Lotazen": {"moe": ScaledInputMoeArgs}, "Viladra": {"moe": Relu2MoeArgs}, "Dimorax": {"dense": GeluGluArgs, "moe": GroupedMoeArgs}}
+DESIGN_MIXER_ARGS = {"Viladra": {"attention": SigmoidAttentionArgs, "retention": RetentionArgs, "gla": GlaArgs},
+                     "Dimorax": {"attention": CappedAttentionArgs, "latent_attention": SinkLatentAttentionArgs, "channel_delta": DeltaArgs}}
 
 
 @dataclass
@@ -405,10 +500,13 @@ class LayeredArgs:
     norm_eps: float
     layers: List[LayerArgs]
     max_batch_size: int = 0
-    norm: str = "rms"            # "rms": weight only; "rms_scalar": one number as weight; "layer": mean removed, weight and bias
+    norm: str = "rms"            # "rms": weight only; "rms_around_one": weight stored as its distance from 1; "rms_scalar": one number as
+                                 # weight; "layer": mean removed, weight and bias
     post_norm: bool = False      # x <- x + norm_b(sublayer(norm(x))) instead of x <- x + sublayer(norm(x))
     loop: Optional[LoopArgs] = None
     parallel_block: bool = False     # h = norm1(x); x <- x + mixer(h) + ff(h): one norm per layer, both sublayers read it
+    parallel_norms: int = 1          # 2: each sublayer of a parallel block has a norm of its own, x <- x + m (mixer(norm1(x)) + ff(norm2(x)))
+    residual_mult: float = 1.0       # m above: what the sublayers' results are multiplied by on their way into the stream
     learned_positions: bool = False  # x = embed[token] + pos[position]; max_positions rows
     max_positions: int = 0
     logit_softcap: float = 0.0       # > 0: logits <- cap * tanh(logits / cap)
@@ -453,6 +551,16 @@ class LayeredArgs:
                     raise ValueError(f"unknown feed-forward kind {kind!r}")
                 mlp = mlp_args[kind].from_dict(L["mlp"])
             layers.append(LayerArgs(type=L["type"], mixer=mixer_args[L["type"]].from_dict(L["mixer"]), mlp=mlp))
+        for i, L in enumerate(layers):
+            j = getattr(L.mixer, "kv_from", None)
+            if j is not None:
+                assert 0 <= j < i and type(layers[j].mixer) is type(L.mixer), f"layer {i}: kv_from names an earlier layer of the same kind"
+                src = layers[j].mixer
+                assert src.kv_from is None and src.window is None and L.mixer.window is None, "the layer that owns the keys keeps the whole sequence"
+                assert (src.kv_heads, src.dim, src.vdim) == (L.mixer.kv_heads, L.mixer.dim, L.mixer.vdim), "shared keys and values have the sizes of their layer"
+        if d.get("residual_mult") is not None:
+            design["residual_mult"] = float(d["residual_mult"])
+            assert design.get("parallel_norms") == 2 or design["residual_mult"] == 1.0, "a factor on the sublayers' results belongs to blocks with two parallel norms"
         loop = None
         if d.get("loop"):
             lp = d["loop"]

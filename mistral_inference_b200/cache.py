@@ -42,7 +42,8 @@ class LayerCacheSpec:
     dtype (window None = the whole sequence).  kind "state": one fp32 tensor of `state_shape`, carried from token to token.  A ring
     layer with a non-empty `state_shape` keeps both (a layer whose mixer is an attention beside a recurrence).  `conv_shape`: beside
     either, an fp32 tensor with the last inputs of the layer's short convolutions over time (a layer whose sublayers read their
-    input through a causal convolution)."""
+    input through a causal convolution, or a mixer with convolutions of its own).  kind "shared": nothing of its own, the layer reads the
+    ring of layer run `source`."""
     kind: str = "ring"
     n_kv_heads: int = 0
     k_dim: int = 0
@@ -50,6 +51,7 @@ class LayerCacheSpec:
     window: Optional[int] = None
     state_shape: Tuple[int, ...] = ()
     conv_shape: Tuple[int, ...] = ()
+    source: int = -1
 
 
 @dataclass
@@ -124,6 +126,10 @@ class BufferCache:
             if sp is None:
                 self.cache_k[i] = torch.empty((max_batch_size, cache_size, n_kv_heads, head_dim))
                 self.cache_v[i] = torch.empty((max_batch_size, cache_size, n_kv_heads, head_dim))
+            elif sp.kind == "shared":
+                assert 0 <= sp.source < i and layer_specs[sp.source].kind == "ring" and layer_specs[sp.source].window is None, (
+                    "a shared entry reads the whole-sequence ring of an earlier layer run")
+                continue
             elif sp.kind == "ring":
                 self.cache_k[i] = torch.empty((max_batch_size, cache_size, sp.n_kv_heads, sp.k_dim))
                 self.cache_v[i] = torch.empty((max_batch_size, cache_size, sp.n_kv_heads, sp.v_dim))
@@ -140,7 +146,9 @@ class BufferCache:
     # -- reference API --------------------------------------------------------------------------
     def get_view(self, layer_id: int, metadata: CacheInputMetadata) -> CacheView:
         assert self._kv_seqlens_host is not None
-        return CacheView(self.cache_k.get(layer_id), self.cache_v.get(layer_id), metadata, self._kv_seqlens_host,
+        sp = self.layer_specs[layer_id] if self.layer_specs is not None else None
+        ring = sp.source if sp is not None and sp.kind == "shared" else layer_id
+        return CacheView(self.cache_k.get(ring), self.cache_v.get(ring), metadata, self._kv_seqlens_host,
                          state=self.cache_state.get(layer_id), conv=self.cache_conv.get(layer_id))
 
     def reset(self) -> None:

@@ -9,6 +9,7 @@
 #include "hybrid_rotary.cuh"
 #include "hybrid_gated_scan.cuh"
 #include "hybrid_stream.cuh"
+#include "hybrid_delta.cuh"
 #include "../../../include/mistral_b200_hybrid.h"
 
 #include <stdio.h>
@@ -102,14 +103,15 @@ template <typename T> static void run_layernorm(const void* x32, const void* w, 
 }
 template <typename T> static void run_attn_wide(const AttnArgs& a, size_t smem, cudaStream_t st) {
     attn_bias_kernel<T, AT_MAXR_WIDE><<<dim3((unsigned)(a.T * a.H), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
-    if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid);
+    if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H);
 }
 template <typename T> static void run_moe_sparse(const MoeSparseArgs& a, int64_t T_, cudaStream_t st) {
     moe_gateup_sparse_kernel<T><<<dim3((unsigned)((a.ff + MOE_WARPS - 1) / MOE_WARPS), (unsigned)(T_ * a.top)), MOE_WARPS * 32, 0, st>>>(a);
     moe_down_sparse_kernel<T><<<dim3((unsigned)((a.width + MOE_WARPS - 1) / MOE_WARPS), (unsigned)T_), MOE_WARPS * 32, 0, st>>>(a);
 }
-template <typename T> static void run_rmsnorm(const void* x32, const void* w, void* y, int64_t T_, int64_t D, float eps, cudaStream_t st) {
-    rmsnorm_f32_kernel<T><<<(unsigned)T_, D >= 1024 ? 256 : 128, 0, st>>>((const float*)x32, (const T*)w, (T*)y, (int)D, eps);
+template <typename T> static void run_rmsnorm(const void* x32, const void* w, const void* w2, void* y, void* y2, int64_t T_, int64_t D, float eps, float offset,
+                                              cudaStream_t st) {
+    rmsnorm_f32_kernel<T><<<(unsigned)T_, D >= 1024 ? 256 : 128, 0, st>>>((const float*)x32, (const T*)w, (const T*)w2, (T*)y, (T*)y2, (int)D, eps, offset);
 }
 template <typename T> static void run_epilogue(const LinearArgs& a, const void* y, cudaStream_t st) {
     const size_t pairs = (size_t)a.M * (a.N >> 1);
@@ -118,27 +120,64 @@ template <typename T> static void run_epilogue(const LinearArgs& a, const void* 
 template <typename T> static void run_prep(const AttnPrepArgs& a, int64_t T_, cudaStream_t st) { attn_prep_kernel<T><<<(unsigned)T_, 128, 0, st>>>(a); }
 template <typename T> static void run_attn(const AttnArgs& a, size_t smem, cudaStream_t st) {
     attn_bias_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
-    if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid);
+    if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H);
 }
 template <typename T> static void run_headnorm(const void* o32, const void* w, const void* g, int64_t g_pitch, int64_t g_off, void* y, int64_t T_,
                                                int64_t N, float eps, cudaStream_t st) {
     gated_headnorm_kernel<T><<<(unsigned)T_, 128, 0, st>>>((const float*)o32, (const T*)w, (const T*)g, (int)g_pitch, (int)g_off, (T*)y, (int)N, eps);
 }
 
-template <typename T, int HPW> static cudaError_t run_latent_decode(const LatentDecodeArgs& a, void* out, size_t smem, cudaStream_t st) {
+template <typename T, int HPW> static cudaError_t run_latent_decode(const LatentDecodeArgs& a, void* out, const float* sink, size_t smem, cudaStream_t st) {
     cudaError_t e = cudaFuncSetAttribute(attn_latent_decode_kernel<T, HPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e) return e;
     attn_latent_decode_kernel<T, HPW><<<dim3((unsigned)a.B, (unsigned)a.splits), LD_WARPS * 32, smem, st>>>(a);
-    attn_merge_kernel<T><<<dim3((unsigned)(a.B * a.H), (unsigned)((a.kv_rank + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)out, a.splits, a.kv_rank);
+    attn_merge_kernel<T><<<dim3((unsigned)(a.B * a.H), (unsigned)((a.kv_rank + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)out, a.splits, a.kv_rank, 0, sink, a.H);
     return cudaGetLastError();
 }
-template <typename T> static cudaError_t launch_latent_decode(const LatentDecodeArgs& a, void* out, cudaStream_t st) {
+template <typename T> static cudaError_t launch_latent_decode(const LatentDecodeArgs& a, void* out, const float* sink, cudaStream_t st) {
     const int d = a.kv_rank + a.rot_dim, kp = d + (sizeof(T) == 2 ? 2 : 1);
     const size_t smem = sizeof(float) * ((size_t)a.H * d + (size_t)a.H * LD_KT) + sizeof(T) * (size_t)LD_KT * kp;
     if (smem > 220 * 1024) return cudaErrorInvalidValue;
-    if (a.H <= LD_WARPS) return run_latent_decode<T, 1>(a, out, smem, st);
-    if (a.H <= 2 * LD_WARPS) return run_latent_decode<T, 2>(a, out, smem, st);
-    return run_latent_decode<T, 4>(a, out, smem, st);
+    if (a.H <= LD_WARPS) return run_latent_decode<T, 1>(a, out, sink, smem, st);
+    if (a.H <= 2 * LD_WARPS) return run_latent_decode<T, 2>(a, out, sink, smem, st);
+    return run_latent_decode<T, 4>(a, out, sink, smem, st);
+}
+
+// key size -> lanes per state column and float4 per lane; tokens per shared-memory tile
+static cudaError_t launch_delta_scan(const DeltaArgs& a, cudaStream_t st) {
+    auto grid = [&](int lanes) { return dim3((unsigned)(a.B * a.H), (unsigned)((a.e + DS_THREADS / lanes - 1) / (DS_THREADS / lanes))); };
+    if (a.d <= 32) delta_scan_kernel<8, 1, 16><<<grid(8), DS_THREADS, 0, st>>>(a);
+    else if (a.d <= 64) delta_scan_kernel<8, 2, 16><<<grid(8), DS_THREADS, 0, st>>>(a);
+    else if (a.d <= 128) delta_scan_kernel<8, 4, 8><<<grid(8), DS_THREADS, 0, st>>>(a);
+    else if (a.d <= 256) delta_scan_kernel<8, 8, 4><<<grid(8), DS_THREADS, 0, st>>>(a);
+    else delta_scan_kernel<32, 8, 1><<<grid(32), DS_THREADS, 0, st>>>(a);
+    return cudaGetLastError();
+}
+template <typename T> static cudaError_t launch_delta_prep(const DeltaArgs& a, cudaStream_t st) {
+    // few tokens: the units of a token are spread over CTAs; long prompts: each CTA walks several units of its tokens
+    const unsigned tiles = (unsigned)((a.T + DP_WARPS - 1) / DP_WARPS), units = (unsigned)(a.G + a.H);
+    const dim3 grid(tiles, units < 65535u ? units : 65535u);
+    if (a.d <= 64) delta_prep_kernel<T, 2><<<grid, DP_WARPS * 32, 0, st>>>(a);
+    else if (a.d <= 128) delta_prep_kernel<T, 4><<<grid, DP_WARPS * 32, 0, st>>>(a);
+    else if (a.d <= 256) delta_prep_kernel<T, 8><<<grid, DP_WARPS * 32, 0, st>>>(a);
+    else delta_prep_kernel<T, 32><<<grid, DP_WARPS * 32, 0, st>>>(a);
+    if (a.taps > 1) delta_conv_state_kernel<T><<<dim3((unsigned)a.B, (unsigned)((2 * a.G * a.d + a.H * a.e + 255) / 256)), 256, 0, st>>>(a);
+    return cudaGetLastError();
+}
+template <typename T, int LANES, int RPL4> static cudaError_t run_delta_step(const DeltaArgs& a, cudaStream_t st) {
+    const size_t smem = sizeof(float) * (5 * (size_t)DeltaColumn<LANES, RPL4>::DMAX + 3 * (size_t)a.e + a.ra + a.rg);
+    if (smem > 220 * 1024) return cudaErrorInvalidValue;
+    cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, LANES, RPL4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e) return e;
+    delta_step_kernel<T, LANES, RPL4><<<(unsigned)(a.B * a.H), DT_THREADS, smem, st>>>(a);
+    return cudaGetLastError();
+}
+template <typename T> static cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st) {
+    if (a.d <= 32) return run_delta_step<T, 8, 1>(a, st);
+    if (a.d <= 64) return run_delta_step<T, 8, 2>(a, st);
+    if (a.d <= 128) return run_delta_step<T, 8, 4>(a, st);
+    if (a.d <= 256) return run_delta_step<T, 8, 8>(a, st);
+    return run_delta_step<T, 32, 8>(a, st);
 }
 
 extern "C" {
@@ -154,22 +193,37 @@ int mbh_embed_scale(const void* tokens, const void* table, float scale, void* x3
     return e ? fail(e, "mbh_embed_scale") : 0;
 }
 
-int mbh_rmsnorm(const void* x32, const void* w, void* y, int64_t T, int64_t D, float eps, int dt, void* stream) {
+int mbh_rmsnorm(const void* x32, const void* w, const void* w2, void* y, void* y2, int64_t T, int64_t D, float eps, float offset, int dt, void* stream) {
     if (T == 0) return 0;
+    if (!w2 != !y2) return bad("mbh_rmsnorm: a second norm needs its weight and its output");
     cudaStream_t st = (cudaStream_t)stream;
-    DISPATCH(dt, run_rmsnorm<ST>(x32, w, y, T, D, eps, st));
+    DISPATCH(dt, run_rmsnorm<ST>(x32, w, w2, y, y2, T, D, eps, offset, st));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_rmsnorm") : 0;
 }
 
-int mbh_linear(const void* x, const void* w, const void* bias, void* out, void* out32, int64_t M, int64_t N, int64_t K, int epi, int64_t n_act,
+int mbh_linear(const void* x, int64_t ldx, const void* w, const void* bias, void* out, void* out32, int64_t M, int64_t N, int64_t K, int epi, int64_t n_act,
                float limit, float alpha, int dt, void* stream) {
+    if (ldx < K) return bad("mbh_linear: rows of x overlap");
     if ((epi < 0 || epi > 3) && epi != EPI_RESIDUAL_SCALED) return bad("mbh_linear: unknown epilogue");  // EPI_SWIGLU: mbh_linear_swiglu
     if (epi == EPI_GLU && (N & 1)) return bad("mbh_linear: the gated epilogue needs interleaved (even) rows");
     LinearArgs a{x, w, bias, out, (float*)out32, (int)M, (int)N, (int)K, epi, (int)n_act, limit, alpha};
+    a.ldx = (int)ldx;
     cudaError_t e = cudaSuccess;
     DISPATCH(dt, e = launch_linear<ST>(a, (cudaStream_t)stream));
     return e ? fail(e, "mbh_linear") : 0;
+}
+
+int mbh_linear_decay(const void* x, int64_t ldx, const void* w, const void* bias, const void* a_log, int64_t group, void* out32, int64_t M, int64_t N, int64_t K,
+                     int dt, void* stream) {
+    if (ldx < K) return bad("mbh_linear_decay: rows of x overlap");
+    if (group < 1 || N % group) return bad("mbh_linear_decay: a_log covers equal groups of the outputs");
+    LinearArgs a{x, w, bias, nullptr, (float*)out32, (int)M, (int)N, (int)K, EPI_DECAY, 0, 0.f, 0.f, nullptr, 0, (int)group};
+    a.a_log = a_log;
+    a.ldx = (int)ldx;
+    cudaError_t e = cudaSuccess;
+    DISPATCH(dt, e = launch_linear<ST>(a, (cudaStream_t)stream));
+    return e ? fail(e, "mbh_linear_decay") : 0;
 }
 
 int mbh_linear_epilogue(const void* y, const void* bias, void* out, void* out32, int64_t M, int64_t N, int epi, int64_t n_act, float limit, float alpha,
@@ -199,15 +253,16 @@ int mbh_attn_bias(const void* q, const void* cache_k, const void* cache_v, const
                   const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
                   float scale, int64_t n_tiles, int64_t splits, void* scratch, int dt, void* stream) {
     return mbh_attn_window(q, cache_k, cache_v, bias_tab, n_tab, positions, q_start, slots, out, T, B, W, H, G, d, e, scale, n_tiles, splits, scratch,
-                           0, nullptr, nullptr, nullptr, 0, 0, dt, stream);
+                           0, nullptr, nullptr, nullptr, 0, 0, 0.f, nullptr, dt, stream);
 }
 
 int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, const void* bias_tab, int64_t n_tab, const void* positions,
                     const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
                     float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, const void* own_k, const void* own_v,
-                    const void* seqpos, int64_t chunk, int weights, int dt, void* stream) {
+                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, int dt, void* stream) {
     if (T == 0) return 0;
     if (weights != 0 && weights != 1) return bad("mbh_attn_window: weights are 0 (softmax) or 1 (sigmoid)");
+    if (weights == 1 && (softcap > 0.f || sink)) return bad("mbh_attn_window: a soft cap and sinks belong to the softmax");
     if (chunk < 0 || chunk > AT_CHUNK) return bad("mbh_attn_window: chunk is 0 (default) or 1 .. 128 keys");
     if (e > 32 * AT_MAXR) return bad("mbh_attn_bias: value size above 256");
     if (H % G) return bad("mbh_attn_bias: heads must be a multiple of kv heads");
@@ -215,7 +270,7 @@ int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, con
     if (window < 0 || (!own_k != !own_v) || (own_k && !seqpos)) return bad("mbh_attn_window: window >= 0; own keys, own values and seqpos come together");
     AttnArgs a{q, cache_k, cache_v, (const float*)bias_tab, (int)n_tab, (const int*)positions, (const int*)q_start, (const int*)slots, out,
                (int)T, (int)B, (int)W, (int)H, (int)G, (int)d, (int)e, scale, (int)(splits > 1 && scratch ? splits : 1), (float*)scratch, 0, 0,
-               (int)window, own_k, own_v, (const int*)seqpos, (int)chunk, weights};
+               (int)window, own_k, own_v, (const int*)seqpos, (int)chunk, softcap, (const float*)sink, 0, 0, weights};
     const size_t smem = sizeof(float) * ((size_t)d + AT_WARPS * AT_CHUNK + AT_WARPS * (2 + 32 * AT_MAXR));
     cudaStream_t st = (cudaStream_t)stream;
     // prompts in bf16: the tensor-core kernel, when the caller counted the 64-query tiles and the sizes are instantiated
@@ -266,21 +321,21 @@ int mbh_layernorm(const void* x32, const void* w, const void* b, void* y, void* 
 }
 
 int mbh_linear_swiglu(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, const void* rowscale, int64_t rs_pitch,
-                      int64_t rs_group, int dt, void* stream) {
+                      int64_t rs_group, int act, int dt, void* stream) {
     if (N & 1) return bad("mbh_linear_swiglu: the gated epilogue needs interleaved (even) rows");
     if (rowscale && rs_group <= 0) return bad("mbh_linear_swiglu: rs_group must be positive");
-    LinearArgs a{x, w, nullptr, out, nullptr, (int)M, (int)N, (int)K, EPI_SWIGLU, 0, 0.f, 0.f, (const float*)rowscale, (int)rs_pitch, (int)rs_group};
+    LinearArgs a{x, w, nullptr, out, nullptr, (int)M, (int)N, (int)K, act ? EPI_GEGLU : EPI_SWIGLU, 0, 0.f, 0.f, (const float*)rowscale, (int)rs_pitch, (int)rs_group};
     cudaError_t e = cudaSuccess;
     DISPATCH(dt, e = launch_linear<ST>(a, (cudaStream_t)stream));
     return e ? fail(e, "mbh_linear_swiglu") : 0;
 }
 
-int mbh_swiglu_epilogue(const void* y, void* out, int64_t M, int64_t N, const void* rowscale, int64_t rs_pitch, int64_t rs_group, int dt,
+int mbh_swiglu_epilogue(const void* y, void* out, int64_t M, int64_t N, const void* rowscale, int64_t rs_pitch, int64_t rs_group, int act, int dt,
                         void* stream) {
     if (N & 1) return bad("mbh_swiglu_epilogue: odd N");
     if (rowscale && rs_group <= 0) return bad("mbh_swiglu_epilogue: rs_group must be positive");
     if (M == 0) return 0;
-    LinearArgs a{nullptr, nullptr, nullptr, out, nullptr, (int)M, (int)N, 0, EPI_SWIGLU, 0, 0.f, 0.f, (const float*)rowscale, (int)rs_pitch, (int)rs_group};
+    LinearArgs a{nullptr, nullptr, nullptr, out, nullptr, (int)M, (int)N, 0, act ? EPI_GEGLU : EPI_SWIGLU, 0, 0.f, 0.f, (const float*)rowscale, (int)rs_pitch, (int)rs_group};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, run_epilogue<ST>(a, y, st));
     cudaError_t e = cudaGetLastError();
@@ -288,37 +343,36 @@ int mbh_swiglu_epilogue(const void* y, void* out, int64_t M, int64_t N, const vo
 }
 
 int mbh_latent_prep(const void* y, const void* qnorm, const void* cnorm, const void* freq, const void* positions, const void* cache_rows, void* cq,
-                    void* ring, int64_t T, int64_t pitch, int64_t q_rank, int64_t kv_rank, int64_t rot_dim, int64_t rot_dims, float eps, float mag,
-                    int dt, void* stream) {
+                    void* ring, int64_t T, int64_t pitch, int64_t q_rank, int64_t kv_off, int64_t kv_rank, int64_t rot_dim, int64_t rot_dims, int halves, float eps,
+                    float mag, void* own, int dt, void* stream) {
     if (T == 0) return 0;
+    if (cache_rows && !ring) return bad("mbh_latent_prep: ring rows without a ring");
     if (rot_dims > rot_dim || (rot_dims & 1)) return bad("mbh_latent_prep: rot_dims must be even and at most rot_dim");
     LatentPrepArgs a{y, qnorm, cnorm, (const double*)freq, (const int*)positions, (const int*)cache_rows, cq, ring,
-                     (int)q_rank, (int)kv_rank, (int)rot_dim, (int)rot_dims, (int)pitch, eps, mag};
+                     (int)q_rank, (int)kv_rank, (int)rot_dim, (int)rot_dims, (int)pitch, eps, mag, (int)kv_off, halves, own};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, latent_prep_kernel<ST><<<(unsigned)T, 128, 0, st>>>(a));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_latent_prep") : 0;
 }
 
-int mbh_latent_absorb(const void* q, const void* w_uk, const void* freq, const void* positions, void* qa, int64_t T, int64_t H, int64_t dn,
-                      int64_t rot_dim, int64_t rot_dims, int64_t kv_rank, float mag, int dt, void* stream) {
+int mbh_latent_absorb(const void* q, int64_t q_pitch, const void* w_uk, const void* freq, const void* positions, void* qa, int64_t T, int64_t H, int64_t dn,
+                      int64_t rot_dim, int64_t rot_dims, int halves, int64_t kv_rank, float mag, int dt, void* stream) {
     if (T == 0) return 0;
+    if (q_pitch < H * (dn + rot_dim)) return bad("mbh_latent_absorb: rows of q overlap");
     if (rot_dims > rot_dim || (rot_dims & 1)) return bad("mbh_latent_absorb: rot_dims must be even and at most rot_dim");
-    LatentAbsorbArgs a{q, w_uk, (const double*)freq, (const int*)positions, qa, (int)H, (int)dn, (int)rot_dim, (int)rot_dims, (int)kv_rank, mag};
+    LatentAbsorbArgs a{q, w_uk, (const double*)freq, (const int*)positions, qa, (int)H, (int)dn, (int)rot_dim, (int)rot_dims, (int)kv_rank, mag, (int)q_pitch, halves};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, latent_absorb_kernel<ST><<<dim3((unsigned)(T * H), (unsigned)(w_uk ? (kv_rank + 127) / 128 : 1)), 128, sizeof(float) * (size_t)dn, st>>>(a));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_latent_absorb") : 0;
 }
 
-int mbh_latent_expand(const void* kn, const void* v, const void* ring, const void* positions, const void* cache_rows, const void* q_start, void* kfull,
-                      void* vfull, int64_t T, int64_t B, int64_t Wt, int64_t H, int64_t dn, int64_t rot_dim, int64_t dv, int64_t kv_rank, int dt,
-                      void* stream) {
-    if (T == 0) return 0;
-    LatentExpandArgs a{kn, v, ring, (const int*)positions, (const int*)cache_rows, (const int*)q_start, kfull, vfull,
-                       (int)B, (int)Wt, (int)H, (int)dn, (int)rot_dim, (int)dv, (int)kv_rank};
+int mbh_latent_expand(const void* kn, const void* rows, void* kfull, int64_t R, int64_t H, int64_t dn, int64_t rot_dim, int64_t kv_rank, int dt, void* stream) {
+    if (R == 0) return 0;
+    LatentExpandArgs a{kn, rows, kfull, (int)H, (int)dn, (int)rot_dim, (int)kv_rank};
     cudaStream_t st = (cudaStream_t)stream;
-    DISPATCH(dt, latent_expand_kernel<ST><<<(unsigned)T, 128, 0, st>>>(a));
+    DISPATCH(dt, latent_expand_kernel<ST><<<(unsigned)R, 256, 0, st>>>(a));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_latent_expand") : 0;
 }
@@ -332,14 +386,16 @@ int mbh_head_gate(void* out, const void* gate, int64_t g_pitch, int64_t g_off, i
 }
 
 int mbh_attn_latent(const void* qa, const void* ring, const void* positions, const void* q_start, const void* slots, void* o_lat, int64_t T,
-                    int64_t B, int64_t W, int64_t H, int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int dt,
-                    void* stream) {
+                    int64_t B, int64_t W, int64_t H, int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int64_t window,
+                    const void* own, const void* seqpos, const void* sink, int dt, void* stream) {
     if (T == 0) return 0;
+    if (window < 0 || (own && !seqpos)) return bad("mbh_attn_latent: window >= 0; own rows come with seqpos");
     if (kv_rank > 32 * AT_MAXR_WIDE) return bad("mbh_attn_latent: latent size above 512");
     if (splits > AT_MAX_SPLITS) return bad("mbh_attn_latent: at most 64 splits");
     const int d = (int)(kv_rank + rot_dim);
     AttnArgs a{qa, ring, ring, nullptr, 0, (const int*)positions, (const int*)q_start, (const int*)slots, o_lat,
-               (int)T, (int)B, (int)W, (int)H, 1, d, (int)kv_rank, scale, (int)(splits > 1 && scratch ? splits : 1), (float*)scratch, d, d};
+               (int)T, (int)B, (int)W, (int)H, 1, d, (int)kv_rank, scale, (int)(splits > 1 && scratch ? splits : 1), (float*)scratch, d, d,
+               (int)window, own, own, (const int*)seqpos, 0, 0.f, (const float*)sink, d, d, 0};
     const bool wide = kv_rank > 32 * AT_MAXR;
     const size_t smem = sizeof(float) * ((size_t)d + AT_WARPS * AT_CHUNK + AT_WARPS * (2 + 32 * (wide ? AT_MAXR_WIDE : AT_MAXR)));
     cudaStream_t st = (cudaStream_t)stream;
@@ -350,14 +406,16 @@ int mbh_attn_latent(const void* qa, const void* ring, const void* positions, con
 }
 
 int mbh_attn_latent_decode(const void* qa, const void* ring, const void* positions, const void* slots, void* o_lat, int64_t B, int64_t W, int64_t H,
-                           int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int dt, void* stream) {
+                           int64_t kv_rank, int64_t rot_dim, float scale, int64_t splits, void* scratch, int64_t window, const void* sink, int dt,
+                           void* stream) {
     if (B == 0) return 0;
+    if (window < 0) return bad("mbh_attn_latent_decode: window >= 0");
     if (H > 4 * LD_WARPS || kv_rank > 32 * LD_CPL) return bad("mbh_attn_latent_decode: at most 32 heads and a latent of 512");
     if (splits < 1 || splits > AT_MAX_SPLITS || !scratch) return bad("mbh_attn_latent_decode: needs 1 <= splits <= 64 and scratch");
     LatentDecodeArgs a{qa, ring, (const int*)positions, (const int*)slots, (float*)scratch, (int)B, (int)W, (int)H, (int)kv_rank, (int)rot_dim, scale,
-                       (int)splits};
+                       (int)splits, (int)window};
     cudaError_t e = cudaSuccess;
-    DISPATCH(dt, e = launch_latent_decode<ST>(a, o_lat, (cudaStream_t)stream));
+    DISPATCH(dt, e = launch_latent_decode<ST>(a, o_lat, (const float*)sink, (cudaStream_t)stream));
     return e ? fail(e, "mbh_attn_latent_decode") : 0;
 }
 
@@ -374,14 +432,14 @@ int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_
 }
 
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int dt, void* stream) {
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, int dt, void* stream) {
     if (T == 0) return 0;
     if (groups < 1 || n % groups || keep < 1 || keep > groups) return bad("mbh_moe_route: groups must divide the routed outputs, 1 <= keep <= groups");
     if (top < 1 || top > n / groups * keep) return bad("mbh_moe_route: top exceeds the eligible outputs");
     const size_t smem = sizeof(float) * (size_t)(2 * n + 2 * groups);
     if (smem > 48 * 1024) return bad("mbh_moe_route: too many routed outputs");
     if (score != 0 && score != 1) return bad("mbh_moe_route: score is 0 (softmax) or 1 (sigmoid)");
-    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, scale};
+    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, scale, group_two, renorm};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, moe_route_kernel<ST><<<(unsigned)T, MOE_ROUTE_THREADS, smem, st>>>(a));
     cudaError_t e = cudaGetLastError();
@@ -439,14 +497,14 @@ int mbh_embed_pos(const void* tokens, const void* positions, const void* table, 
 }
 
 int mbh_rot_prep(const void* qkv, const void* freq, const void* positions, const void* cache_rows, void* q_out, void* k_out, void* v_out, void* ring_k,
-                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int unit_norm, float eps, int dt, void* stream) {
+                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int halves, float mag, int unit_norm, float eps, int dt, void* stream) {
     if (T == 0) return 0;
     if (d > 64 * RP_MAXP) return bad("mbh_rot_prep: head size above 256");
     if (rot_dims > d || (rot_dims & 1)) return bad("mbh_rot_prep: rot_dims must be even and at most the head size");
     if (!k_out != !v_out) return bad("mbh_rot_prep: k_out and v_out come together");
     if (cache_rows && (!ring_k || !ring_v)) return bad("mbh_rot_prep: ring rows without a ring");
     RotPrepArgs a{qkv, (const double*)freq, (const int*)positions, (const int*)cache_rows, q_out, k_out, v_out, ring_k, ring_v,
-                  (int)H, (int)G, (int)d, (int)e, (int)rot_dims, unit_norm, eps};
+                  (int)H, (int)G, (int)d, (int)e, (int)rot_dims, unit_norm, eps, halves, mag};
     cudaStream_t st = (cudaStream_t)stream;
     // few tokens (decode): the heads of a token are spread over CTAs; prompts: one CTA per token
     const unsigned hb = T < 512 ? (unsigned)((H + G + 3) / 4) : 1u;
@@ -623,6 +681,51 @@ int mbh_relu2_epilogue(const void* y, void* out, int64_t M, int64_t N, const voi
     DISPATCH(dt, run_epilogue<ST>(a, y, st));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_relu2_epilogue") : 0;
+}
+
+int mbh_delta_prep(const void* y, int64_t y_pitch, const void* conv, int64_t taps, void* cstate, const void* positions, const void* q_start, const void* seqpos,
+                   const void* slots, void* qk, void* kq, void* v, void* beta, int64_t T, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, int dt,
+                   void* stream) {
+    if (T == 0 || B == 0) return 0;
+    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_prep: key size 1 .. 1024, heads a multiple of key heads");
+    if (taps < 1) return bad("mbh_delta_prep: at least one tap");
+    DeltaArgs a{};
+    a.y = y; a.y_pitch = (int)y_pitch; a.conv = conv; a.taps = (int)taps; a.cstate = (float*)cstate;
+    a.positions = (const int*)positions; a.q_start = (const int*)q_start; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots;
+    a.T = (int)T; a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e;
+    a.qk = (float*)qk; a.kq = (float*)kq; a.v = (float*)v; a.beta = (float*)beta;
+    cudaError_t err = cudaSuccess;
+    DISPATCH(dt, err = launch_delta_prep<ST>(a, (cudaStream_t)stream));
+    return err ? fail(err, "mbh_delta_prep") : 0;
+}
+
+int mbh_delta_scan(const void* qk, const void* kq, const void* v, const void* beta, const void* g, void* state, const void* q_start, const void* seqpos,
+                   const void* slots, void* o32, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, void* stream) {
+    if (B == 0) return 0;
+    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_scan: key size 1 .. 1024, heads a multiple of key heads");
+    DeltaArgs a{};
+    a.q_start = (const int*)q_start; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots; a.state = (float*)state;
+    a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e;
+    a.qk = (float*)const_cast<void*>(qk); a.kq = (float*)const_cast<void*>(kq); a.v = (float*)const_cast<void*>(v); a.beta = (float*)const_cast<void*>(beta);
+    a.g = (const float*)g; a.o = (float*)o32;
+    cudaError_t err = launch_delta_scan(a, (cudaStream_t)stream);
+    return err ? fail(err, "mbh_delta_scan") : 0;
+}
+
+int mbh_delta_step(const void* y, int64_t y_pitch, int64_t ra, int64_t rg, const void* conv, int64_t taps, void* cstate, void* state, const void* w_a2,
+                   const void* dt_bias, const void* a_log, const void* w_g2, const void* norm, const void* positions, const void* seqpos, const void* slots,
+                   void* out, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, float eps, int dt, void* stream) {
+    if (B == 0) return 0;
+    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_step: key size 1 .. 1024, heads a multiple of key heads");
+    if (taps < 1) return bad("mbh_delta_step: at least one tap");
+    DeltaArgs a{};
+    a.y = y; a.y_pitch = (int)y_pitch; a.ra = (int)ra; a.rg = (int)rg; a.conv = conv; a.taps = (int)taps; a.cstate = (float*)cstate; a.state = (float*)state;
+    a.w_a2 = w_a2; a.dt_bias = dt_bias; a.a_log = a_log; a.w_g2 = w_g2; a.norm = norm;
+    a.positions = (const int*)positions; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots;
+    a.T = (int)B; a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e; a.eps = eps; a.out = out;
+    cudaError_t err = cudaSuccess;
+    DISPATCH(dt, err = launch_delta_step<ST>(a, (cudaStream_t)stream));
+    return err ? fail(err, "mbh_delta_step") : 0;
 }
 
 }  // extern "C"

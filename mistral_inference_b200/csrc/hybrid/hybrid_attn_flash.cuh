@@ -4,6 +4,7 @@
 // ring; S = Q K^T with mma.sync.m16n8k16 (Q fragments stay in registers); score = S * scale + bias[min(distance, n_tab - 1), h],
 // causal mask, running (max, sum) per query row in fp32; P is rounded to bf16 and multiplies V on the tensor cores with fp32
 // accumulators.  Query tiles never straddle two sequences; positions inside a tile are consecutive.
+// AttnArgs::softcap and AttnArgs::sink as in attn_bias_kernel (the cap's tanh through one fast exponential).
 // With AttnArgs::sigmoid the weights are sigmoid(score) (fp32, then bf16 for P V) and nothing is normalised.
 #pragma once
 #include "hybrid_mixers.cuh"
@@ -76,6 +77,7 @@ __global__ void __launch_bounds__(128) attn_bias_flash_kernel(AttnArgs a) {
     const int w0 = a.window > 0 ? a.window : 0x40000000;  // row at position p sees keys j with p - j < w0
     const float* bias = a.bias_tab ? a.bias_tab + h : nullptr;  // null: no bias
     const int last_tab = a.n_tab - 1;
+    const float scale = a.softcap > 0.f ? 1.f : a.scale;  // a capped score has its scale inside the cap
 
     for (int j0 = (j_lo / FA_BK) * FA_BK; j0 <= pos_last; j0 += FA_BK) {
         __syncthreads();
@@ -107,13 +109,20 @@ __global__ void __launch_bounds__(128) attn_bias_flash_kernel(AttnArgs a) {
                 mma_bf16(s[nt], qf[ks], *reinterpret_cast<const uint32_t*>(p), *reinterpret_cast<const uint32_t*>(p + 8));
             }
         float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (a.softcap > 0.f) {
+            const float f = 2.f * a.scale / a.softcap;
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s[nt][c] = softcap_fast(s[nt][c], a.softcap, f);
+        }
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
             for (int c = 0; c < 2; ++c) {
                 const int j = j0 + nt * 8 + tig * 2 + c;
-                const float x0 = (j <= p0 && p0 - j < w0) ? s[nt][c] * a.scale + (bias ? bias[(size_t)min(p0 - j, last_tab) * a.H] : 0.f) : -INFINITY;
-                const float x1 = (j <= p1 && p1 - j < w0) ? s[nt][2 + c] * a.scale + (bias ? bias[(size_t)min(p1 - j, last_tab) * a.H] : 0.f) : -INFINITY;
+                const float x0 = (j <= p0 && p0 - j < w0) ? s[nt][c] * scale + (bias ? bias[(size_t)min(p0 - j, last_tab) * a.H] : 0.f) : -INFINITY;
+                const float x1 = (j <= p1 && p1 - j < w0) ? s[nt][2 + c] * scale + (bias ? bias[(size_t)min(p1 - j, last_tab) * a.H] : 0.f) : -INFINITY;
                 s[nt][c] = x0; s[nt][2 + c] = x1;
                 mx0 = fmaxf(mx0, x0); mx1 = fmaxf(mx1, x1);
             }
@@ -152,6 +161,7 @@ __global__ void __launch_bounds__(128) attn_bias_flash_kernel(AttnArgs a) {
     }
     l0 = quad_sum(l0); l1 = quad_sum(l1);
     if (a.sigmoid) l0 = l1 = 1.f;
+    if (a.sink) { l0 = sink_denominator(m0, l0, a.sink[h]); l1 = sink_denominator(m1, l1, a.sink[h]); }
     bf16* out = static_cast<bf16*>(a.out);
 #pragma unroll
     for (int ne = 0; ne < E / 8; ++ne) {
@@ -165,7 +175,7 @@ __global__ void __launch_bounds__(128) attn_bias_flash_kernel(AttnArgs a) {
 inline bool launch_attn_flash(const AttnArgs& a, int n_tiles, cudaStream_t st) {
     dim3 grid(n_tiles, a.H);
 #define MBH_FA(DD, EE) if (a.d == DD && a.e == EE) { attn_bias_flash_kernel<DD, EE><<<grid, 128, 0, st>>>(a); return true; }
-    MBH_FA(32, 32) MBH_FA(64, 32) MBH_FA(64, 64) MBH_FA(128, 64) MBH_FA(64, 128) MBH_FA(128, 128) MBH_FA(96, 64) MBH_FA(192, 128)
+    MBH_FA(32, 32) MBH_FA(64, 32) MBH_FA(64, 64) MBH_FA(128, 64) MBH_FA(64, 128) MBH_FA(128, 128) MBH_FA(96, 64) MBH_FA(96, 96) MBH_FA(48, 32) MBH_FA(192, 128)
 #undef MBH_FA
     return false;
 }

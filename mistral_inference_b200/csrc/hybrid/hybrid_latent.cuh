@@ -2,19 +2,20 @@
 // token, [c (kv_rank) | rotated key part (rot_dim)], shared by all heads.
 //
 //   latent_prep     from the packed input projection y = [W_dq h | W_dkv h | W_g h]: RMS norm of the query latent -> cq;
-//                   RMS norm of the key/value latent c and the rotated shared key part -> the token's ring row
+//                   RMS norm of the key/value latent c and the rotated shared key part -> the token's ring row and / or its row of a
+//                   token-major copy (prompts over a ring shorter than the sequence attend to the copy beside the old ring)
 //   latent_absorb   per head: rotates the rotated part of q and folds the key up-projection into the query,
 //                   qa = [W_uk[h]^T q_plain | rot(q_rot)], so that q.k = qa . [c | k_rot] and attention runs over the latent rows
 //                   (attn_bias_kernel with one key/value head, key size kv_rank + rot_dim, value = the row's first kv_rank entries)
 //   latent_vup      per head: out = W_uv[h] o_latent, times the sigmoid of the head's output-gate logit
 //   attn_latent_decode  one token per sequence: a CTA takes a span of one sequence's latent rows for ALL heads, so a row is read
 //                   from memory once per step instead of once per head; partial (max, sum, acc) per head go to attn_merge_kernel
-//   latent_expand   whole prompts in bf16 take the other form: keys [W_uk c | rot(k_r)] and values W_uv c of the prompt's own tokens
-//                   are written out per head (two Linears, then this scatter into a temporary ring) and the tensor-core prompt
-//                   kernel runs ordinary multi-head attention on them; latent_absorb without W_uk only rotates q; head_gate
-//                   applies the output gate
+//   latent_expand   prompts in bf16 take the other form: keys [W_uk c | rot(k_r)] and values W_uv c of the prompt's own tokens (and of
+//                   the rows that earlier portions left in the ring) are written out per head (two Linears, then this kernel) and the
+//                   tensor-core prompt kernel runs ordinary multi-head attention on them; latent_absorb without W_uk only rotates q;
+//                   head_gate applies the output gate
 //
-// Rotation: interleaved pairs (2i, 2i+1) of the first rot_dims entries, angle = position * freq[i] evaluated in double
+// Rotation: interleaved pairs (2i, 2i+1), or pairs (i, i + rot_dims / 2) with `halves`, of the first rot_dims entries, angle = position * freq[i] evaluated in double
 // precision (the table of frequencies comes from the host, any frequency scaling already applied), cos and sin multiplied by `mag`.
 #pragma once
 #include "hybrid_common.cuh"
@@ -22,16 +23,18 @@
 namespace mbh {
 
 struct LatentPrepArgs {
-    const void* y;           // [T, q_rank + kv_rank + rot_dim + n_extra]
+    const void* y;           // [T, pitch]: query latent (q_rank) at 0 (q_rank 0: the design has none), kv latent and shared key part at kv_off
     const void* qnorm;       // [q_rank]
     const void* cnorm;       // [kv_rank]
     const double* freq;      // [rot_dims / 2]
     const int* positions;    // [T]
-    const int* cache_rows;   // [T] ring row or -1
+    const int* cache_rows;   // [T] ring row or -1; null: nothing goes to the ring in this call
     void* cq;                // [T, q_rank]
     void* ring;              // [rows, kv_rank + rot_dim]
     int q_rank, kv_rank, rot_dim, rot_dims, pitch;
     float eps, mag;
+    int kv_off, halves;
+    void* own;               // [T, kv_rank + rot_dim] the same rows token-major, or null
 };
 
 __device__ __forceinline__ void rot_pair(float u, float v, int pos, double f, float mag, float& ou, float& ov) {
@@ -42,6 +45,10 @@ __device__ __forceinline__ void rot_pair(float u, float v, int pos, double f, fl
     ov = v * c + u * s;
 }
 
+// places of the two entries of rotated pair i
+__device__ __forceinline__ int rot_first(int i, int halves) { return halves ? i : 2 * i; }
+__device__ __forceinline__ int rot_second(int i, int halves, int rot_dims) { return halves ? i + (rot_dims >> 1) : 2 * i + 1; }
+
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
     __shared__ float red[32];
@@ -49,40 +56,49 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentPrepArgs a) {
     const T* row = static_cast<const T*>(a.y) + (size_t)t * a.pitch;
     const int pos = a.positions[t], crow = a.cache_rows ? a.cache_rows[t] : -1;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) { const float v = to_f(row[i]); ss = fmaf(v, v, ss); }
-    ss = block_sum(ss, red);
-    const float inv_q = 1.f / sqrtf(ss / (float)a.q_rank + a.eps);
-    T* cq = static_cast<T*>(a.cq) + (size_t)t * a.q_rank;
-    const T* qn = static_cast<const T*>(a.qnorm);
-    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = from_f<T>(to_f(row[i]) * inv_q * to_f(qn[i]));
-    if (crow < 0) return;
-    const T* kv = row + a.q_rank;
+    if (a.q_rank > 0) {
+        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) { const float v = to_f(row[i]); ss = fmaf(v, v, ss); }
+        ss = block_sum(ss, red);
+        const float inv_q = 1.f / sqrtf(ss / (float)a.q_rank + a.eps);
+        T* cq = static_cast<T*>(a.cq) + (size_t)t * a.q_rank;
+        const T* qn = static_cast<const T*>(a.qnorm);
+        for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = from_f<T>(to_f(row[i]) * inv_q * to_f(qn[i]));
+    }
+    if (crow < 0 && !a.own) return;
+    const T* kv = row + a.kv_off;
     ss = 0.f;
     for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) { const float v = to_f(kv[i]); ss = fmaf(v, v, ss); }
     ss = block_sum(ss, red);
     const float inv_c = 1.f / sqrtf(ss / (float)a.kv_rank + a.eps);
-    T* dst = static_cast<T*>(a.ring) + (size_t)crow * (a.kv_rank + a.rot_dim);
+    const int width = a.kv_rank + a.rot_dim;
+    T* dst = crow >= 0 ? static_cast<T*>(a.ring) + (size_t)crow * width : nullptr;
+    T* own = a.own ? static_cast<T*>(a.own) + (size_t)t * width : nullptr;
+    auto put = [&](int i, T v) {
+        if (dst) dst[i] = v;
+        if (own) own[i] = v;
+    };
     const T* cn = static_cast<const T*>(a.cnorm);
-    for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) dst[i] = from_f<T>(to_f(kv[i]) * inv_c * to_f(cn[i]));
+    for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) put(i, from_f<T>(to_f(kv[i]) * inv_c * to_f(cn[i])));
     const T* kr = kv + a.kv_rank;
-    T* dr = dst + a.kv_rank;
     for (int i = threadIdx.x; i < a.rot_dims / 2; i += blockDim.x) {
+        const int i0 = rot_first(i, a.halves), i1 = rot_second(i, a.halves, a.rot_dims);
         float u, v;
-        rot_pair(to_f(kr[2 * i]), to_f(kr[2 * i + 1]), pos, a.freq[i], a.mag, u, v);
-        dr[2 * i] = from_f<T>(u);
-        dr[2 * i + 1] = from_f<T>(v);
+        rot_pair(to_f(kr[i0]), to_f(kr[i1]), pos, a.freq[i], a.mag, u, v);
+        put(a.kv_rank + i0, from_f<T>(u));
+        put(a.kv_rank + i1, from_f<T>(v));
     }
-    for (int i = a.rot_dims + threadIdx.x; i < a.rot_dim; i += blockDim.x) dr[i] = kr[i];
+    for (int i = a.rot_dims + threadIdx.x; i < a.rot_dim; i += blockDim.x) put(a.kv_rank + i, kr[i]);
 }
 
 struct LatentAbsorbArgs {
-    const void* q;           // [T, H, dn + rot_dim]
+    const void* q;           // [T, q_pitch]: [H, dn + rot_dim] at the start of every row
     const void* w_uk;        // [H * dn, kv_rank]
     const double* freq;
     const int* positions;
     void* qa;                // [T, H, kv_rank + rot_dim]
     int H, dn, rot_dim, rot_dims, kv_rank;
     float mag;
+    int q_pitch, halves;
 };
 
 // grid (token * head, blocks of 128 latent columns); thread r owns one latent column: W_uk[h] is read row by row, coalesced over r,
@@ -91,7 +107,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) latent_absorb_kernel(LatentAbsorbArgs a) {
     extern __shared__ float qs[];  // [dn]
     const int t = blockIdx.x / a.H, h = blockIdx.x % a.H;
-    const T* q = static_cast<const T*>(a.q) + ((size_t)t * a.H + h) * (a.dn + a.rot_dim);
+    const T* q = static_cast<const T*>(a.q) + (size_t)t * a.q_pitch + h * (a.dn + a.rot_dim);
     T* qa = static_cast<T*>(a.qa) + ((size_t)t * a.H + h) * (a.kv_rank + a.rot_dim);
     for (int i = threadIdx.x; i < a.dn; i += blockDim.x) qs[i] = to_f(q[i]);
     __syncthreads();
@@ -120,10 +136,11 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(LatentAbsorbArgs a) 
     const T* qr = q + a.dn;
     const int pos = a.positions[t];
     for (int i = threadIdx.x; i < a.rot_dims / 2; i += blockDim.x) {
+        const int i0 = rot_first(i, a.halves), i1 = rot_second(i, a.halves, a.rot_dims);
         float u, v;
-        rot_pair(to_f(qr[2 * i]), to_f(qr[2 * i + 1]), pos, a.freq[i], a.mag, u, v);
-        dr[2 * i] = from_f<T>(u);
-        dr[2 * i + 1] = from_f<T>(v);
+        rot_pair(to_f(qr[i0]), to_f(qr[i1]), pos, a.freq[i], a.mag, u, v);
+        dr[i0] = from_f<T>(u);
+        dr[i1] = from_f<T>(v);
     }
     for (int i = a.rot_dims + threadIdx.x; i < a.rot_dim; i += blockDim.x) dr[i] = qr[i];
 }
@@ -175,6 +192,7 @@ struct LatentDecodeArgs {
     int B, W, H, kv_rank, rot_dim;
     float scale;
     int splits;
+    int window;              // > 0: the token at position p sees rows p - window + 1 .. p only; 0: every row up to p
 };
 
 constexpr int LD_WARPS = 8, LD_KT = 32, LD_CPL = 16;  // kv_rank <= 32 * LD_CPL; heads <= LD_WARPS * HPW
@@ -191,10 +209,10 @@ __global__ void __launch_bounds__(LD_WARPS * 32) attn_latent_decode_kernel(Laten
     float* ps = qs + (size_t)a.H * d;                               // [H][LD_KT]
     T* ks = reinterpret_cast<T*>(ps + (size_t)a.H * LD_KT);         // [LD_KT][kp]
     const int b = blockIdx.x, split = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n = a.positions[b] + 1;
-    int span = (n + a.splits - 1) / a.splits;
+    const int n = a.positions[b] + 1, lo = a.window > 0 ? max(0, n - a.window) : 0;
+    int span = (n - lo + a.splits - 1) / a.splits;
     span = (span + LD_KT - 1) / LD_KT * LD_KT;
-    const int c0 = split * span, c1 = min(n, c0 + span);
+    const int c0 = lo + split * span, c1 = min(n, c0 + span);
     const T* q = static_cast<const T*>(a.qa) + (size_t)b * a.H * d;
     {
         constexpr int V = Vec<T>::N;
@@ -314,32 +332,33 @@ __global__ void __launch_bounds__(LD_WARPS * 32) attn_latent_decode_kernel(Laten
 }
 
 struct LatentExpandArgs {
-    const void* kn;          // [T, H * dn]   W_uk c
-    const void* v;           // [T, H * dv]   W_uv c
-    const void* ring;        // [rows, kv_rank + rot_dim]; the rotated key part of token t is in row cache_rows[t]
-    const int* positions; const int* cache_rows; const int* q_start;
-    void* kfull;             // [B * Wt, H, dn + rot_dim]: token at position p of sequence b in row b * Wt + p
-    void* vfull;             // [B * Wt, H, dv]
-    int B, Wt, H, dn, rot_dim, dv, kv_rank;
+    const void* kn;          // [R, H * dn]   W_uk c of R latent rows
+    const void* rows;        // [R, kv_rank + rot_dim] the latent rows; the rotated key part is their tail
+    void* kfull;             // [R, H, dn + rot_dim]
+    int H, dn, rot_dim, kv_rank;
 };
 
+// grid (rows); four entries at a time when the sizes allow it
 template <typename T>
-__global__ void __launch_bounds__(128) latent_expand_kernel(LatentExpandArgs a) {
-    const int t = blockIdx.x;
-    int b = 0;
-    while (b + 1 < a.B && a.q_start[b + 1] <= t) ++b;
-    const size_t row = (size_t)b * a.Wt + a.positions[t];
+__global__ void __launch_bounds__(256) latent_expand_kernel(LatentExpandArgs a) {
+    const size_t r = blockIdx.x;
     const int d = a.dn + a.rot_dim;
-    const T* kn = static_cast<const T*>(a.kn) + (size_t)t * a.H * a.dn;
-    const T* kr = static_cast<const T*>(a.ring) + (size_t)a.cache_rows[t] * (a.kv_rank + a.rot_dim) + a.kv_rank;
-    T* kf = static_cast<T*>(a.kfull) + row * a.H * d;
+    const T* kn = static_cast<const T*>(a.kn) + r * a.H * a.dn;
+    const T* kr = static_cast<const T*>(a.rows) + r * (a.kv_rank + a.rot_dim) + a.kv_rank;
+    T* kf = static_cast<T*>(a.kfull) + r * a.H * d;
+    if (a.dn % 4 == 0 && a.rot_dim % 4 == 0 && a.kv_rank % 4 == 0 &&
+        (reinterpret_cast<uintptr_t>(a.kn) | reinterpret_cast<uintptr_t>(a.rows) | reinterpret_cast<uintptr_t>(a.kfull)) % 16 == 0) {
+        struct alignas(4 * sizeof(T)) Quad { T v[4]; };
+        for (int i = threadIdx.x * 4; i < a.H * d; i += blockDim.x * 4) {
+            const int h = i / d, c = i % d;
+            *reinterpret_cast<Quad*>(kf + i) = *reinterpret_cast<const Quad*>(c < a.dn ? kn + h * a.dn + c : kr + c - a.dn);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < a.H * d; i += blockDim.x) {
         const int h = i / d, c = i % d;
         kf[i] = c < a.dn ? kn[h * a.dn + c] : kr[c - a.dn];
     }
-    const T* v = static_cast<const T*>(a.v) + (size_t)t * a.H * a.dv;
-    T* vf = static_cast<T*>(a.vfull) + row * a.H * a.dv;
-    for (int i = threadIdx.x; i < a.H * a.dv; i += blockDim.x) vf[i] = v[i];
 }
 
 // out[t, h, :] *= sigmoid(gate[t * g_pitch + g_off + h])

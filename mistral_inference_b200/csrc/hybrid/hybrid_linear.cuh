@@ -12,6 +12,8 @@
 //                 (rowscale fp32 [M, rs_pitch] or null: a mixture of experts run densely, every expert's hidden units scaled by
 //                 the token's routing weight, 0 for an expert that the token did not choose)
 //   EPI_RELU2     out[M, N]    = max(acc, 0)^2 * rowscale[m, n / rs_group]   (plain rows, no gate; rowscale as for EPI_SWIGLU)
+//   EPI_GEGLU     as EPI_SWIGLU with the tanh form of gelu in place of SiLU
+//   EPI_DECAY     out32[M, N]  = exp(-exp(a_log[n / rs_group]) * softplus(acc + b))   (decays of a gated recurrence; a_log [N / rs_group])
 //
 // In bf16 mode the Linear's own output is rounded to bf16 before the epilogue's arithmetic (the rounding point of a bf16
 // Linear); accumulation is fp32 in both modes.
@@ -25,7 +27,7 @@
 
 namespace mbh {
 
-enum { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GLU = 2, EPI_F32 = 3, EPI_SWIGLU = 4, EPI_RESIDUAL_SCALED = 5, EPI_RELU2 = 6 };
+enum { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GLU = 2, EPI_F32 = 3, EPI_SWIGLU = 4, EPI_RESIDUAL_SCALED = 5, EPI_RELU2 = 6, EPI_GEGLU = 7, EPI_DECAY = 8 };
 
 struct LinearArgs {
     const void* x; const void* w; const void* bias;
@@ -34,14 +36,19 @@ struct LinearArgs {
     int epi, n_act;
     float limit, alpha;
     const float* rowscale; int rs_pitch, rs_group;  // EPI_SWIGLU
+    const void* a_log;        // EPI_DECAY
+    int ldx;                  // elements between rows of x; 0: K (rows follow one another)
+    __host__ __device__ int x_pitch() const { return ldx ? ldx : K; }
 };
+
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
 
 template <typename T>
 __device__ __forceinline__ void epilogue_pair(const LinearArgs& a, int m, int n, float v0, float v1, bool has1) {
     // (m, n) and (m, n + 1); n is even
     const T* bias = static_cast<const T*>(a.bias);
     if (bias) { v0 += to_f(bias[n]); if (has1) v1 += to_f(bias[n + 1]); }
-    if (a.epi != EPI_F32) { v0 = rnd<T>(v0); v1 = rnd<T>(v1); }
+    if (a.epi != EPI_F32 && a.epi != EPI_DECAY) { v0 = rnd<T>(v0); v1 = rnd<T>(v1); }
     switch (a.epi) {
     case EPI_STORE: {
         T* o = static_cast<T*>(a.out) + (size_t)m * a.N + n;
@@ -65,10 +72,11 @@ __device__ __forceinline__ void epilogue_pair(const LinearArgs& a, int m, int n,
         float g = fminf(v0, a.limit), u = fminf(fmaxf(v1, -a.limit), a.limit);
         static_cast<T*>(a.out)[(size_t)m * (a.N >> 1) + (n >> 1)] = from_f<T>(g * sigmoid_exact(a.alpha * g) * (u + 1.f));
         break; }
-    case EPI_SWIGLU: {
+    case EPI_SWIGLU:
+    case EPI_GEGLU: {
         if (!has1) break;
         const int c = n >> 1;
-        float v = v0 * sigmoid_exact(v0) * v1;
+        float v = (a.epi == EPI_GEGLU ? gelu_tanh(v0) : v0 * sigmoid_exact(v0)) * v1;
         if (a.rowscale) v *= a.rowscale[(size_t)m * a.rs_pitch + c / a.rs_group];
         static_cast<T*>(a.out)[(size_t)m * (a.N >> 1) + c] = from_f<T>(v);
         break; }
@@ -82,6 +90,12 @@ __device__ __forceinline__ void epilogue_pair(const LinearArgs& a, int m, int n,
         }
         o[0] = from_f<T>(v0);
         if (has1) o[1] = from_f<T>(v1);
+        break; }
+    case EPI_DECAY: {
+        const T* al = static_cast<const T*>(a.a_log);
+        float* o = a.out32 + (size_t)m * a.N + n;
+        o[0] = expf(-expf(to_f(al[n / a.rs_group])) * softplus_exact(v0));
+        if (has1) o[1] = expf(-expf(to_f(al[(n + 1) / a.rs_group])) * softplus_exact(v1));
         break; }
     default: {
         float* o = a.out32 + (size_t)m * a.N + n;
@@ -110,7 +124,7 @@ __global__ void __launch_bounds__(LT_THREADS) linear_tiled_fma(LinearArgs a) {
         for (int i = 0; i < 4; ++i) {
             int k = k0 + lc + i;
             int m = m0 + lr, n = n0 + lr;
-            As[lc + i][lr] = (m < a.M && k < a.K) ? to_f(X[(size_t)m * a.K + k]) : 0.f;
+            As[lc + i][lr] = (m < a.M && k < a.K) ? to_f(X[(size_t)m * a.x_pitch() + k]) : 0.f;
             Ws[lc + i][lr] = (n < a.N && k < a.K) ? to_f(W[(size_t)n * a.K + k]) : 0.f;
         }
         __syncthreads();
@@ -151,7 +165,7 @@ __global__ void __launch_bounds__(MM_THREADS) linear_tiled_mma(LinearArgs a) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int wm = (warp >> 2) * 64, wn = (warp & 3) * 32;
     const int gid = lane >> 2, tig = lane & 3;
-    const bool vec_ok = (a.K % 8 == 0) && ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) % 16 == 0);
+    const bool vec_ok = (a.K % 8 == 0) && (a.x_pitch() % 8 == 0) && ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) % 16 == 0);
     float acc[4][4][4] = {};
 
     // loader: 128 rows x 32 k = 512 chunks of 8 bf16 per operand, 2 per thread
@@ -162,13 +176,13 @@ __global__ void __launch_bounds__(MM_THREADS) linear_tiled_mma(LinearArgs a) {
             int k = k0 + kc;
             uint4 va = make_uint4(0, 0, 0, 0), vw = make_uint4(0, 0, 0, 0);
             if (vec_ok) {
-                if (m0 + r < a.M && k < a.K) va = *reinterpret_cast<const uint4*>(X + (size_t)(m0 + r) * a.K + k);
+                if (m0 + r < a.M && k < a.K) va = *reinterpret_cast<const uint4*>(X + (size_t)(m0 + r) * a.x_pitch() + k);
                 if (n0 + r < a.N && k < a.K) vw = *reinterpret_cast<const uint4*>(W + (size_t)(n0 + r) * a.K + k);
             } else {
                 bf16* pa = reinterpret_cast<bf16*>(&va);
                 bf16* pw = reinterpret_cast<bf16*>(&vw);
                 for (int i = 0; i < 8; ++i) {
-                    if (m0 + r < a.M && k + i < a.K) pa[i] = X[(size_t)(m0 + r) * a.K + k + i];
+                    if (m0 + r < a.M && k + i < a.K) pa[i] = X[(size_t)(m0 + r) * a.x_pitch() + k + i];
                     if (n0 + r < a.N && k + i < a.K) pw[i] = W[(size_t)(n0 + r) * a.K + k + i];
                 }
             }
@@ -242,7 +256,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) linear_skinny(LinearArgs a) {
 #pragma unroll
         for (int m = 0; m < MM; ++m) acc[r][m] = 0.f;
     constexpr int V = Vec<T>::N;
-    const bool vec_ok = (a.K % V == 0) && ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) % 16 == 0);
+    const bool vec_ok = (a.K % V == 0) && (a.x_pitch() % V == 0) && ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) % 16 == 0);
     if (vec_ok) {
         for (int k = lane * V; k < a.K; k += 32 * V) {
             float wv[R][V], xv[V];
@@ -251,7 +265,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) linear_skinny(LinearArgs a) {
 #pragma unroll
             for (int m = 0; m < MM; ++m) {
                 if (m < a.M) {
-                    Vec<T>::load(X + (size_t)m * a.K + k, xv);
+                    Vec<T>::load(X + (size_t)m * a.x_pitch() + k, xv);
 #pragma unroll
                     for (int r = 0; r < R; ++r)
 #pragma unroll
@@ -267,7 +281,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) linear_skinny(LinearArgs a) {
 #pragma unroll
             for (int m = 0; m < MM; ++m)
                 if (m < a.M) {
-                    const float xv = to_f(X[(size_t)m * a.K + k]);
+                    const float xv = to_f(X[(size_t)m * a.x_pitch() + k]);
 #pragma unroll
                     for (int r = 0; r < R; ++r) acc[r][m] = fmaf(wv[r], xv, acc[r][m]);
                 }
@@ -298,7 +312,7 @@ __global__ void __launch_bounds__(SKM_WARPS * 32) linear_skinny_mma(LinearArgs a
     const bf16* wa = W + (size_t)min(n0 + gid, a.N - 1) * a.K;
     const bf16* wb = W + (size_t)min(n0 + gid + 8, a.N - 1) * a.K;
     const bool xrow = gid < a.M;
-    const bf16* xr = X + (size_t)(xrow ? gid : 0) * a.K;
+    const bf16* xr = X + (size_t)(xrow ? gid : 0) * a.x_pitch();
     float c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4  // four steps of loads in flight per warp: the kernel waits on global memory, not on the tensor pipe
     for (int kb = warp * 32; kb < a.K; kb += SKM_WARPS * 32) {
@@ -341,7 +355,7 @@ template <typename T>
 inline cudaError_t launch_linear(const LinearArgs& a, cudaStream_t st) {
     if (a.M <= 0 || a.N <= 0) return cudaSuccess;
     if constexpr (sizeof(T) == 2) {
-        if (a.M > 2 && a.M <= 8 && a.K % 8 == 0 && (reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w)) % 16 == 0) {
+        if (a.M > 2 && a.M <= 8 && a.K % 8 == 0 && a.x_pitch() % 8 == 0 && (reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w)) % 16 == 0) {
             linear_skinny_mma<<<(a.N + 15) / 16, SKM_WARPS * 32, 0, st>>>(a);
             return cudaGetLastError();
         }

@@ -1,14 +1,16 @@
 // Token mixers of the layered decoder and the elementwise steps around them.
 //
 //   embed_scale       x[t] = E[token[t]] * scale                       -> fp32 residual stream
-//   rmsnorm_f32       y = x / sqrt(mean(x^2) + eps) * w                 fp32 in, storage type out
+//   rmsnorm_f32       y = x / sqrt(mean(x^2) + eps) * (offset + w)      fp32 in, storage type out; one or two weights (two norms of the
+//                     same row for sublayers that run side by side)
 //   layernorm_f32     y = (x - mean) / sqrt(var + eps) * w + b          fp32 in; storage type out, or added to the residual stream
 //   attn_prep         per-head RMS norm of q and k (shared weight), query temperature by position, value mixing with an
 //                     earlier layer's values, scatter of k and v into the layer's cache ring
 //   whole_norm_prep   RMS norm of a token's whole query and whole key projection (weights of that size), k and v to the ring
 //   attn_bias         causal softmax attention over the ring with a per-(distance, head) additive bias, GQA, separate
 //                     key and value sizes; one kernel for prompts, prompt portions and decode; optionally a sliding window and
-//                     sigmoid weights instead of the softmax (every visible key weighs sigmoid(score), nothing is normalised)
+//                     sigmoid weights instead of the softmax (every visible key weighs sigmoid(score), nothing is normalised), soft-capped
+//                     scores, a learned sink per head in the softmax denominator
 //   lightning_scan    decayed linear attention S <- a S + k v^T, o = S^T q with the fp32 state carried in the cache
 //   gated_headnorm    y = rms(o over all heads) * w * sigmoid(g)
 #pragma once
@@ -49,16 +51,64 @@ __global__ void layernorm_f32_kernel(const float* __restrict__ x, const T* __res
     }
 }
 
+// One fp32 row per CTA.  w2 / y2 (both or neither): a second norm of the same row with its own weight.  offset: what the stored weight counts
+// from (0: the weight itself, 1: a weight stored around zero)
 template <typename T>
-__global__ void rmsnorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w, T* __restrict__ y, int D, float eps) {
+__global__ void rmsnorm_f32_kernel(const float* __restrict__ x, const T* __restrict__ w, const T* __restrict__ w2, T* __restrict__ y, T* __restrict__ y2, int D,
+                                   float eps, float offset) {
     __shared__ float red[32];
     const float* r = x + (size_t)blockIdx.x * D;
+    T* o = y + (size_t)blockIdx.x * D;
+    T* o2 = y2 ? y2 + (size_t)blockIdx.x * D : nullptr;
     float ss = 0.f;
+    const bool quads = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(w2) |
+                                       reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(y2)) % 16 == 0);
+    if (quads) {
+        // four neighbouring columns per thread and step, the first KEEP steps kept in registers for the second pass
+        constexpr int KEEP = 4;
+        float4 keep[KEEP];
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (k * blockDim.x + threadIdx.x) * 4;
+            keep[k] = i < D ? *reinterpret_cast<const float4*>(r + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            ss = fmaf(keep[k].x, keep[k].x, fmaf(keep[k].y, keep[k].y, fmaf(keep[k].z, keep[k].z, fmaf(keep[k].w, keep[k].w, ss))));
+        }
+        for (int i = (KEEP * blockDim.x + threadIdx.x) * 4; i < D; i += blockDim.x * 4) {
+            const float4 v = *reinterpret_cast<const float4*>(r + i);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+        ss = block_sum(ss, red);
+        const float inv = 1.f / sqrtf(ss / (float)D + eps);
+        auto emit = [&](int i, float4 v) {
+            const float u[4] = {v.x * inv, v.y * inv, v.z * inv, v.w * inv};
+            float wv[4], t[4];
+            load4(w + i, wv);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) t[k] = u[k] * (offset + wv[k]);
+            store4<T>(o + i, t);
+            if (o2) {
+                load4(w2 + i, wv);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) t[k] = u[k] * (offset + wv[k]);
+                store4<T>(o2 + i, t);
+            }
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (k * blockDim.x + threadIdx.x) * 4;
+            if (i < D) emit(i, keep[k]);
+        }
+        for (int i = (KEEP * blockDim.x + threadIdx.x) * 4; i < D; i += blockDim.x * 4) emit(i, *reinterpret_cast<const float4*>(r + i));
+        return;
+    }
     for (int i = threadIdx.x; i < D; i += blockDim.x) ss = fmaf(r[i], r[i], ss);
     ss = block_sum(ss, red);
     const float inv = 1.f / sqrtf(ss / (float)D + eps);
-    T* o = y + (size_t)blockIdx.x * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) o[i] = from_f<T>(r[i] * inv * to_f(w[i]));
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        const float v = r[i] * inv;
+        o[i] = from_f<T>(v * (offset + to_f(w[i])));
+        if (o2) o2[i] = from_f<T>(v * (offset + to_f(w2[i])));
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ attention: q/k/v preparation
@@ -178,6 +228,9 @@ struct AttnArgs {
     const int* seqpos;      // [B] tokens cached before this call (with own_k)
     int chunk;              // keys per warp and step, at most AT_CHUNK (0: AT_CHUNK).  A short ring read by few (token, head) pairs -- a decode
                             // step of a small batch over a sliding window -- is spread over more CTAs with a smaller chunk
+    float softcap;          // > 0: score <- softcap * tanh(score / softcap) (before a bias)
+    const float* sink;      // [H] or null: the softmax denominator of head h also holds exp(sink[h]), which has no key and no value
+    int own_k_pitch, own_v_pitch;  // elements per row of own_k / own_v; 0: G*d / G*e
     int sigmoid;            // 1: the weight of a visible key is sigmoid(score), not normalised over the keys (no softmax): partial results
                             // simply add, so the running maximum stays 0 and the sum is never divided by
 };
@@ -190,6 +243,10 @@ struct KeySource {
         return j >= own_from ? own + (size_t)(j - own_from) * own_pitch : ring + (size_t)(j % W) * ring_pitch;
     }
 };
+
+// sum of exp(. - M) over the keys and a sink, in units that suit numerators relative to M: L + exp(sink - M), kept in range
+// when the sink is far above every score (the weights then go to 0, as they must)
+__device__ __forceinline__ float sink_denominator(float M, float L, float sink) { return L + expf(sink - M); }
 
 constexpr int AT_WARPS = 4, AT_CHUNK = 128, AT_MAXR = 8, AT_MAXR_WIDE = 16;  // e <= 32 * MAXR
 
@@ -214,12 +271,13 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
     const size_t ks = a.k_pitch ? (size_t)a.k_pitch : (size_t)a.G * a.d, vs = a.v_pitch ? (size_t)a.v_pitch : (size_t)a.G * a.e;
     const int own_from = a.own_k ? a.seqpos[b] : 0x7fffffff;
     const size_t own_row = a.own_k ? (size_t)a.q_start[b] : 0;
+    const size_t oks = a.own_k_pitch ? (size_t)a.own_k_pitch : (size_t)a.G * a.d, ovs = a.own_v_pitch ? (size_t)a.own_v_pitch : (size_t)a.G * a.e;
     const KeySource<T> Ksrc{static_cast<const T*>(a.cache_k) + base * ks + (size_t)g * a.d,
-                            static_cast<const T*>(a.own_k) + own_row * a.G * a.d + (size_t)g * a.d, ks, (size_t)a.G * a.d, a.W, own_from};
+                            static_cast<const T*>(a.own_k) + own_row * oks + (size_t)g * a.d, ks, oks, a.W, own_from};
     const KeySource<T> Vsrc{static_cast<const T*>(a.cache_v) + base * vs + (size_t)g * a.e,
-                            static_cast<const T*>(a.own_v) + own_row * a.G * a.e + (size_t)g * a.e, vs, (size_t)a.G * a.e, a.W, own_from};
+                            static_cast<const T*>(a.own_v) + own_row * ovs + (size_t)g * a.e, vs, ovs, a.W, own_from};
     constexpr int V = Vec<T>::N;
-    const bool vec_ok = (a.d % V == 0) && (ks % V == 0) && (reinterpret_cast<uintptr_t>(a.cache_k) % 16 == 0)
+    const bool vec_ok = (a.d % V == 0) && (ks % V == 0) && (oks % V == 0) && (reinterpret_cast<uintptr_t>(a.cache_k) % 16 == 0)
                         && (!a.own_k || reinterpret_cast<uintptr_t>(a.own_k) % 16 == 0);
     const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;  // first visible key
     float m = a.sigmoid ? 0.f : -INFINITY, l = 0.f, acc[MAXR];
@@ -247,6 +305,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
             } else {
                 for (int i = 0; i < a.d; ++i) s = fmaf(qs[i], to_f(kr[i]), s);
             }
+            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
             if (a.bias_tab) s += a.bias_tab[(size_t)min(pos - j, a.n_tab - 1) * a.H + h];
             sc[jj] = s;
             cmax = fmaxf(cmax, s);
@@ -314,6 +373,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
                 if (r < cpl && lane * cpl + r < a.e) part[2 + lane * cpl + r] = o[r];
         } else {
             T* out = static_cast<T*>(a.out) + ((size_t)t * a.H + h) * a.e;
+            if (a.sink) L = sink_denominator(M, L, a.sink[h]);
 #pragma unroll
             for (int r = 0; r < MAXR; ++r)
                 if (r < cpl && lane * cpl + r < a.e) out[lane * cpl + r] = from_f<T>(a.sigmoid ? o[r] : o[r] / L);
@@ -326,7 +386,8 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
 // loads in flight).  grid (token * head, blocks of blockDim columns)
 constexpr int AT_MAX_SPLITS = 64;
 template <typename T>
-__global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restrict__ out, int splits, int e, int sigmoid = 0) {
+__global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restrict__ out, int splits, int e, int sigmoid = 0, const float* __restrict__ sink = nullptr,
+                                  int H = 1) {
     __shared__ float f[AT_MAX_SPLITS];
     __shared__ float red[32];
     const float* part = scratch + (size_t)blockIdx.x * splits * (2 + e);
@@ -339,8 +400,9 @@ __global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restri
         f[s] = w;
         lpart += w * part[(size_t)s * (2 + e) + 1];
     }
-    const float L = sigmoid ? 1.f : block_sum(lpart, red);  // its barriers also publish f[]
+    float L = sigmoid ? 1.f : block_sum(lpart, red);  // its barriers also publish f[]
     if (sigmoid) __syncthreads();
+    if (sink) L = sink_denominator(M, L, sink[blockIdx.x % H]);
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= e) return;
     const float* col = part + 2 + c;

@@ -2,8 +2,8 @@
 //
 //   moe_route         fp32 router: z = W_r h, s = softmax(z) over all n routed outputs (the last n_identity of them are identity
 //                     experts: output = input); choice = s + correction; the n outputs form `groups` equal groups of
-//                     neighbours, a group scores its largest choice, only the best `keep` groups stay eligible; the `top`
-//                     largest eligible choices are taken, each weighted by its s (not renormalised).  Ties go to the lower index.
+//                     neighbours, a group scores its largest choice (or the sum of its two largest), only the best `keep` groups stay eligible; the `top`
+//                     largest eligible choices are taken, each weighted by its s, optionally divided by the sum of the chosen ones' s.  Ties go to the lower index.
 //                     Writes the dense weights [T, n] (0 where not chosen) and the chosen (index, weight) pairs [T, top].
 //   moe_gateup_sparse / moe_down_sparse   few tokens (decode): one CTA column per (token, chosen expert) streams only that
 //                     expert's rows: act = silu(W_gate h) * (W_up h), then y = sum_k w_k W_down[e_k] act_k + (identity weights) h
@@ -27,6 +27,8 @@ struct MoeRouteArgs {
     int width, n, groups, keep, top;
     int score;                // 0: softmax over the outputs; 1: sigmoid of each output
     float scale;              // the weights (dense and wsel) are the chosen scores times this
+    int group_two;            // a group scores the sum of its two largest choices instead of its largest
+    int renorm;               // the weights are divided by (the sum of the chosen scores + 1e-20)
 };
 
 // (value, index) argmax over a warp; the lower index wins a tie
@@ -99,9 +101,12 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
     if (a.groups > 1 && a.keep < a.groups) {
         const int gs = a.n / a.groups;
         for (int g = lane; g < a.groups; g += 32) {
-            float b = -INFINITY;
-            for (int e = g * gs; e < (g + 1) * gs; ++e) b = fmaxf(b, ch[e]);
-            gb[g] = b;
+            float b = -INFINITY, b2 = -INFINITY;
+            for (int e = g * gs; e < (g + 1) * gs; ++e) {
+                b2 = fmaxf(b2, fminf(b, ch[e]));
+                b = fmaxf(b, ch[e]);
+            }
+            gb[g] = (a.group_two && gs > 1) ? b + b2 : b;
             kept[g] = 0.f;
         }
         __syncwarp();
@@ -118,19 +123,30 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
             if (kept[e / gs] == 0.f) ch[e] = -INFINITY;
         __syncwarp();
     }
+    float total = 0.f;  // of the chosen scores, the same in every lane
     for (int k = 0; k < a.top; ++k) {
         float v = -INFINITY; int ei = 0x7fffffff;
         for (int e = lane; e < a.n; e += 32)
             if (ch[e] > v) { v = ch[e]; ei = e; }
         warp_argmax(v, ei);
         if (ei == 0x7fffffff) ei = 0;  // fewer eligible outputs than `top` (a configuration error): weight 0 below
+        const float w = (v == -INFINITY) ? 0.f : z[ei];
+        total += w;
         if (lane == 0) {
-            const float w = (v == -INFINITY) ? 0.f : z[ei] * a.scale;
             a.idx[(size_t)t * a.top + k] = ei;
-            a.wsel[(size_t)t * a.top + k] = w;
-            if (v != -INFINITY) { a.dense[(size_t)t * a.n + ei] = w; ch[ei] = -INFINITY; }
+            a.wsel[(size_t)t * a.top + k] = w * a.scale;
+            if (v != -INFINITY) { a.dense[(size_t)t * a.n + ei] = w * a.scale; ch[ei] = -INFINITY; }
         }
         __syncwarp();
+    }
+    if (a.renorm) {  // every value was written by this warp; the barrier above ordered the writes
+        const float den = total + 1e-20f;
+        for (int k = lane; k < a.top; k += 32) {
+            const int ei = a.idx[(size_t)t * a.top + k];
+            const float w = z[ei] / den * a.scale;
+            a.wsel[(size_t)t * a.top + k] = w;
+            a.dense[(size_t)t * a.n + ei] = w;
+        }
     }
 }
 

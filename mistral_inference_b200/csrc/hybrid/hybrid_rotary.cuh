@@ -2,7 +2,7 @@
 //
 //   embed_pos        x[t] = E[token[t]] * scale + P[position[t]]            -> fp32 residual stream
 //   rot_prep         splits qkv[T, H*d + G*d + G*e]; rotates the first rot_dims entries of every q and k head as interleaved pairs
-//                    (2i, 2i + 1) by position * freq[i]; optionally divides each head by its root mean square (no weight);
+//                    (2i, 2i + 1), or as pairs (i, i + rot_dims / 2), by position * freq[i], cos and sin times `mag`; optionally divides each head by its root mean square (no weight);
 //                    writes q[T, H*d], k[T, G*d], v[T, G*e] token-major and, for tokens with a ring row, k and v into the ring
 //   kv_scatter       k[T, G*d], v[T, G*e] -> ring rows cache_rows[t] (after a prompt's attention has read the old ring)
 //
@@ -33,6 +33,8 @@ struct RotPrepArgs {
     int H, G, d, e, rot_dims;
     int unit_norm;          // divide every rotated q and k head by sqrt(mean(x^2) + eps)
     float eps;
+    int halves;             // pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)
+    float mag;              // factor on cos and sin
 };
 
 constexpr int RP_MAXP = 4;  // pairs per lane: head sizes up to 256
@@ -46,6 +48,10 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
     const int pos = a.positions[t];
     const int crow = a.cache_rows ? a.cache_rows[t] : -1;
     const int half = a.d >> 1;  // pairs; an odd last entry passes unchanged
+    const int rh = a.rot_dims >> 1;
+    // entries of pair pi: rotated ones by the layout, the rest two neighbours each
+    auto first = [&](int pi) { return a.halves && pi < rh ? pi : 2 * pi; };
+    auto second = [&](int pi) { return a.halves && pi < rh ? pi + rh : 2 * pi + 1; };
     for (int h = blockIdx.y * nw + warp; h < a.H + a.G; h += gridDim.y * nw) {
         const bool is_q = h < a.H;
         const T* src = row + (is_q ? h * a.d : Nq + (h - a.H) * a.d);
@@ -55,11 +61,11 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
             const int pi = lane + 32 * r;
             u[r] = v[r] = 0.f;
             if (pi < half) {
-                float x0 = to_f(src[2 * pi]), x1 = to_f(src[2 * pi + 1]);
-                if (2 * pi + 1 < a.rot_dims) {
+                float x0 = to_f(src[first(pi)]), x1 = to_f(src[second(pi)]);
+                if (pi < rh) {
                     double sn, cs;
                     sincos((double)pos * a.freq[pi], &sn, &cs);
-                    const float c = (float)cs, s = (float)sn;
+                    const float c = (float)cs * a.mag, s = (float)sn * a.mag;
                     const float y0 = x0 * c - x1 * s, y1 = x1 * c + x0 * s;
                     x0 = y0; x1 = y1;
                 }
@@ -79,8 +85,8 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
             const int pi = lane + 32 * r;
             if (pi < half) {
                 const T y0 = from_f<T>(u[r] * inv), y1 = from_f<T>(v[r] * inv);
-                if (dst0) { dst0[2 * pi] = y0; dst0[2 * pi + 1] = y1; }
-                if (dst1) { dst1[2 * pi] = y0; dst1[2 * pi + 1] = y1; }
+                if (dst0) { dst0[first(pi)] = y0; dst0[second(pi)] = y1; }
+                if (dst1) { dst1[first(pi)] = y0; dst1[second(pi)] = y1; }
             }
         }
         if ((a.d & 1) && lane == 0) {

@@ -55,15 +55,6 @@ __global__ void canon_conv_kernel(CanonArgs a) {
 // TAPS - 1 rows where a tile or a sequence starts).  Needs D % 4 == 0.  grid (ceil(T / CANON_TILE), ceil(D / (4 * blockDim)))
 constexpr int CANON_TILE = 16;
 
-template <typename T> __device__ __forceinline__ void store4(T* p, const float* v);
-template <> __device__ __forceinline__ void store4<float>(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-template <> __device__ __forceinline__ void store4<bf16>(bf16* p, const float* v) {
-    __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-    uint2 u;
-    u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(p) = u;
-}
-
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) canon_conv_tiled_kernel(CanonArgs a, int T_total) {
     constexpr int BACK = TAPS - 1;

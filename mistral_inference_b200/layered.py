@@ -1,7 +1,7 @@
 """Layered decoder: a model given as a list of layers, each with its own kind of token mixer (softmax attention with a
 distance bias, lightning attention with a recurrent state, latent attention, ...) and an optional feed-forward (gated, or a
 mixture of experts), optionally with a span of layers that runs several times (args.LayeredArgs; architectures "Fesenex",
-"Taruvik", "Lotazen", "Viladra").  It plugs into the same places as `Transformer`: `from_folder`, `forward(input_ids, seqlens, cache)` over ragged
+"Taruvik", "Lotazen", "Viladra", "Dimorax").  It plugs into the same places as `Transformer`: `from_folder`, `forward(input_ids, seqlens, cache)` over ragged
 batches, `BufferCache` (per-layer rings and states, `make_cache`), `forward_logprobs` / `next_token_logits` for `generate()`.
 
 On disk: config.json + model.safetensors with tensors `embed`, `l<i>.norm1|norm2` (and `norm1b|norm2b` with norms after the
@@ -45,6 +45,7 @@ class LayeredTransformer(nn.Module):
                 mixer = MIXERS[L.type](args.width, L.mixer, args.norm_eps)
             mlp = FEED_FORWARDS[type(L.mlp)](args.width, L.mlp) if L.mlp is not None else None
             blocks.append(LayeredBlock(args.width, args.norm_eps, mixer, mlp, norm=args.norm, post_norm=args.post_norm, parallel=args.parallel_block,
+                                       parallel_norms=args.parallel_norms, residual_mult=args.residual_mult,
                                        pre_norm=args.pre_norm, canon_taps=args.canon_taps if args.canon else 0,
                                        depth_results=li + 2 if args.depth_average else 0))
         self.layers = nn.ModuleList(blocks)
@@ -65,10 +66,14 @@ class LayeredTransformer(nn.Module):
 
     def make_cache(self, max_batch_size: int, max_seq_len: int) -> BufferCache:
         """The cache of this model, one entry per layer RUN (a layer that runs in several passes keeps each pass's keys apart): a
-        whole-sequence ring per attention layer, an fp32 state per lightning layer."""
+        whole-sequence ring per attention layer, an fp32 state per lightning layer.  A layer that reads another layer's keys and values
+        shares the ring of that layer's latest run before its own."""
         specs = [self.layers[i].mix.cache_spec() for i in self.runs]
+        for r, sp in enumerate(specs):
+            if sp.kind == "shared":  # the mixer names a layer; the cache wants its run
+                sp.source = max(q for q in range(r) if self.runs[q] == sp.source)
         for sp, i in zip(specs, self.runs):
-            sp.conv_shape = self.layers[i].conv_shape()
+            sp.conv_shape = self.layers[i].conv_shape() or sp.conv_shape
         cache = BufferCache(len(specs), max_batch_size, max_seq_len, 0, 0, None, layer_specs=specs)
         cache.to(device=self.device, dtype=self.dtype)
         cache.reset()

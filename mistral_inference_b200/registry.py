@@ -30,6 +30,7 @@ register("Fesenex", _layered)
 register("Taruvik", _layered)
 register("Lotazen", _layered)
 register("Viladra", _layered)
+register("Dimorax", _layered)
 register("transformer", _reference_format)
 
 

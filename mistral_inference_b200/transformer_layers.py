@@ -191,8 +191,9 @@ import math  # noqa: E402
 from typing import Dict  # noqa: E402
 
 from . import _abi_hybrid as _h  # noqa: E402
-from .args import (BiasedAttentionArgs, ClampedGluArgs, GlaArgs, Hgrn2Args, LatentAttentionArgs, LightningArgs, MlstmArgs, MoeFfArgs,  # noqa: E402
-                   Relu2FfArgs, Relu2MoeArgs, RetentionArgs, RotaryAttentionArgs, ScaledInputMoeArgs, SideBySideArgs, SigmoidAttentionArgs)
+from .args import (BiasedAttentionArgs, CappedAttentionArgs, ClampedGluArgs, DeltaArgs, GeluGluArgs, GlaArgs, GroupedMoeArgs, Hgrn2Args, LatentAttentionArgs, LightningArgs, MlstmArgs, MoeFfArgs,  # noqa: E402
+                   Relu2FfArgs, Relu2MoeArgs, RetentionArgs, RotaryAttentionArgs, ScaledInputMoeArgs, SideBySideArgs, SigmoidAttentionArgs,
+                   SinkLatentAttentionArgs)
 from .rope import scaled_frequencies  # noqa: E402
 from .cache import LayerCacheSpec  # noqa: E402
 
@@ -202,7 +203,7 @@ MOE_SPARSE_MAX_TOKENS = 16  # up to this many tokens a mixture of experts stream
 
 
 class Norm(nn.Module):
-    """The norm of a layered decoder: "rms" (weight), "rms_scalar" (ONE number as weight; kept as a vector of equal entries, so the
+    """The norm of a layered decoder: "rms" (weight), "rms_around_one" (the weight is stored as its distance from 1), "rms_scalar" (ONE number as weight; kept as a vector of equal entries, so the
     same kernel serves it) or "layer" (mean removed; weight and bias).  Reads the fp32 residual stream (or an fp32 sublayer output)
     and either returns the normed rows in the model dtype or adds them, in fp32, to `add_to`.  `mix` = (stack, n, coef, out), with an
     rms norm that adds: the depth average out = sum_j coef[j] * stack[j] over the n layer results so far follows in the same kernel
@@ -210,8 +211,8 @@ class Norm(nn.Module):
 
     def __init__(self, width: int, eps: float, kind: str):
         super().__init__()
-        assert kind in ("rms", "rms_scalar", "layer"), kind
-        self.kind, self.eps = kind, eps
+        assert kind in ("rms", "rms_around_one", "rms_scalar", "layer"), kind
+        self.kind, self.eps, self.offset = kind, eps, 1.0 if kind == "rms_around_one" else 0.0
         self.weight = nn.Parameter(torch.empty(width), requires_grad=False)
         self.bias = nn.Parameter(torch.empty(width), requires_grad=False) if kind == "layer" else None
 
@@ -220,9 +221,15 @@ class Norm(nn.Module):
             assert mix is None, "a depth average after a layer norm is not built"
             return _h.layernorm(x32, self.weight, self.bias, self.eps, add_to=add_to)
         if add_to is not None:
+            assert self.offset == 0.0, "a norm that adds to the stream with its weight stored around zero is not built"
             stack, n, coef, out = mix if mix is not None else (None, 0, None, None)
             return _h.rmsnorm_add(x32, self.weight, add_to, self.eps, stack, n, coef, out)
-        return _h.rmsnorm(x32, self.weight, self.eps)
+        return _h.rmsnorm(x32, self.weight, self.eps, self.offset)
+
+    def with_second(self, x32: torch.Tensor, other: "Norm") -> Tuple[torch.Tensor, torch.Tensor]:
+        """(self(x32), other(x32)) for two rms norms of the same rows, in one pass over them."""
+        assert self.kind == other.kind and self.kind != "layer" and self.eps == other.eps
+        return _h.rmsnorm_pair(x32, self.weight, other.weight, self.eps, self.offset)
 
     def load_weight(self, v: torch.Tensor) -> None:
         """Takes the checkpoint's weight: a vector, or the single number of an "rms_scalar" norm."""
@@ -245,6 +252,16 @@ def project_out(y: torch.Tensor, w: torch.Tensor, x32: torch.Tensor, post, scale
     else:
         assert scale == 1.0, "a scaled sublayer with a norm after it is not built"
         post(_h.linear(y, w, bias, epi=_h.EPI_F32), add_to=x32)
+
+
+def padded_rows(n: int) -> int:
+    """Rows of a packed input projection: a large one is padded to the prompt GEMM's tile (128 rows; nobody reads the extra outputs)."""
+    return (n + 127) // 128 * 128 if n >= 1024 else n
+
+
+def query_tiles(md) -> int:
+    """The number of 64-query tiles of this call for the tensor-core prompt kernel, 0 for the exact one."""
+    return sum((n + 63) // 64 for n in md.seqlens) if md.max_seqlen >= FLASH_MIN_QUERIES else 0
 
 
 def distance_buckets(rows: int, far: float) -> List[int]:
@@ -370,32 +387,41 @@ class ClampedGLU(nn.Module):
 
 class LatentAttention(nn.Module):
     """Causal softmax attention through latents (args.LatentAttentionArgs).  With h the normed input:
-        c_q = rms(W_dq h) * n_q,  q = W_uq c_q  (per head [dim plain | rot_dim rotated]);
+        c_q = rms(W_dq h) * n_q,  q = W_uq c_q   (q_rank 0: q = W_q h; per head [dim plain | rot_dim rotated]);
         [c' | k_r] = W_dkv h,  c = rms(c') * n_c;   k_h = [W_uk,h c | rot(k_r)],  v_h = W_uv,h c;
-        out = W_o concat_h( sigmoid(W_g h)_h * softmax(q_h . k_h * scale) v_h ).
-    The ring holds one row [c | rot(k_r)] per token.  Attention runs on the rows themselves: W_uk is folded into the query
-    (q_h . W_uk,h c = (W_uk,h^T q_h) . c) and W_uv is applied to the attention-weighted sum of latents, so a decode step reads
-    kv_rank + rot_dim numbers per cached token, whatever the number of heads.  Packed weights: w_in = dq ++ dkv ++ g rows."""
+        out = W_o concat_h( softmax(q_h . k_h * scale) v_h ), optionally each head times sigmoid(W_g h)_h, a sink in the softmax denominator,
+        and a sliding window.
+    The ring holds one row [c | rot(k_r)] per token (min(window, longest sequence) rows per sequence).  Attention runs on the rows themselves:
+    W_uk is folded into the query (q_h . W_uk,h c = (W_uk,h^T q_h) . c) and W_uv is applied to the attention-weighted sum of latents, so a decode
+    step reads kv_rank + rot_dim numbers per cached token, whatever the number of heads.  A prompt (portion) attends to the OLD ring and to its
+    own rows, and writes the ring afterwards; in bf16 its keys and values are written out per head for the tensor-core prompt kernel.
+    Packed weights: w_in = dq (or q) ++ dkv ++ g rows."""
 
     def __init__(self, width: int, a: LatentAttentionArgs, eps: float):
         super().__init__()
         self.a, self.eps = a, eps
-        self.n_in = a.q_rank + a.kv_rank + a.rot_dim + a.heads
+        self.nq = a.heads * (a.dim + a.rot_dim)
+        self.kv_off = a.q_rank or self.nq
+        self.g_off = self.kv_off + a.kv_rank + a.rot_dim
+        self.n_used = self.g_off + (a.heads if a.head_gate else 0)
+        self.n_in = padded_rows(self.n_used)
         self.w_in = nn.Parameter(torch.empty(self.n_in, width), requires_grad=False)
-        self.q_norm = nn.Parameter(torch.empty(a.q_rank), requires_grad=False)
         self.c_norm = nn.Parameter(torch.empty(a.kv_rank), requires_grad=False)
-        self.w_uq = nn.Parameter(torch.empty(a.heads * (a.dim + a.rot_dim), a.q_rank), requires_grad=False)
+        self.q_norm = nn.Parameter(torch.empty(a.q_rank), requires_grad=False) if a.q_rank else None
+        self.w_uq = nn.Parameter(torch.empty(self.nq, a.q_rank), requires_grad=False) if a.q_rank else None
         self.w_uk = nn.Parameter(torch.empty(a.heads * a.dim, a.kv_rank), requires_grad=False)
         self.w_uv = nn.Parameter(torch.empty(a.heads * a.vdim, a.kv_rank), requires_grad=False)
+        self.sink = nn.Parameter(torch.empty(a.heads), requires_grad=False) if a.sink else None
         self.wo = nn.Parameter(torch.empty(width, a.heads * a.vdim), requires_grad=False)
         self._freq: Optional[torch.Tensor] = None
+        self._sink32: Optional[torch.Tensor] = None
         self._mag = 1.0
         self.shared_decode = True   # decode steps read each latent row once for all heads (else: the per-head kernel)
-        self.expand_prompts = True  # whole bf16 prompts of suitable head sizes run multi-head attention on the tensor cores
+        self.expand_prompts = True  # bf16 prompts of suitable head sizes run multi-head attention on the tensor cores
 
     def cache_spec(self) -> LayerCacheSpec:
         # one shared "head" whose key row is the latent row; the values are its first kv_rank entries, so no value ring
-        return LayerCacheSpec(kind="ring", n_kv_heads=1, k_dim=self.a.kv_rank + self.a.rot_dim, v_dim=0, window=None)
+        return LayerCacheSpec(kind="ring", n_kv_heads=1, k_dim=self.a.kv_rank + self.a.rot_dim, v_dim=0, window=self.a.window)
 
     def frequencies(self) -> torch.Tensor:
         if self._freq is None or self._freq.device != self.wo.device:
@@ -403,49 +429,81 @@ class LatentAttention(nn.Module):
             self._freq = f.to(self.wo.device)
         return self._freq
 
-    def run(self, hn: torch.Tensor, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], post: Optional[Norm] = None) -> None:
+    def sinks(self) -> Optional[torch.Tensor]:
+        if self.sink is not None and (self._sink32 is None or self._sink32.device != self.sink.device):
+            self._sink32 = self.sink.detach().float().contiguous()
+        return self._sink32
+
+    def heads_of(self, rows: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+        """Keys [R, heads, dim + rot_dim] and values [R, heads * vdim] of latent rows [R, kv_rank + rot_dim]."""
+        a = self.a
+        lat = rows[:, : a.kv_rank].contiguous()
+        return _h.latent_expand(_h.linear(lat, self.w_uk), rows, a.heads, a.dim, a.rot_dim, a.kv_rank), _h.linear(lat, self.w_uv)
+
+    def old_rows(self, view: CacheView) -> Tuple[torch.Tensor, int]:
+        """(latent rows [sequences * n, kv_rank + rot_dim], n) that earlier portions left in the ring: key j of a sequence is row j % n of
+        its block."""
+        md = view.metadata
+        past = view.kv_seqlens_host[: len(md.seqlens)]
+        n = max(1, min(md.window, max(past)))
+        ring = view.cache_k.view(view.cache_k.shape[0], md.window, -1)
+        return ring.index_select(0, md.slots.long())[:, :n].reshape(-1, ring.shape[-1]), n
+
+    def run(self, hn: torch.Tensor, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], post: Optional[Norm] = None,
+            scale: float = 1.0) -> None:
         a, md = self.a, view.metadata
-        T = hn.shape[0]
-        freq = self.frequencies()
+        T, B, window = hn.shape[0], len(md.seqlens), a.window or 0
+        freq, sink = self.frequencies(), self.sinks()
         y = _h.linear(hn, self.w_in)
-        cq = _h.latent_prep(y, self.q_norm, self.c_norm, freq, md.positions, md.cache_rows, view.cache_k, a.q_rank, a.kv_rank, a.rot_dim,
-                            a.rot_dims, self.eps, self._mag)
-        q = _h.linear(cq, self.w_uq)
-        if (md.first_prefill and hn.dtype == torch.bfloat16 and md.max_seqlen >= FLASH_MIN_QUERIES and (a.dim + a.rot_dim, a.vdim) in _h.FLASH_SIZES
+        cq, own = _h.latent_prep(y, self.q_norm, self.c_norm, freq, md.positions, None if md.prefill else md.cache_rows, view.cache_k, a.q_rank, a.kv_rank,
+                                 a.rot_dim, a.rot_dims, self.eps, self._mag, kv_off=self.kv_off, halves=a.rot_halves, own=md.prefill)
+        q = _h.linear(cq, self.w_uq) if a.q_rank else y[:, : self.nq]
+        gate = y if a.head_gate else None
+        if (md.prefill and hn.dtype == torch.bfloat16 and md.max_seqlen >= FLASH_MIN_QUERIES and (a.dim + a.rot_dim, a.vdim) in _h.FLASH_SIZES
                 and self.expand_prompts):
-            # whole prompts: ordinary multi-head attention on the tensor cores over keys and values written out per head
-            B = len(md.seqlens)
-            # the latents of this call's tokens, gathered from their ring rows (every token of a whole prompt has one)
-            lat = view.cache_k.view(-1, a.kv_rank + a.rot_dim).index_select(0, md.cache_rows.long())[:, : a.kv_rank].contiguous()
-            kfull, vfull = _h.latent_expand(_h.linear(lat, self.w_uk), _h.linear(lat, self.w_uv), view.cache_k, md.positions, md.cache_rows, md.q_start,
-                                            B, md.max_seqlen, a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank)
-            qr = _h.latent_absorb(q, None, freq, md.positions, a.heads, a.dim, a.rot_dim, a.rot_dims, a.kv_rank, self._mag)
+            # ordinary multi-head attention on the tensor cores over keys and values written out per head
+            k, v = self.heads_of(own)
+            old_k, old_v, n_old = k, v, 1  # nothing before this call: no old key is ever addressed
+            if not md.first_prefill:
+                rows, n_old = self.old_rows(view)
+                old_k, old_v = self.heads_of(rows)
+            qr = _h.latent_absorb(q, None, freq, md.positions, a.heads, a.dim, a.rot_dim, a.rot_dims, a.kv_rank, self._mag, halves=a.rot_halves)
             out = torch.empty(T, a.heads * a.vdim, dtype=hn.dtype, device=hn.device)
-            _h.attn_bias(qr, kfull, vfull, None, md.positions, md.q_start, _h.iota(B, hn.device), out, B, md.max_seqlen, a.heads, a.heads,
-                         a.dim + a.rot_dim, a.vdim, a.scale, n_tiles=sum((n + 63) // 64 for n in md.seqlens))
-            _h.head_gate(out, y, self.n_in, a.q_rank + a.kv_rank + a.rot_dim, a.heads, a.vdim)
-            return project_out(out, self.wo, x32, post)
-        qa = _h.latent_absorb(q, self.w_uk, freq, md.positions, a.heads, a.dim, a.rot_dim, a.rot_dims, a.kv_rank, self._mag)
-        if not md.prefill and self.shared_decode and a.heads <= _h.LATENT_DECODE_MAX_HEADS and a.kv_rank <= _h.LATENT_DECODE_MAX_RANK:
-            # one token per sequence: every latent row is read once for all heads
-            o_lat = _h.attn_latent_decode(qa, view.cache_k, md.positions, md.slots, T, md.window, a.heads, a.kv_rank, a.rot_dim, a.scale)
+            _h.attn_window(qr, old_k, old_v, md.positions, md.q_start, _h.iota(B, hn.device), out, B, n_old, a.heads, a.heads, a.dim + a.rot_dim, a.vdim,
+                           a.scale, window, own_k=k, own_v=v, seqpos=md.seqpos, n_tiles=query_tiles(md), sink=sink)
+            if gate is not None:
+                _h.head_gate(out, gate, self.n_in, self.g_off, a.heads, a.vdim)
         else:
-            o_lat = _h.attn_latent(qa, view.cache_k, md.positions, md.q_start, md.slots, len(md.seqlens), md.window, a.heads, a.kv_rank, a.rot_dim,
-                                   a.scale, splits=_h.attn_splits(T, a.heads, md.window))
-        out = _h.latent_vup(o_lat, self.w_uv, y, self.n_in, a.q_rank + a.kv_rank + a.rot_dim, a.heads, a.vdim, a.kv_rank)
-        project_out(out, self.wo, x32, post)
+            qa = _h.latent_absorb(q, self.w_uk, freq, md.positions, a.heads, a.dim, a.rot_dim, a.rot_dims, a.kv_rank, self._mag, halves=a.rot_halves)
+            if not md.prefill and self.shared_decode and a.heads <= _h.LATENT_DECODE_MAX_HEADS and a.kv_rank <= _h.LATENT_DECODE_MAX_RANK:
+                # one token per sequence: every latent row is read once for all heads
+                o_lat = _h.attn_latent_decode(qa, view.cache_k, md.positions, md.slots, T, md.window, a.heads, a.kv_rank, a.rot_dim, a.scale, window, sink)
+            else:
+                o_lat = _h.attn_latent(qa, view.cache_k, md.positions, md.q_start, md.slots, B, md.window, a.heads, a.kv_rank, a.rot_dim, a.scale,
+                                       splits=_h.attn_splits(T, a.heads, md.window), window=window, own=own, seqpos=md.seqpos if own is not None else None,
+                                       sink=sink)
+            out = _h.latent_vup(o_lat, self.w_uv, gate, self.n_in, self.g_off, a.heads, a.vdim, a.kv_rank)
+        if own is not None:
+            _h.kv_scatter(own, own[:, :0], md.cache_rows, view.cache_k, view.cache_k)
+        project_out(out, self.wo, x32, post, scale)
 
     def checkpoint_names(self) -> List[str]:
-        return ["dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "g", "o"]
+        a = self.a
+        return ((["dq", "dq.norm", "uq"] if a.q_rank else ["q"]) + ["dkv", "dkv.norm", "uk", "uv"] + (["g"] if a.head_gate else [])
+                + (["sink"] if a.sink else []) + ["o"])
 
     def assign(self, name: str, put) -> bool:
         a = self.a
-        o1, o2 = a.q_rank, a.q_rank + a.kv_rank + a.rot_dim
-        targets = {"dq": lambda: self.w_in[:o1], "dkv": lambda: self.w_in[o1:o2], "g": lambda: self.w_in[o2:], "dq.norm": lambda: self.q_norm,
-                   "dkv.norm": lambda: self.c_norm, "uq": lambda: self.w_uq, "uk": lambda: self.w_uk, "uv": lambda: self.w_uv, "o": lambda: self.wo}
-        if name not in targets:
+        if name not in self.checkpoint_names():
             return False
-        put(targets[name]())
+        rows = {"dq": (0, self.kv_off), "q": (0, self.kv_off), "dkv": (self.kv_off, self.g_off), "g": (self.g_off, self.n_used)}
+        direct = {"dq.norm": "q_norm", "dkv.norm": "c_norm", "uq": "w_uq", "uk": "w_uk", "uv": "w_uv", "sink": "sink", "o": "wo"}
+        if name in rows:
+            self.w_in[self.n_used:].zero_()
+            put(self.w_in[rows[name][0]: rows[name][1]])
+        else:
+            put(getattr(self, direct[name]))
+            self._sink32 = None
         return True
 
 
@@ -506,63 +564,84 @@ class MoeFeedForward(nn.Module):
 
 
 class RotaryWindowAttention(nn.Module):
-    """Causal softmax attention with rotary positions, a unit RMS norm of the rotated q and k heads, grouped key/value heads and an
-    optional sliding window (args.RotaryAttentionArgs).  The ring holds min(window, longest sequence) rows per sequence.  A decode
-    step writes its key and value into the ring, then attends over it; a prompt (portion) attends over the OLD ring plus its own
-    keys and values, and writes the ring afterwards, so a prompt longer than the ring still finds every key inside each token's
-    window.  Packed weights: wqkv = q ++ k ++ v rows."""
+    """Causal softmax attention with rotary positions, grouped key/value heads and, as the arguments say (args.RotaryAttentionArgs), a unit RMS
+    norm of the rotated q and k heads, a sliding window, biases on q, k and v, soft-capped scores, a sink per head in the softmax denominator.
+    The ring holds min(window, longest sequence) rows per sequence.  A decode step writes its key and value into the ring, then attends over
+    it; a prompt (portion) attends over the OLD ring plus its own keys and values, and writes the ring afterwards, so a prompt longer than
+    the ring still finds every key inside each token's window.  With `kv_from` the layer has queries only and attends over the ring of an
+    earlier layer (whole sequence, no window), which that layer has just brought up to date.  Packed weights: wqkv = q ++ k ++ v rows."""
 
     def __init__(self, width: int, a: RotaryAttentionArgs, eps: float):
         super().__init__()
         self.a, self.eps = a, eps
-        self.nq, self.nk, self.nv = a.heads * a.dim, a.kv_heads * a.dim, a.kv_heads * a.vdim
-        self.wqkv = nn.Parameter(torch.empty(self.nq + self.nk + self.nv, width), requires_grad=False)
+        own_kv = a.kv_from is None
+        self.nq, self.nk, self.nv = a.heads * a.dim, a.kv_heads * a.dim * own_kv, a.kv_heads * a.vdim * own_kv
+        n = self.nq + self.nk + self.nv
+        self.wqkv = nn.Parameter(torch.empty(n, width), requires_grad=False)
+        self.bqkv = nn.Parameter(torch.empty(n), requires_grad=False) if a.qkv_bias else None
+        self.sink = nn.Parameter(torch.empty(a.heads), requires_grad=False) if a.sink else None
         self.wo = nn.Parameter(torch.empty(width, a.heads * a.vdim), requires_grad=False)
         self._freq: Optional[torch.Tensor] = None
+        self._sink32: Optional[torch.Tensor] = None
+        self._mag = 1.0
 
     def cache_spec(self) -> LayerCacheSpec:
+        if self.a.kv_from is not None:
+            return LayerCacheSpec(kind="shared", source=self.a.kv_from)
         return LayerCacheSpec(kind="ring", n_kv_heads=self.a.kv_heads, k_dim=self.a.dim, v_dim=self.a.vdim, window=self.a.window)
 
     def frequencies(self) -> torch.Tensor:
-        """float64 [rot_dims / 2]: rot_base^(-2i / rot_dims) / rot_factor, evaluated on the host in double precision."""
+        """float64 [rot_dims / 2]: rot_base^(-2i / rot_dims) under the frequency scaling, evaluated on the host in double precision."""
         if self._freq is None or self._freq.device != self.wo.device:
-            f, _ = scaled_frequencies(self.a.rot_dims, self.a.rot_base, None) if self.a.rot_dims else (torch.zeros(0, dtype=torch.float64), 1.0)
+            f, self._mag = (scaled_frequencies(self.a.rot_dims, self.a.rot_base, self.a.rot_scaling) if self.a.rot_dims
+                            else (torch.zeros(0, dtype=torch.float64), 1.0))
             self._freq = (f / self.a.rot_factor).to(self.wo.device)
         return self._freq
+
+    def sinks(self) -> Optional[torch.Tensor]:
+        if self.sink is not None and (self._sink32 is None or self._sink32.device != self.sink.device):
+            self._sink32 = self.sink.detach().float().contiguous()
+        return self._sink32
 
     def run(self, hn: torch.Tensor, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], post: Optional[Norm] = None,
             scale: float = 1.0) -> None:
         a, md = self.a, view.metadata
         T, B, W = hn.shape[0], len(md.seqlens), md.window
-        qkv = _h.linear(hn, self.wqkv)
+        qkv = _h.linear(hn, self.wqkv, self.bqkv)
         out = torch.empty(T, a.heads * a.vdim, dtype=hn.dtype, device=hn.device)
-        window = a.window or 0
+        window, own_kv, freq, sink = a.window or 0, a.kv_from is None, self.frequencies(), self.sinks()
+        own = md.prefill and own_kv
+        rows = None if (own or not own_kv) else md.cache_rows
+        q, k, v = _h.rot_prep(qkv, freq, md.positions, rows, view.cache_k if rows is not None else None, view.cache_v if rows is not None else None, a.heads,
+                              a.kv_heads if own_kv else 0, a.dim, a.vdim, a.rot_dims, a.unit_norm, self.eps, own=own, halves=a.rot_halves, mag=self._mag)
         if md.prefill:
-            q, k, v = _h.rot_prep(qkv, self.frequencies(), md.positions, None, None, None, a.heads, a.kv_heads, a.dim, a.vdim, a.rot_dims, a.unit_norm,
-                                  self.eps, own=True)
-            _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale,
-                           window, own_k=k, own_v=v, seqpos=md.seqpos,
-                           n_tiles=sum((n + 63) // 64 for n in md.seqlens) if md.max_seqlen >= FLASH_MIN_QUERIES else 0)
-            _h.kv_scatter(k, v, md.cache_rows, view.cache_k, view.cache_v)
+            plan = dict(n_tiles=query_tiles(md))
         else:
-            q, _, _ = _h.rot_prep(qkv, self.frequencies(), md.positions, md.cache_rows, view.cache_k, view.cache_v, a.heads, a.kv_heads, a.dim, a.vdim,
-                                  a.rot_dims, a.unit_norm, self.eps, own=False)
             splits, chunk = _h.window_decode_plan(T, a.heads, W)
-            _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale,
-                           window, splits=splits, chunk=chunk)
+            plan = dict(splits=splits, chunk=chunk)
+        _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, window,
+                       own_k=k, own_v=v, seqpos=md.seqpos if own else None, softcap=a.softcap, sink=sink, **plan)
+        if own:
+            _h.kv_scatter(k, v, md.cache_rows, view.cache_k, view.cache_v)
         project_out(out, self.wo, x32, post, scale)
 
     def checkpoint_names(self) -> List[str]:
-        return ["q", "k", "v", "o"]
+        proj = ["q", "k", "v"] if self.a.kv_from is None else ["q"]
+        return proj + ([n + ".b" for n in proj] if self.a.qkv_bias else []) + (["sink"] if self.a.sink else []) + ["o"]
 
     def assign(self, name: str, put) -> bool:
+        if name not in self.checkpoint_names():
+            return False
         spans = {"q": (0, self.nq), "k": (self.nq, self.nq + self.nk), "v": (self.nq + self.nk, self.nq + self.nk + self.nv)}
         if name in spans:
             put(self.wqkv[spans[name][0]: spans[name][1]])
-        elif name == "o":
-            put(self.wo)
+        elif name.endswith(".b"):
+            put(self.bqkv[spans[name[:-2]][0]: spans[name[:-2]][1]])
+        elif name == "sink":
+            put(self.sink)
+            self._sink32 = None
         else:
-            return False
+            put(self.wo)
         return True
 
 
@@ -1021,6 +1100,182 @@ class Relu2Moe(nn.Module):
         return True
 
 
+class DeltaMixer(nn.Module):
+    """Gated delta rule (args.DeltaArgs).  q, k (kv_heads x dim) and v (heads x vdim) are projections through a causal convolution over time per
+    channel and SiLU; q and k unit vectors per head, q times dim^(-1/2); per head, in fp32 with the state in the cache,
+        S <- diag(g) S;   S <- S + k (beta (v - S^T k))^T;   o = S^T q,
+    beta = sigmoid(W_b h), g = exp(-exp(A_log) softplus(W_a2 W_a1 h + dt_bias)) per head and key channel; every head divided by its root mean
+    square, times one weight [vdim] and sigmoid(W_g2 W_g1 h).  The ranks of the two low-rank projections come with the checkpoint.  Packed
+    weights: w_in = q ++ k ++ v ++ b ++ a1 ++ g1 rows (padded); conv = the taps of q, k and v.  A decode step is one kernel between the
+    input and the output projection."""
+
+    def __init__(self, width: int, a: DeltaArgs, eps: float):
+        super().__init__()
+        self.a, self.eps, self.width = a, eps, width
+        self.nqk, self.nv = a.kv_heads * a.dim, a.heads * a.vdim
+        self.channels = 2 * self.nqk + self.nv
+        self.ra = self.rg = 1                                            # resized by the loader to the checkpoint's ranks
+        self.w_in = nn.Parameter(torch.empty(padded_rows(self.channels + a.heads + 2), width), requires_grad=False)
+        self.conv = nn.Parameter(torch.empty(self.channels, a.conv), requires_grad=False)
+        self.wa2 = nn.Parameter(torch.empty(a.heads * a.dim, 1), requires_grad=False)
+        self.wg2 = nn.Parameter(torch.empty(self.nv, 1), requires_grad=False)
+        self.dt_bias = nn.Parameter(torch.empty(a.heads * a.dim), requires_grad=False)
+        self.a_log = nn.Parameter(torch.empty(a.heads), requires_grad=False)
+        self.norm = nn.Parameter(torch.empty(a.vdim), requires_grad=False)
+        self.wo = nn.Parameter(torch.empty(width, self.nv), requires_grad=False)
+
+    def cache_spec(self) -> LayerCacheSpec:
+        return LayerCacheSpec(kind="state", state_shape=(self.a.heads, self.a.vdim, self.a.dim), conv_shape=(self.a.conv, self.channels))
+
+    def run(self, hn: torch.Tensor, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], post=None, scale: float = 1.0) -> None:
+        a, md = self.a, view.metadata
+        B, o = len(md.seqlens), self.channels + a.heads
+        y = _h.linear(hn, self.w_in)
+        if md.prefill:
+            g = _h.linear_decay(y[:, o: o + self.ra], self.wa2, self.dt_bias, self.a_log, a.dim)
+            gate = _h.linear(y[:, o + self.ra: o + self.ra + self.rg], self.wg2)
+            qk, kq, v, beta = _h.delta_prep(y, self.conv, view.conv, md.positions, md.q_start, md.seqpos, md.slots, B, a.heads, a.kv_heads, a.dim, a.vdim)
+            o32 = _h.delta_scan(qk, kq, v, beta, g, view.state, md.q_start, md.seqpos, md.slots, B, a.heads, a.kv_heads, a.dim, a.vdim)
+            out = _h.scan_post(o32, None, self.norm, False, gate, self.nv, 0, a.heads, a.vdim, False, self.eps)
+        else:
+            out = _h.delta_step(y, self.ra, self.rg, self.conv, view.conv, view.state, self.wa2, self.dt_bias, self.a_log, self.wg2, self.norm, md.positions,
+                                md.seqpos, md.slots, a.heads, a.kv_heads, a.dim, a.vdim, self.eps)
+        project_out(out, self.wo, x32, post, scale)
+
+    def checkpoint_names(self) -> List[str]:
+        return ["q", "q.conv", "k", "k.conv", "v", "v.conv", "b", "A_log", "norm", "a1", "a2", "dt_bias", "g1", "g2", "o"]
+
+    def _spans(self) -> Dict[str, Tuple[int, int]]:
+        out, at = {}, 0
+        for name, n in (("q", self.nqk), ("k", self.nqk), ("v", self.nv), ("b", self.a.heads), ("a1", self.ra), ("g1", self.rg)):
+            out[name] = (at, at + n)
+            at += n
+        return out
+
+    def resize(self, ra: int, rg: int) -> None:
+        """Takes the ranks of the decay and gate projections; rows already loaded keep their values."""
+        old, was = self.w_in, self._spans()
+        self.ra, self.rg = ra, rg
+        spans = self._spans()
+        like = dict(dtype=old.dtype, device=old.device)
+        self.w_in = nn.Parameter(torch.zeros(padded_rows(spans["g1"][1]), self.width, **like), requires_grad=False)
+        with torch.no_grad():
+            for name, (lo, hi) in spans.items():
+                if hi - lo == was[name][1] - was[name][0]:
+                    self.w_in[lo:hi].copy_(old[was[name][0]: was[name][1]])
+        if self.wa2.shape[1] != ra:
+            self.wa2 = nn.Parameter(torch.empty(self.wa2.shape[0], ra, **like), requires_grad=False)
+        if self.wg2.shape[1] != rg:
+            self.wg2 = nn.Parameter(torch.empty(self.wg2.shape[0], rg, **like), requires_grad=False)
+
+    def prepare(self, name: str, shape: Tuple[int, ...]) -> None:
+        """Called by the loader before `assign`: the low-rank projections take the rank of the checkpoint's tensors."""
+        if len(shape) == 2 and name in ("a1", "g1", "a2", "g2"):
+            rank = shape[0] if name[1] == "1" else shape[1]
+            ra, rg = (rank, self.rg) if name[0] == "a" else (self.ra, rank)
+            if (ra, rg) != (self.ra, self.rg):
+                self.resize(ra, rg)
+
+    def assign(self, name: str, put) -> bool:
+        spans = self._spans()
+        taps = {"q.conv": "q", "k.conv": "k", "v.conv": "v"}
+        direct = {"A_log": "a_log", "norm": "norm", "a2": "wa2", "g2": "wg2", "dt_bias": "dt_bias", "o": "wo"}
+        if name in spans:
+            put(self.w_in[spans[name][0]: spans[name][1]])
+        elif name in taps:
+            lo, hi = spans[taps[name]]
+            put(self.conv[lo:hi])
+        elif name in direct:
+            put(getattr(self, direct[name]))
+        else:
+            return False
+        return True
+
+
+class GatedFeedForward(nn.Module):
+    """Feed-forward W_down (act(W_gate h) * (W_up h)), act SiLU or the tanh form of gelu, in the epilogue of one Linear over interleaved gate / up
+    rows.  `rowscale` (fp32 [T, 1]): one number per token on the hidden units."""
+
+    def __init__(self, width: int, ff: int, gelu: bool):
+        super().__init__()
+        self.ff, self.width, self.gelu = ff, width, gelu
+        self.w13 = nn.Parameter(torch.empty(2 * ff, width), requires_grad=False)
+        self.w2 = nn.Parameter(torch.empty(width, ff), requires_grad=False)
+
+    def run(self, hn: torch.Tensor, x32: torch.Tensor, post=None, scale: float = 1.0, rowscale: Optional[torch.Tensor] = None) -> None:
+        project_out(_h.linear_swiglu(hn, self.w13, rowscale=rowscale, group=self.ff if rowscale is not None else 0, gelu=self.gelu), self.w2, x32, post, scale)
+
+    def checkpoint_names(self) -> List[str]:
+        return ["gate", "up", "down"]
+
+    def assign(self, name: str, put) -> bool:
+        if name in ("gate", "up"):
+            put(self.w13.view(self.ff, 2, self.width)[:, int(name == "up")])
+        elif name == "down":
+            put(self.w2)
+        else:
+            return False
+        return True
+
+
+class GeluGlu(GatedFeedForward):
+    def __init__(self, width: int, a: GeluGluArgs):
+        super().__init__(width, a.ff, gelu=True)
+
+
+class GroupedMoe(nn.Module):
+    """Mixture of SiLU-gated experts with an fp32 sigmoid router limited to groups and renormalised weights (args.GroupedMoeArgs), plus a shared
+    expert times sigmoid(W_sg h).  Packed like MoeFeedForward.  Few tokens (decode) stream the chosen experts only; prompts run all experts as
+    two Linears, the first one's epilogue scaling every expert's hidden units by the token's weight (0 when not chosen).  Every part adds
+    into the residual stream; a factor on the result (`scale`) goes into the routing weights and the output Linears."""
+
+    def __init__(self, width: int, a: GroupedMoeArgs):
+        super().__init__()
+        self.a, self.width = a, width
+        self.router = nn.Parameter(torch.empty(a.experts, width), requires_grad=False)
+        self.correction = nn.Parameter(torch.empty(a.experts), requires_grad=False)
+        self.w13 = nn.Parameter(torch.empty(a.experts * 2 * a.ff, width), requires_grad=False)
+        self.w2 = nn.Parameter(torch.empty(width, a.experts * a.ff), requires_grad=False)
+        self.shared = GatedFeedForward(width, a.shared_ff, gelu=False) if a.shared_ff else None
+        self.shared_gate = nn.Parameter(torch.empty(1, width), requires_grad=False) if a.shared_ff else None
+        self.sparse_max_tokens = MOE_SPARSE_MAX_TOKENS
+
+    def run(self, hn: torch.Tensor, x32: torch.Tensor, post=None, scale: float = 1.0) -> None:
+        assert post is None, "a norm after this feed-forward is not built"
+        a = self.a
+        dense, idx, wsel = _h.moe_route(hn, self.router, self.correction, a.groups, a.keep, a.top, score=1, scale=a.router_scale * scale, group_two=True,
+                                        renorm=True)
+        if hn.shape[0] <= self.sparse_max_tokens:
+            _h.moe_sparse(hn, self.w13, self.w2, idx, wsel, a.experts, a.ff, add_to=x32)
+        else:
+            _h.linear(_h.linear_swiglu(hn, self.w13, rowscale=dense, group=a.ff), self.w2, epi=_h.EPI_RESIDUAL, residual=x32)
+        if self.shared is not None:
+            # a router over one output: its sigmoid is the shared expert's gate
+            gate, _, _ = _h.moe_route(hn, self.shared_gate, None, 1, 1, 1, score=1)
+            self.shared.run(hn, x32, None, scale, rowscale=gate)
+
+    def checkpoint_names(self) -> List[str]:
+        names = ["router", "correction"] + [f"e{e}.{n}" for e in range(self.a.experts) for n in ("gate", "up", "down")]
+        return names + (["shared.sg"] + ["shared." + n for n in self.shared.checkpoint_names()] if self.shared is not None else [])
+
+    def assign(self, name: str, put) -> bool:
+        a = self.a
+        head, _, part = name.partition(".")
+        if name in ("router", "correction"):
+            put(getattr(self, name))
+        elif head == "shared" and self.shared is not None:
+            if part == "sg":
+                put(self.shared_gate)
+                return True
+            return self.shared.assign(part, put)
+        elif head[:1] == "e" and head[1:].isdigit() and int(head[1:]) < a.experts and part in ("gate", "up", "down"):
+            e = int(head[1:])
+            put(self.w2.view(self.width, a.experts, a.ff)[:, e] if part == "down" else self.w13.view(a.experts, a.ff, 2, self.width)[e, :, int(part == "up")])
+        else:
+            return False
+        return True
+
+
 class CanonConv(nn.Module):
     """What a sublayer reads, replaced by itself plus a causal convolution over time on every channel: h_t = x_t + sum_j w[:, j]
     x_(t - taps + 1 + j), zeros before the sequence's start.  Reads the fp32 stream, writes the model dtype.  The last taps - 1 inputs
@@ -1040,8 +1295,10 @@ class CanonConv(nn.Module):
 MIXERS = {"attention": BiasedAttention, "lightning": LightningMixer, "latent_attention": LatentAttention, "parallel": SideBySideMixer,
           "mlstm": MlstmMixer, "mlstm_2": MlstmMixer}
 # mixers that a design names with a type another design uses differently are found by their argument class first
-MIXERS_BY_ARGS = {RetentionArgs: RetentionMixer, GlaArgs: GlaMixer, SigmoidAttentionArgs: SigmoidWindowAttention}
-FEED_FORWARDS = {ClampedGluArgs: ClampedGLU, MoeFfArgs: MoeFeedForward, ScaledInputMoeArgs: ScaledInputMoe, Relu2MoeArgs: Relu2Moe}
+MIXERS_BY_ARGS = {RetentionArgs: RetentionMixer, GlaArgs: GlaMixer, SigmoidAttentionArgs: SigmoidWindowAttention,
+                  CappedAttentionArgs: RotaryWindowAttention, SinkLatentAttentionArgs: LatentAttention, DeltaArgs: DeltaMixer}
+FEED_FORWARDS = {ClampedGluArgs: ClampedGLU, MoeFfArgs: MoeFeedForward, ScaledInputMoeArgs: ScaledInputMoe, Relu2MoeArgs: Relu2Moe,
+                 GeluGluArgs: GeluGlu, GroupedMoeArgs: GroupedMoe}
 
 
 class _PostNorm:
@@ -1058,7 +1315,8 @@ class _PostNorm:
 class LayeredBlock(nn.Module):
     """x <- x + mixer(norm1(x)); x <- x + ff(norm2(x)) when the layer has a feed-forward; with `post_norm` each sublayer's output
     goes through a norm of its own (norm1b, norm2b) before it is added.  `parallel`: one norm, h = norm1(x), and both sublayers read
-    it: x <- x + mixer(h) + ff(h).  Without `pre_norm` (and with `post_norm`) the sublayers read the stream itself and norm1 / norm2
+    it: x <- x + mixer(h) + ff(h); with `parallel_norms` 2 each has a norm of its own and a fixed factor goes on both results:
+    x <- x + residual_mult * (mixer(norm1(x)) + ff(norm2(x))).  Without `pre_norm` (and with `post_norm`) the sublayers read the stream itself and norm1 / norm2
     act on their outputs: x <- x + norm1(mixer(x)), x <- x + norm2(ff(x)).  `canon_taps` > 0: what a sublayer reads (normed or not) is
     first replaced by itself plus a causal convolution over time (canon1 for the mixer, canon2 for the feed-forward; their last inputs
     are the layer's convolution state in the cache).  `depth_results` = n > 0: the block holds n weights `dwa` and, given
@@ -1066,8 +1324,11 @@ class LayeredBlock(nn.Module):
     `x32` is updated in place."""
 
     def __init__(self, width: int, eps: float, mixer: nn.Module, mlp: Optional[nn.Module], norm: str = "rms", post_norm: bool = False,
-                 parallel: bool = False, pre_norm: bool = True, canon_taps: int = 0, depth_results: int = 0):
+                 parallel: bool = False, pre_norm: bool = True, canon_taps: int = 0, depth_results: int = 0,
+                 parallel_norms: int = 1, residual_mult: float = 1.0):
         super().__init__()
+        assert parallel_norms in (1, 2) and (parallel_norms == 1 or parallel) and (residual_mult == 1.0 or parallel_norms == 2)
+        self.two_norms, self.residual_mult = parallel_norms == 2, residual_mult
         assert not (parallel and post_norm), "a parallel block with norms after the sublayers is not built"
         assert pre_norm or (post_norm and not parallel and canon_taps > 0), "sublayers that read the stream itself: norms after them, through a convolution"
         self.eps, self.parallel, self.pre_norm, self.width = eps, parallel, pre_norm, width
@@ -1075,7 +1336,7 @@ class LayeredBlock(nn.Module):
         self.norm1b = Norm(width, eps, norm) if post_norm and pre_norm else None
         self.mix = mixer
         self.mlp = mlp
-        self.norm2 = Norm(width, eps, norm) if mlp is not None and not parallel else None
+        self.norm2 = Norm(width, eps, norm) if mlp is not None and (not parallel or self.two_norms) else None
         self.norm2b = Norm(width, eps, norm) if mlp is not None and post_norm and pre_norm else None
         assert canon_taps == 0 or not pre_norm, "a convolution after a norm is not built"
         self.canon1 = CanonConv(width, canon_taps, 0) if canon_taps > 0 else None
@@ -1098,6 +1359,12 @@ class LayeredBlock(nn.Module):
                 self.mlp.run(self.canon2(x32, view), x32, _PostNorm(self.norm2, m))
             return x32
         assert mix is None, "the depth average follows a norm that adds to the stream"
+        if self.two_norms:  # both sublayers read the stream as it was: their norms come first, then each adds its result
+            hn, hn2 = self.norm1.with_second(x32, self.norm2) if self.mlp is not None else (self.norm1(x32), None)
+            self.mix.run(hn, x32, view, ctx, None, self.residual_mult)
+            if self.mlp is not None:
+                self.mlp.run(hn2, x32, None, self.residual_mult)
+            return x32
         if self.parallel:  # the sublayers read hn only, so each may add its output to the stream as it finishes
             hn = self.norm1(x32)
             self.mix.run(hn, x32, view, ctx, None)
