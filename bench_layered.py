@@ -1,11 +1,12 @@
-"""`bench.py --design fesenex|taruvik|lotazen|viladra`: prefill and decode throughput of the layered decoder at layer sizes of real models (random
+"""`bench.py --design fesenex|taruvik|lotazen|viladra|dimorax`: prefill and decode throughput of the layered decoder at layer sizes of real models (random
 weights), beside the dense `Transformer` of equal width / heads / feed-forward size / depth / vocabulary, plus the time of each
 hybrid kernel at those shapes against its roofline (bf16 tensor peak or HBM copy bandwidth from MEASURED_PEAKS.json).
 For `taruvik` (latent attention, mixture of experts) the neighbour is the `Transformer` with a mixture of experts of equal
 width / heads / experts / depth; for `lotazen` (rotary window attention beside a gated recurrence, matrix memories, experts with scaled
 input) it is the Fesenex design at equal width / heads / depth, and every new kernel is timed next to the like kernel at the same shape;
 for `viladra` (convolution on the stream, norms after the sublayers with a depth average, retention, gated linear attention,
-sigmoid-weight window attention, ungated experts) the neighbour is the Lotazen design at equal width / heads / experts / depth.  Timed with CUDA events after warm-up; the prompt batch and the weights exceed L2 at the larger size, and L2 is flushed between
+sigmoid-weight window attention, ungated experts) the neighbour is the Lotazen design at equal width / heads / experts / depth; for
+`dimorax` (gated delta rule, soft-capped attention with sinks, windowed latent attention, group-limited experts) too.  Timed with CUDA events after warm-up; the prompt batch and the weights exceed L2 at the larger size, and L2 is flushed between
 timed kernel launches.  Prints one JSON line."""
 import json
 import math
@@ -745,7 +746,216 @@ def run_viladra(a, peaks: dict) -> dict:
     return res
 
 
+# ----------------------------------------------------------------------------------------------- Dimorax
+DIMORAX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, lat_heads=16, lat_dim=128, rot_dim=64, kv_rank=512, window=1024, rec_heads=16, rec_kv_heads=16, taps=4, rank=64,
+                  experts=16, top=2, groups=4, keep=2, ff=1408, shared_ff=2816, dense_ff=5632, vocab=32768, order="dald"),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, lat_heads=32, lat_dim=128, rot_dim=64, kv_rank=512, window=2048, rec_heads=32, rec_kv_heads=16, taps=4, rank=128,
+                  experts=8, top=2, groups=4, keep=2, ff=3584, shared_ff=7168, dense_ff=14336, vocab=32768, order="adl"),
+}
+
+
+def dimorax_config(s: dict) -> dict:
+    d = s["dim"]
+    mixers = {
+        "a": {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 30.0,
+                                             "rot": {"base": 500000.0, "dims": d // 2, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}},
+        "l": {"type": "latent_attention", "mixer": {"heads": s["lat_heads"], "dim": s["lat_dim"], "rot_dim": s["rot_dim"], "vdim": s["lat_dim"], "kv_rank": s["kv_rank"],
+                                                    "scale": (s["lat_dim"] + s["rot_dim"]) ** -0.5, "mask": {"size": s["window"]}, "rot": {"base": 10000.0, "dims": s["rot_dim"]}}},
+        "d": {"type": "channel_delta", "mixer": {"heads": s["rec_heads"], "kv_heads": s["rec_kv_heads"], "dim": d, "vdim": d, "conv": s["taps"]}},
+    }
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"], "scale": 1.5, "groups": {"count": s["groups"], "keep": s["keep"]}},
+           "shared": {"ff": s["shared_ff"]}}
+    return {"architecture": "Dimorax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "layers": [{**mixers[c], "mlp": moe if i % 3 != 2 else {"kind": "dense", "ff": s["dense_ff"]}} for i, c in enumerate(s["order"])]}
+
+
+def build_dimorax(s: dict, dev):
+    from mistral_inference_b200.args import LayeredArgs
+    from mistral_inference_b200.layered import LayeredTransformer
+    from mistral_inference_b200.transformer_layers import DeltaMixer
+
+    m = LayeredTransformer.empty(LayeredArgs.from_dict(dimorax_config(s)), dev, torch.bfloat16)
+    for blk in m.layers:  # the ranks of the low-rank projections come with a checkpoint; here they are the size table's
+        if isinstance(blk.mix, DeltaMixer):
+            blk.mix.resize(s["rank"], s["rank"])
+    g = torch.Generator(device=dev).manual_seed(0)
+    with torch.no_grad():
+        for n, p in m.named_parameters():
+            last = n.rsplit(".", 1)[-1]
+            if p.dim() >= 2:
+                p.copy_(torch.randn(p.shape, generator=g, device=dev, dtype=torch.float32) / math.sqrt(p.shape[-1]))
+            elif last in ("norm", "c_norm"):
+                p.fill_(1.0)
+            elif last in ("dt_bias", "a_log"):
+                p.fill_(-2.0)
+            else:
+                p.copy_(torch.randn(p.shape, generator=g, device=dev, dtype=torch.float32) * 0.1)
+    return m.eval()
+
+
+def lotazen_like_dimorax(s: dict) -> dict:
+    """The closest existing design at equal size: rotary window attention beside a gated recurrence where Dimorax has attention, a matrix memory
+    elsewhere, gated experts of the same sizes in every layer."""
+    return dict(width=s["width"], heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"], window=s["window"], rec_heads=s["rec_heads"], experts=s["experts"],
+                top=s["top"], ff=s["ff"], shared_ff=s["shared_ff"], vocab=s["vocab"], order="".join("p" if c == "a" else "m" for c in s["order"]),
+                lin_heads=s["rec_heads"])
+
+
+def dimorax_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
+    """Every kernel the design added or extended, alone at this size, each next to the like kernel of an existing design at the same shape."""
+    from mistral_inference_b200 import _abi_hybrid as h
+    from mistral_inference_b200.cache import BufferCache, LayerCacheSpec
+    from mistral_inference_b200.rope import scaled_frequencies
+
+    bf = torch.bfloat16
+    W, H, G, d, E, ff, top, RH, RG, taps, rank = (s[k] for k in ("width", "heads", "kv_heads", "dim", "experts", "ff", "top", "rec_heads", "rec_kv_heads", "taps", "rank"))
+    LH, dn, dr, rk, win = (s[k] for k in ("lat_heads", "lat_dim", "rot_dim", "kv_rank", "window"))
+    flush = torch.zeros(160 << 20, dtype=torch.float32, device=dev)
+    rows = {}
+
+    def rec(name, fn, flops=0.0, bytes_=0.0, note=None, n=(3, 8)):
+        ms = _time(fn, n[0], n[1], flush)
+        r = {"ms": round(ms, 4)}
+        if flops:
+            r["tflops"] = round(flops / ms / 1e9, 2)
+            r["of_bf16_peak"] = round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)
+        if bytes_:
+            r["gb_s"] = round(bytes_ / ms / 1e6, 1)
+            r["of_hbm_peak"] = round(bytes_ / ms / 1e6 / peaks["hbm_gbs"], 3)
+        if note:
+            r["note"] = note
+        rows[name] = r
+
+    def rnd(*shape, scale=1.0):
+        return (torch.randn(*shape, device=dev) * scale).to(bf)
+
+    B, nt = 8, (T + 63) // 64
+    zero, one = torch.zeros(1, dtype=torch.int32, device=dev), torch.ones(B, dtype=torch.int32, device=dev)
+    # ---- norms
+    x32, nw = torch.randn(T, W, device=dev), torch.ones(W, device=dev).to(bf)
+    rec("rmsnorm_pair prompt (two norms, one pass)", lambda: h.rmsnorm_pair(x32, nw, nw, 1e-5, 1.0), bytes_=T * W * 8.0)
+    rec("like: rmsnorm prompt", lambda: h.rmsnorm(x32, nw, 1e-5), bytes_=T * W * 6.0)
+    # ---- attention
+    ring = BufferCache(1, B, ctx + 8, 0, 0, None, layer_specs=[LayerCacheSpec(kind="ring", n_kv_heads=G, k_dim=d, v_dim=d)]).to(dev, bf)
+    ring.cache_k[0].normal_(); ring.cache_v[0].normal_()
+    md = ring.get_input_metadata([T])[0]
+    qkv = rnd(T, (H + 2 * G) * d)
+    fh, fd = scaled_frequencies(d // 2, 5e5, None)[0].to(dev), scaled_frequencies(d, 5e5, None)[0].to(dev)
+    rec("rot_prep prompt (halves, half of each head)", lambda: h.rot_prep(qkv, fh, md.positions, None, None, None, H, G, d, d, d // 2, False, 0.0, own=True, halves=True, mag=1.2),
+        bytes_=4.0 * qkv.numel())
+    rec("like: rot_prep prompt (neighbours, unit norm)", lambda: h.rot_prep(qkv, fd, md.positions, None, None, None, H, G, d, d, d, True, 1e-5, own=True), bytes_=4.0 * qkv.numel())
+    q, k, v = h.rot_prep(qkv, fh, md.positions, None, None, None, H, G, d, d, d // 2, False, 0.0, own=True, halves=True)
+    o, sink = torch.empty(T, H * d, device=dev, dtype=bf), torch.zeros(H, device=dev)
+    for label, kw in (("attn_window prompt, soft cap and sinks", dict(softcap=30.0, sink=sink)), ("like: attn_window prompt, softmax", {})):
+        rec(f"{label} (tensor-core kernel)", lambda: h.attn_window(q, ring.cache_k[0], ring.cache_v[0], md.positions, md.q_start, md.slots, o, 1, md.window, H, G, d, d, 0.09, 0,
+                                                                   own_k=k, own_v=v, seqpos=md.seqpos, n_tiles=nt, **kw), flops=4.0 * d * H * T * (T + 1) / 2, n=(2, 5))
+    ring.reset(); ring.init_kvseqlens(B); ring.update_seqlens([ctx] * B)
+    md2 = ring.get_input_metadata([1] * B)[0]
+    q2, o2 = q[:B].contiguous(), torch.empty(B, H * d, device=dev, dtype=bf)
+    sp, ch = h.window_decode_plan(B, H, md2.window)
+    for label, kw in (("attn_window decode, soft cap and sinks", dict(softcap=30.0, sink=sink)), ("like: attn_window decode, softmax", {})):
+        rec(f"{label} B={B}", lambda: h.attn_window(q2, ring.cache_k[0], ring.cache_v[0], md2.positions, md2.q_start, md2.slots, o2, B, md2.window, H, G, d, d, 0.09, 0, splits=sp,
+                                                    chunk=ch, **kw), bytes_=2.0 * B * (ctx + 1) * G * d * 2)
+    # ---- latent attention
+    lat = BufferCache(2, B, ctx + 8, 0, 0, None, layer_specs=[LayerCacheSpec(kind="ring", n_kv_heads=1, k_dim=rk + dr, v_dim=0, window=w) for w in (win, None)]).to(dev, bf)
+    lat.cache_k[0].normal_(); lat.cache_k[1].normal_()
+    mw, mf = lat.get_input_metadata([T])
+    freq = scaled_frequencies(dr, 1e4, None)[0].to(dev)
+    nq = LH * (dn + dr)
+    y, cn, qn = rnd(T, nq + rk + dr), torch.ones(rk, device=dev).to(bf), torch.ones(rk, device=dev).to(bf)
+    rec("latent_prep prompt (rows beside the ring)", lambda: h.latent_prep(y, None, cn, freq, mw.positions, None, lat.cache_k[0], 0, rk, dr, dr, 1e-5, 1.0, kv_off=nq, halves=True, own=True),
+        bytes_=T * (rk + dr) * 4.0)
+    y2 = rnd(T, 2 * rk + dr)
+    rec("like: latent_prep prompt (query latent, ring)", lambda: h.latent_prep(y2, qn, cn, freq, mf.positions, mf.cache_rows, lat.cache_k[1], rk, rk, dr, dr, 1e-5, 1.0),
+        bytes_=T * (2 * rk + dr) * 4.0)
+    kf, vf, qr, of = rnd(T, LH, dn + dr), rnd(T, LH, dn), rnd(T, nq), torch.empty(T, LH * dn, device=dev, dtype=bf)
+    lsink, iota = torch.zeros(LH, device=dev), h.iota(1, dev)
+    pairs = sum(min(p + 1, win) for p in range(T))
+    for label, w, kw, n_pairs in ((f"latent prompt attention, window {win}, sinks", win, dict(sink=lsink), pairs), ("like: latent prompt attention, whole", 0, {}, T * (T + 1) / 2)):
+        rec(f"{label} (tensor-core kernel)", lambda: h.attn_window(qr, kf, vf, md.positions, md.q_start, iota, of, 1, 1, LH, LH, dn + dr, dn, 0.07, w, own_k=kf, own_v=vf, seqpos=zero,
+                                                                   n_tiles=nt, **kw), flops=2.0 * LH * (2 * dn + dr) * n_pairs, n=(2, 5))
+    kn, rows_ = rnd(T, LH * dn), rnd(T, rk + dr)
+    rec("latent_expand prompt", lambda: h.latent_expand(kn, rows_, LH, dn, dr, rk), bytes_=T * 2.0 * (LH * dn + dr + nq))
+    lat.reset(); lat.init_kvseqlens(B); lat.update_seqlens([ctx] * B)
+    mw2, mf2 = lat.get_input_metadata([1] * B)
+    qa = rnd(B, LH * (rk + dr))
+    for label, m_, i, w, kw, n in ((f"attn_latent_decode, window {win}, sinks", mw2, 0, win, dict(sink=lsink), min(ctx + 1, win)), ("like: attn_latent_decode, whole", mf2, 1, 0, {}, ctx + 1)):
+        rec(f"{label} B={B}", lambda: h.attn_latent_decode(qa, lat.cache_k[i], m_.positions, m_.slots, B, m_.window, LH, rk, dr, 0.07, w, **kw), bytes_=B * n * (rk + dr) * 2.0)
+    # ---- gated delta rule
+    Nk, He, Hd = RG * d, RH * d, RH * d
+    ch_, N = 2 * Nk + He, 2 * Nk + He + RH + 2 * rank
+    N = (N + 127) // 128 * 128
+    yd, conv = rnd(T, N), rnd(ch_, taps, scale=0.3)
+    cstate, state = torch.zeros(B, taps, ch_, device=dev), torch.zeros(B, RH, d, d, device=dev)
+    wa2, wg2, dtb, alog, hw = rnd(Hd, rank, scale=0.1), rnd(He, rank, scale=0.1), torch.full((Hd,), -2.0, device=dev).to(bf), torch.full((RH,), -2.0, device=dev).to(bf), torch.ones(d, device=dev).to(bf)
+    prep = lambda: h.delta_prep(yd, conv, cstate, md.positions, md.q_start, zero, md.slots, 1, RH, RG, d, d)  # noqa: E731
+    rec("delta_prep prompt (convolutions, unit norms; incl. the carried inputs' launch)", prep, bytes_=T * ch_ * (2 + 4.0))
+    z32 = torch.randn(T, Hd, device=dev)
+    qkvg = rnd(T, 4 * Hd, scale=0.1)
+    rec("like: gla_qab prompt", lambda: h.gla_qab(qkvg, z32, Hd, d ** -0.5, 1 / 16.0), bytes_=T * Hd * (2 * 2 + 4 + 3 * 4.0))
+    xa = yd[:, ch_ + RH: ch_ + RH + rank]
+    rec(f"linear_decay prompt (rank {rank} -> decays, fp32 out)", lambda: h.linear_decay(xa, wa2, dtb, alog, d), bytes_=T * (rank * 2 + Hd * 4.0))
+    xc = xa.contiguous()
+    rec(f"like: linear prompt (rank {rank}, fp32 out)", lambda: h.linear(xc, wa2, dtb, epi=h.EPI_F32), bytes_=T * (rank * 2 + Hd * 4.0))
+    qk, kq, vv, beta = prep()
+    g = h.linear_decay(xa, wa2, dtb, alog, d)
+    rec("delta_scan prompt", lambda: h.delta_scan(qk, kq, vv, beta, g, state, md.q_start, zero, md.slots, 1, RH, RG, d, d), flops=6.0 * T * RH * d * d, n=(2, 5),
+        note="useful FLOPs, fp32 FMA, one dependent step per token")
+    qab = h.gla_qab(qkvg, z32, Hd, d ** -0.5, 1 / 16.0)
+    gst = torch.zeros(B, RH, d, d, device=dev)
+    rec("like: gated_scan prompt, chunk-parallel", lambda: h.gated_scan(qab, qkvg, 4 * Hd, 2 * Hd, gst, md.q_start, zero, md.slots, 1, RH, d, d, ones=False, max_seqlen=T),
+        flops=4.0 * T * RH * d * d, n=(2, 5), note="useful FLOPs, the chunks run twice, fp32 FMA")
+    ydB, qabB = yd[:B].contiguous(), qab[:B].contiguous()
+    rec(f"delta_step decode B={B} (convolutions, decays, state, norm, gate in one)",
+        lambda: h.delta_step(ydB, rank, rank, conv, cstate, state, wa2, dtb, alog, wg2, hw, md2.positions, one, md2.slots, RH, RG, d, d, 1e-5), bytes_=2.0 * state.numel() * 4)
+    rec(f"like: gated_scan decode B={B} (the state only)", lambda: h.gated_scan(qabB, qkvg, 4 * Hd, 2 * Hd, gst, md2.q_start, one, md2.slots, B, RH, d, d, ones=False),
+        bytes_=2.0 * gst.numel() * 4)
+    # ---- feed-forward
+    x = rnd(T, W)
+    w13, w2, wr, corr = rnd(E * 2 * ff, W, scale=0.02), rnd(W, E * ff, scale=0.02), rnd(E, W, scale=4 / math.sqrt(W)), torch.zeros(E, device=dev).to(bf)
+    route = lambda t: h.moe_route(t, wr, corr, s["groups"], s["keep"], top, score=1, scale=1.5, group_two=True, renorm=True)  # noqa: E731
+    rec("moe_route prompt (groups by two, renormalised)", lambda: route(x), bytes_=T * W * 2.0)
+    rec("like: moe_route prompt (sigmoid)", lambda: h.moe_route(x, wr, None, 1, 1, top, score=1), bytes_=T * W * 2.0)
+    dense, idx, wsel = route(x)
+    xr = torch.zeros(T, W, device=dev)
+    rec("experts prompt (all experts, masked)", lambda: h.linear(h.linear_swiglu(x, w13, rowscale=dense, group=ff), w2, epi=h.EPI_RESIDUAL, residual=xr), flops=6.0 * T * top * ff * W,
+        note=f"useful FLOPs (top {top} of {E}); the kernels compute all {E} experts", n=(2, 5))
+    rec("like: experts prompt of the scaled-input gated mixture", lambda: h.linear(h.linear_glu(x, w13, 7.0, 1.702, rowscale=dense, group=ff), w2, epi=h.EPI_RESIDUAL, residual=xr),
+        flops=6.0 * T * top * ff * W, n=(2, 5))
+    for M in (1, B):
+        xs, ii, ww, xm = x[:M].contiguous(), idx[:M].contiguous(), wsel[:M].contiguous(), xr[:M].contiguous()
+        rec(f"experts decode (chosen only) M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, add_to=xm), bytes_=M * top * 3.0 * ff * W * 2)
+        rec(f"like: experts decode of the scaled-input gated mixture M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, glu=1, limit=7.0, alpha=1.702, add_to=xm),
+            bytes_=M * top * 3.0 * ff * W * 2)
+    wd = rnd(2 * s["dense_ff"], W, scale=0.02)
+    rec("linear_swiglu prompt (gelu)", lambda: h.linear_swiglu(x, wd, gelu=True), flops=4.0 * T * s["dense_ff"] * W, n=(2, 5))
+    rec("like: linear prompt (clamped gated unit)", lambda: h.linear_glu(x, wd, 7.0, 1.702), flops=4.0 * T * s["dense_ff"] * W, n=(2, 5))
+    return rows
+
+
+def run_dimorax(a, peaks: dict) -> dict:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    T, ctx = a.prefill, a.prefill
+    res = {"design": "Dimorax", "dtype": "bf16", "data": "synthetic", "prompt_tokens": T, "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
+    for name, s in DIMORAX_SIZES.items():
+        t0 = time.time()
+        m = build_dimorax(s, dev)
+        new = end_to_end(m, s["vocab"], T, ctx, (1, 8), a.warmup, a.steps, dev)
+        del m
+        torch.cuda.empty_cache()
+        d = build_lotazen(lotazen_like_dimorax(s), dev)
+        old = end_to_end(d, s["vocab"], T, ctx, (1, 8), a.warmup, a.steps, dev)
+        del d
+        torch.cuda.empty_cache()
+        res["sizes"][name] = {"config": s, "layered": new, "lotazen_equal_size": old, "kernels": dimorax_kernel_table(s, T, ctx, peaks, dev),
+                              "seconds": round(time.time() - t0, 1)}
+    return res
+
+
 def run(a, peaks: dict) -> dict:
+    if a.design == "dimorax":
+        return run_dimorax(a, peaks)
     if a.design == "viladra":
         return run_viladra(a, peaks)
     if a.design == "taruvik":

@@ -72,7 +72,7 @@ def build_hybrid(force: bool = False) -> Path:
     """libmb200_hybrid.so: the kernels of layered decoders (csrc/hybrid/), a separate, small library so that a fresh checkout
     that only serves such a model compiles only them (seconds).  Safe when several processes start at once: the output is
     written under a private name and renamed."""
-    files = sorted(HYBRID_SRC.glob("*.cu")) + sorted(HYBRID_SRC.glob("*.cuh")) + [PKG.parent / "include" / "mistral_b200_hybrid.h"]
+    files = sorted(HYBRID_SRC.glob("*.cu")) + sorted(HYBRID_SRC.glob("*.cuh")) + sorted(HYBRID_SRC.glob("*.h")) + [PKG.parent / "include" / "mistral_b200_hybrid.h"]
     h = hashlib.sha256()
     for f in files:
         h.update(f.name.encode())
@@ -84,7 +84,7 @@ def build_hybrid(force: bool = False) -> Path:
         return HYBRID_LIB
     nvcc = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
     tmp = PKG / f".libmb200_hybrid.{os.getpid()}.so"
-    cmd = [nvcc, *NVCC_FLAGS, "-o", str(tmp)] + [str(f) for f in sorted(HYBRID_SRC.glob("*.cu"))]
+    cmd = [nvcc, *NVCC_FLAGS, "--threads", "0", "-o", str(tmp)] + [str(f) for f in sorted(HYBRID_SRC.glob("*.cu"))]
     proc = subprocess.run(cmd, capture_output=True, text=True)
     if proc.returncode != 0:
         sys.stderr.write(proc.stdout + proc.stderr)

@@ -9,7 +9,7 @@
 #include "hybrid_rotary.cuh"
 #include "hybrid_gated_scan.cuh"
 #include "hybrid_stream.cuh"
-#include "hybrid_delta.cuh"
+#include "hybrid_error.h"
 #include "../../../include/mistral_b200_hybrid.h"
 
 #include <stdio.h>
@@ -18,20 +18,16 @@ using namespace mbh;
 
 static thread_local char g_err[256] = "";
 
-static int fail(cudaError_t e, const char* what) {
+__attribute__((visibility("hidden"))) int mbh_fail(cudaError_t e, const char* what) {
     snprintf(g_err, sizeof(g_err), "%s: %s", what, cudaGetErrorString(e));
     return (int)e;
 }
-static int bad(const char* what) {
+__attribute__((visibility("hidden"))) int mbh_bad(const char* what) {
     snprintf(g_err, sizeof(g_err), "%s", what);
     return -1;
 }
-#define DISPATCH(dt, ...)                                   \
-    do {                                                    \
-        if ((dt) == 0) { using ST = bf16; __VA_ARGS__; }     \
-        else if ((dt) == 1) { using ST = float; __VA_ARGS__; } \
-        else return bad("dt must be 0 (bf16) or 1 (fp32)"); \
-    } while (0)
+static int fail(cudaError_t e, const char* what) { return mbh_fail(e, what); }
+static int bad(const char* what) { return mbh_bad(what); }
 
 template <typename T>
 static cudaError_t launch_lightning(const LightningArgs& a, cudaStream_t st) {
@@ -143,43 +139,6 @@ template <typename T> static cudaError_t launch_latent_decode(const LatentDecode
     return run_latent_decode<T, 4>(a, out, sink, smem, st);
 }
 
-// key size -> lanes per state column and float4 per lane; tokens per shared-memory tile
-static cudaError_t launch_delta_scan(const DeltaArgs& a, cudaStream_t st) {
-    auto grid = [&](int lanes) { return dim3((unsigned)(a.B * a.H), (unsigned)((a.e + DS_THREADS / lanes - 1) / (DS_THREADS / lanes))); };
-    if (a.d <= 32) delta_scan_kernel<8, 1, 16><<<grid(8), DS_THREADS, 0, st>>>(a);
-    else if (a.d <= 64) delta_scan_kernel<8, 2, 16><<<grid(8), DS_THREADS, 0, st>>>(a);
-    else if (a.d <= 128) delta_scan_kernel<8, 4, 8><<<grid(8), DS_THREADS, 0, st>>>(a);
-    else if (a.d <= 256) delta_scan_kernel<8, 8, 4><<<grid(8), DS_THREADS, 0, st>>>(a);
-    else delta_scan_kernel<32, 8, 1><<<grid(32), DS_THREADS, 0, st>>>(a);
-    return cudaGetLastError();
-}
-template <typename T> static cudaError_t launch_delta_prep(const DeltaArgs& a, cudaStream_t st) {
-    // few tokens: the units of a token are spread over CTAs; long prompts: each CTA walks several units of its tokens
-    const unsigned tiles = (unsigned)((a.T + DP_WARPS - 1) / DP_WARPS), units = (unsigned)(a.G + a.H);
-    const dim3 grid(tiles, units < 65535u ? units : 65535u);
-    if (a.d <= 64) delta_prep_kernel<T, 2><<<grid, DP_WARPS * 32, 0, st>>>(a);
-    else if (a.d <= 128) delta_prep_kernel<T, 4><<<grid, DP_WARPS * 32, 0, st>>>(a);
-    else if (a.d <= 256) delta_prep_kernel<T, 8><<<grid, DP_WARPS * 32, 0, st>>>(a);
-    else delta_prep_kernel<T, 32><<<grid, DP_WARPS * 32, 0, st>>>(a);
-    if (a.taps > 1) delta_conv_state_kernel<T><<<dim3((unsigned)a.B, (unsigned)((2 * a.G * a.d + a.H * a.e + 255) / 256)), 256, 0, st>>>(a);
-    return cudaGetLastError();
-}
-template <typename T, int LANES, int RPL4> static cudaError_t run_delta_step(const DeltaArgs& a, cudaStream_t st) {
-    const size_t smem = sizeof(float) * (5 * (size_t)DeltaColumn<LANES, RPL4>::DMAX + 3 * (size_t)a.e + a.ra + a.rg);
-    if (smem > 220 * 1024) return cudaErrorInvalidValue;
-    cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, LANES, RPL4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e) return e;
-    delta_step_kernel<T, LANES, RPL4><<<(unsigned)(a.B * a.H), DT_THREADS, smem, st>>>(a);
-    return cudaGetLastError();
-}
-template <typename T> static cudaError_t launch_delta_step(const DeltaArgs& a, cudaStream_t st) {
-    if (a.d <= 32) return run_delta_step<T, 8, 1>(a, st);
-    if (a.d <= 64) return run_delta_step<T, 8, 2>(a, st);
-    if (a.d <= 128) return run_delta_step<T, 8, 4>(a, st);
-    if (a.d <= 256) return run_delta_step<T, 8, 8>(a, st);
-    return run_delta_step<T, 32, 8>(a, st);
-}
-
 extern "C" {
 
 int mbh_abi_version(void) { return MBH_ABI_VERSION; }
@@ -222,6 +181,7 @@ int mbh_linear_decay(const void* x, int64_t ldx, const void* w, const void* bias
     a.a_log = a_log;
     a.ldx = (int)ldx;
     cudaError_t e = cudaSuccess;
+    if (dt == 0 && launch_linear_decay_mma(a, (cudaStream_t)stream, e)) return e ? fail(e, "mbh_linear_decay") : 0;
     DISPATCH(dt, e = launch_linear<ST>(a, (cudaStream_t)stream));
     return e ? fail(e, "mbh_linear_decay") : 0;
 }
@@ -681,51 +641,6 @@ int mbh_relu2_epilogue(const void* y, void* out, int64_t M, int64_t N, const voi
     DISPATCH(dt, run_epilogue<ST>(a, y, st));
     cudaError_t e = cudaGetLastError();
     return e ? fail(e, "mbh_relu2_epilogue") : 0;
-}
-
-int mbh_delta_prep(const void* y, int64_t y_pitch, const void* conv, int64_t taps, void* cstate, const void* positions, const void* q_start, const void* seqpos,
-                   const void* slots, void* qk, void* kq, void* v, void* beta, int64_t T, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, int dt,
-                   void* stream) {
-    if (T == 0 || B == 0) return 0;
-    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_prep: key size 1 .. 1024, heads a multiple of key heads");
-    if (taps < 1) return bad("mbh_delta_prep: at least one tap");
-    DeltaArgs a{};
-    a.y = y; a.y_pitch = (int)y_pitch; a.conv = conv; a.taps = (int)taps; a.cstate = (float*)cstate;
-    a.positions = (const int*)positions; a.q_start = (const int*)q_start; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots;
-    a.T = (int)T; a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e;
-    a.qk = (float*)qk; a.kq = (float*)kq; a.v = (float*)v; a.beta = (float*)beta;
-    cudaError_t err = cudaSuccess;
-    DISPATCH(dt, err = launch_delta_prep<ST>(a, (cudaStream_t)stream));
-    return err ? fail(err, "mbh_delta_prep") : 0;
-}
-
-int mbh_delta_scan(const void* qk, const void* kq, const void* v, const void* beta, const void* g, void* state, const void* q_start, const void* seqpos,
-                   const void* slots, void* o32, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, void* stream) {
-    if (B == 0) return 0;
-    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_scan: key size 1 .. 1024, heads a multiple of key heads");
-    DeltaArgs a{};
-    a.q_start = (const int*)q_start; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots; a.state = (float*)state;
-    a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e;
-    a.qk = (float*)const_cast<void*>(qk); a.kq = (float*)const_cast<void*>(kq); a.v = (float*)const_cast<void*>(v); a.beta = (float*)const_cast<void*>(beta);
-    a.g = (const float*)g; a.o = (float*)o32;
-    cudaError_t err = launch_delta_scan(a, (cudaStream_t)stream);
-    return err ? fail(err, "mbh_delta_scan") : 0;
-}
-
-int mbh_delta_step(const void* y, int64_t y_pitch, int64_t ra, int64_t rg, const void* conv, int64_t taps, void* cstate, void* state, const void* w_a2,
-                   const void* dt_bias, const void* a_log, const void* w_g2, const void* norm, const void* positions, const void* seqpos, const void* slots,
-                   void* out, int64_t B, int64_t H, int64_t G, int64_t d, int64_t e, float eps, int dt, void* stream) {
-    if (B == 0) return 0;
-    if (d < 1 || d > 1024 || e < 1 || G < 1 || H % G) return bad("mbh_delta_step: key size 1 .. 1024, heads a multiple of key heads");
-    if (taps < 1) return bad("mbh_delta_step: at least one tap");
-    DeltaArgs a{};
-    a.y = y; a.y_pitch = (int)y_pitch; a.ra = (int)ra; a.rg = (int)rg; a.conv = conv; a.taps = (int)taps; a.cstate = (float*)cstate; a.state = (float*)state;
-    a.w_a2 = w_a2; a.dt_bias = dt_bias; a.a_log = a_log; a.w_g2 = w_g2; a.norm = norm;
-    a.positions = (const int*)positions; a.seqpos = (const int*)seqpos; a.slots = (const int*)slots;
-    a.T = (int)B; a.B = (int)B; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e; a.eps = eps; a.out = out;
-    cudaError_t err = cudaSuccess;
-    DISPATCH(dt, err = launch_delta_step<ST>(a, (cudaStream_t)stream));
-    return err ? fail(err, "mbh_delta_step") : 0;
 }
 
 }  // extern "C"

@@ -236,8 +236,92 @@ __global__ void __launch_bounds__(MM_THREADS) linear_tiled_mma(LinearArgs a) {
         }
 }
 
+constexpr int SK_MAX_M = 8, SK_WARPS = 8;  // up to SK_MAX_M rows take the skinny kernels
+
+// ------------------------------------------------------------------------------------------------ decays from a low rank (bf16 prompts)
+// EPI_DECAY for K up to LDK_MAX_K: both operands of a 64 x 128 tile lie in shared memory whole (one load phase, no pipeline), the work is the
+// output: per column bias and -exp(a_log) are prepared once per CTA, then softplus, exp and 8-byte stores from the accumulators.
+constexpr int LDK_BM = 64, LDK_BN = 128, LDK_MAX_K = 256;
+
+__global__ void __launch_bounds__(256) linear_decay_mma(LinearArgs a) {
+    extern __shared__ __align__(16) unsigned char ldk_smem[];
+    __shared__ float cb[LDK_BN], ca[LDK_BN];
+    const int ld = a.K + 8;
+    bf16* As = reinterpret_cast<bf16*>(ldk_smem);
+    bf16* Ws = As + LDK_BM * ld;
+    const bf16* X = static_cast<const bf16*>(a.x);
+    const bf16* W = static_cast<const bf16*>(a.w);
+    const int m0 = blockIdx.y * LDK_BM, n0 = blockIdx.x * LDK_BN, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+    const int wm = (warp >> 2) * 32, wn = (warp & 3) * 32, kc = a.K / 8;
+    for (int i = tid; i < (LDK_BM + LDK_BN) * kc; i += 256) {
+        const int r = i / kc, k = (i % kc) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (r < LDK_BM) {
+            if (m0 + r < a.M) v = *reinterpret_cast<const uint4*>(X + (size_t)(m0 + r) * a.x_pitch() + k);
+        } else if (n0 + r - LDK_BM < a.N) {
+            v = *reinterpret_cast<const uint4*>(W + (size_t)(n0 + r - LDK_BM) * a.K + k);
+        }
+        *reinterpret_cast<uint4*>(As + (size_t)r * ld + k) = v;
+    }
+    for (int i = tid; i < LDK_BN; i += 256) {
+        const int n = min(n0 + i, a.N - 1);
+        cb[i] = a.bias ? to_f(static_cast<const bf16*>(a.bias)[n]) : 0.f;
+        ca[i] = -expf(to_f(static_cast<const bf16*>(a.a_log)[n / a.rs_group]));
+    }
+    __syncthreads();
+    float acc[2][4][4] = {};
+    for (int k = 0; k < a.K; k += 16) {
+        uint32_t af[2][4], bfr[4][2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const bf16* p = As + (size_t)(wm + i * 16 + gid) * ld + k + tig * 2;
+            af[i][0] = *reinterpret_cast<const uint32_t*>(p);
+            af[i][1] = *reinterpret_cast<const uint32_t*>(p + 8 * ld);
+            af[i][2] = *reinterpret_cast<const uint32_t*>(p + 8);
+            af[i][3] = *reinterpret_cast<const uint32_t*>(p + 8 * ld + 8);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const bf16* p = Ws + (size_t)(wn + j * 8 + gid) * ld + k + tig * 2;
+            bfr[j][0] = *reinterpret_cast<const uint32_t*>(p);
+            bfr[j][1] = *reinterpret_cast<const uint32_t*>(p + 8);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) mma_bf16(acc[i][j], af[i], bfr[j][0], bfr[j][1]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int c = wn + j * 8 + tig * 2, n = n0 + c;
+            if (n >= a.N) continue;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int m = m0 + wm + i * 16 + gid + 8 * half;
+                if (m >= a.M) continue;
+                float2 o;
+                o.x = expf(ca[c] * softplus_exact(acc[i][j][2 * half] + cb[c]));
+                o.y = expf(ca[c + 1] * softplus_exact(acc[i][j][2 * half + 1] + cb[c + 1]));
+                *reinterpret_cast<float2*>(a.out32 + (size_t)m * a.N + n) = o;
+            }
+        }
+}
+
+// true when the shape suits linear_decay_mma; launches it
+inline bool launch_linear_decay_mma(const LinearArgs& a, cudaStream_t st, cudaError_t& e) {
+    if (a.M <= SK_MAX_M || a.K % 16 || a.K > LDK_MAX_K || a.N % 2 || a.x_pitch() % 8) return false;
+    if ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.out32)) % 16) return false;
+    const size_t smem = sizeof(bf16) * (size_t)(LDK_BM + LDK_BN) * (a.K + 8);
+    e = cudaFuncSetAttribute(linear_decay_mma, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e) return true;
+    linear_decay_mma<<<dim3((a.N + LDK_BN - 1) / LDK_BN, (a.M + LDK_BM - 1) / LDK_BM), 256, smem, st>>>(a);
+    e = cudaGetLastError();
+    return true;
+}
+
 // ------------------------------------------------------------------------------------------------ skinny (decode)
-constexpr int SK_MAX_M = 8, SK_WARPS = 8;
 
 // R weight rows per warp (R even: gate/up pairs stay together); more rows per warp = fewer re-reads of x per weight byte
 template <typename T, int MM, int R>
