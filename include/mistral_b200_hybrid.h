@@ -126,9 +126,10 @@ int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_
 
 /* Router of a mixture of experts, fp32: s = softmax(W_r h) over n outputs (score 0) or sigmoid of each output (score 1), choice = s + correction (null: none); the outputs form
  * `groups` equal groups of neighbours and only those of the `keep` groups with the largest choice (group_two: the largest sum of the two largest
- * choices) stay eligible; the `top` largest eligible choices are taken, weighted by s * scale (renorm: s / (sum of the chosen s + 1e-20) * scale).  dense: fp32 [T, n] (0 where not chosen); idx int32 / wsel fp32 [T, top]. */
+ * choices) stay eligible; the `top` largest eligible choices are taken, weighted by s * scale (renorm: s / (sum of the chosen s + 1e-20) * scale).  w_gate [width], gate fp32 [T] (both or null): gate =
+ * sigmoid(w_gate . h), beside the routing.  dense: fp32 [T, n] (0 where not chosen); idx int32 / wsel fp32 [T, top]. */
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, int dt, void* stream);
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate, int dt, void* stream);
 
 /* The chosen experts of few tokens: y32 [T, width] = sum_k wsel[t, k] * expert(idx[t, k])(h[t]); an index >= E is an identity
  * expert (output = h[t]).  w13 [E * 2 * ff, width] (gate and up rows interleaved), w2 [width, E * ff]; act: scratch [T * top, ff].

@@ -42,7 +42,7 @@ _SIGNATURES = {
     "mbh_attn_latent": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, I, P, P, P, c_int, P]),
     "mbh_attn_latent_decode": (c_int, [P, P, P, P, P, I, I, I, I, I, F, I, P, I, P, c_int, P]),
     "mbh_latent_vup": (c_int, [P, P, P, I, I, P, I, I, I, I, c_int, P]),
-    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, c_int, P]),
+    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, P, P, c_int, P]),
     "mbh_moe_sparse": (c_int, [P, P, P, P, P, P, P, I, I, I, I, I, c_int, F, F, c_int, c_int, P]),
     "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, I, c_int, F, P, c_int, P]),
     "mbh_linear_glu": (c_int, [P, P, P, I, I, I, F, F, P, I, I, c_int, P]),
@@ -275,18 +275,19 @@ def linear_swiglu(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Ten
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], groups: int, keep: int, top: int, score: int = 0,
-              scale: float = 1.0, group_two: bool = False, renorm: bool = False):
+              scale: float = 1.0, group_two: bool = False, renorm: bool = False, w_gate: Optional[torch.Tensor] = None):
     """(dense fp32 [T, n], idx int32 [T, top], wsel fp32 [T, top]) of the fp32 router; score 0: softmax, 1: sigmoid; the weights are the
     chosen scores times `scale` (renorm: first divided by their sum).  group_two: a group of outputs counts the sum of its two largest
-    choices instead of its largest."""
+    choices instead of its largest.  With w_gate ([1, width]) a fourth result: sigmoid(w_gate . h), fp32 [T, 1]."""
     T, D = h.shape
     n = w_router.shape[0]
     dense = torch.empty(T, n, dtype=torch.float32, device=h.device)
     idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
     wsel = torch.empty(T, top, dtype=torch.float32, device=h.device)
+    gate = torch.empty(T, 1, dtype=torch.float32, device=h.device) if w_gate is not None else None
     _check(lib().mbh_moe_route(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(dense), _ptr(idx), _ptr(wsel), T, D, n, groups, keep, top, score,
-                               scale, int(group_two), int(renorm), dt_of(h.dtype), _stream()), "mbh_moe_route")
-    return dense, idx, wsel
+                               scale, int(group_two), int(renorm), _ptr(w_gate), _ptr(gate), dt_of(h.dtype), _stream()), "mbh_moe_route")
+    return (dense, idx, wsel) if gate is None else (dense, idx, wsel, gate)
 
 
 def moe_sparse(h: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, idx: torch.Tensor, wsel: torch.Tensor, E: int, ff: int,
@@ -375,9 +376,9 @@ LATENT_DECODE_MAX_HEADS, LATENT_DECODE_MAX_RANK = 32, 512
 
 
 def latent_decode_splits(B: int, W: int, n_sm: int = 148) -> int:
-    """CTAs per sequence along the keys: two CTAs per SM over the batch, at least 64 ring rows each (batch and ring size only, so a
+    """CTAs per sequence along the keys: two CTAs per SM over the batch, at least a tile of 32 ring rows each (batch and ring size only, so a
     captured decode graph stays valid as the context grows)."""
-    return int(max(1, min((2 * n_sm) // B, (W + 63) // 64, 64)))
+    return int(max(1, min((2 * n_sm) // B, (W + 31) // 32, 64)))
 
 
 def attn_latent_decode(qa, ring, positions, slots, B: int, W: int, H: int, kv_rank: int, rot_dim: int, scale: float, window: int = 0, sink=None) -> torch.Tensor:

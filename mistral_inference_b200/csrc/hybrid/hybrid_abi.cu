@@ -110,6 +110,9 @@ template <typename T> static void run_rmsnorm(const void* x32, const void* w, co
     rmsnorm_f32_kernel<T><<<(unsigned)T_, D >= 1024 ? 256 : 128, 0, st>>>((const float*)x32, (const T*)w, (const T*)w2, (T*)y, (T*)y2, (int)D, eps, offset);
 }
 template <typename T> static void run_epilogue(const LinearArgs& a, const void* y, cudaStream_t st) {
+    if constexpr (sizeof(T) == 2) {
+        if (launch_epilogue8(a, (const bf16*)y, st)) return;
+    }
     const size_t pairs = (size_t)a.M * (a.N >> 1);
     linear_epilogue_kernel<T><<<(unsigned)((pairs + 255) / 256), 256, 0, st>>>(a, (const T*)y);
 }
@@ -392,14 +395,15 @@ int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_
 }
 
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, int dt, void* stream) {
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate, int dt, void* stream) {
     if (T == 0) return 0;
+    if (!w_gate != !gate) return bad("mbh_moe_route: a gate needs its weight and its output");
     if (groups < 1 || n % groups || keep < 1 || keep > groups) return bad("mbh_moe_route: groups must divide the routed outputs, 1 <= keep <= groups");
     if (top < 1 || top > n / groups * keep) return bad("mbh_moe_route: top exceeds the eligible outputs");
     const size_t smem = sizeof(float) * (size_t)(2 * n + 2 * groups);
     if (smem > 48 * 1024) return bad("mbh_moe_route: too many routed outputs");
     if (score != 0 && score != 1) return bad("mbh_moe_route: score is 0 (softmax) or 1 (sigmoid)");
-    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, scale, group_two, renorm};
+    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, scale, group_two, renorm, w_gate, (float*)gate};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, moe_route_kernel<ST><<<(unsigned)T, MOE_ROUTE_THREADS, smem, st>>>(a));
     cudaError_t e = cudaGetLastError();

@@ -435,6 +435,87 @@ __global__ void linear_epilogue_kernel(LinearArgs a, const T* __restrict__ y) {
     epilogue_pair<T>(a, m, n, to_f(y[(size_t)m * a.N + n]), to_f(y[(size_t)m * a.N + n + 1]), true);
 }
 
+// The same eight columns per thread (16-byte loads, 16- or 8-byte stores), one row per grid row; needs N % 8 == 0 and 16-byte aligned rows.
+// Gated units whose rowscale is 0 (experts that the token did not choose) are written as 0 without reading y.
+__global__ void __launch_bounds__(256) linear_epilogue8_kernel(LinearArgs a, const bf16* __restrict__ y) {
+    const int m = blockIdx.y, n = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (n >= a.N) return;
+    const bool glu = a.epi == EPI_GLU || a.epi == EPI_SWIGLU || a.epi == EPI_GEGLU;
+    float rs[4] = {1.f, 1.f, 1.f, 1.f};
+    bf16* out = static_cast<bf16*>(a.out);
+    if (glu && a.rowscale) {
+        const float* r = a.rowscale + (size_t)m * a.rs_pitch;
+        const int c = n >> 1, g = c / a.rs_group;
+        if ((c + 3) / a.rs_group == g) {
+            rs[0] = rs[1] = rs[2] = rs[3] = r[g];
+            if (rs[0] == 0.f) {
+                *reinterpret_cast<uint2*>(out + (size_t)m * (a.N >> 1) + c) = make_uint2(0, 0);
+                return;
+            }
+        } else {
+#pragma unroll
+            for (int u = 0; u < 4; ++u) rs[u] = r[(c + u) / a.rs_group];
+        }
+    }
+    float v[8];
+    Vec<bf16>::load(y + (size_t)m * a.N + n, v);
+    if (a.bias) {
+        float b[8];
+        Vec<bf16>::load(static_cast<const bf16*>(a.bias) + n, b);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) v[u] = a.epi == EPI_F32 ? v[u] + b[u] : rnd<bf16>(v[u] + b[u]);
+    }
+    if (glu) {
+        float o[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            float g = v[2 * u], p = v[2 * u + 1];
+            if (a.epi == EPI_GLU) {
+                g = fminf(g * rs[u], a.limit);
+                p = fminf(fmaxf(p * rs[u], -a.limit), a.limit);
+                o[u] = g * sigmoid_exact(a.alpha * g) * (p + 1.f);
+            } else {
+                o[u] = (a.epi == EPI_GEGLU ? gelu_tanh(g) : g * sigmoid_exact(g)) * p * rs[u];
+            }
+        }
+        store4<bf16>(out + (size_t)m * (a.N >> 1) + (n >> 1), o);
+        return;
+    }
+    if (a.epi == EPI_STORE) {
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (n + u < a.n_act) v[u] = v[u] * sigmoid_exact(v[u]);
+        store4<bf16>(out + (size_t)m * a.N + n, v);
+        store4<bf16>(out + (size_t)m * a.N + n + 4, v + 4);
+        return;
+    }
+    float4* o = reinterpret_cast<float4*>(a.out32 + (size_t)m * a.N + n);
+    if (a.epi == EPI_F32) {
+        if (a.limit > 0.f) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) v[u] = a.limit * tanhf(v[u] / a.limit);
+        }
+        o[0] = make_float4(v[0], v[1], v[2], v[3]);
+        o[1] = make_float4(v[4], v[5], v[6], v[7]);
+        return;
+    }
+    const float f = a.epi == EPI_RESIDUAL_SCALED ? a.alpha : 1.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+        float4 r = o[u];
+        r.x += f * v[4 * u]; r.y += f * v[4 * u + 1]; r.z += f * v[4 * u + 2]; r.w += f * v[4 * u + 3];
+        o[u] = r;
+    }
+}
+
+// true when the shape and the epilogue suit linear_epilogue8_kernel; launches it
+inline bool launch_epilogue8(const LinearArgs& a, const bf16* y, cudaStream_t st) {
+    if (a.N % 8 || a.M > 65535 || a.epi == EPI_RELU2 || a.epi == EPI_DECAY) return false;
+    if ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(a.bias) | reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.out32)) % 16) return false;
+    linear_epilogue8_kernel<<<dim3((unsigned)((a.N / 8 + 255) / 256), (unsigned)a.M), 256, 0, st>>>(a, y);
+    return true;
+}
+
 template <typename T>
 inline cudaError_t launch_linear(const LinearArgs& a, cudaStream_t st) {
     if (a.M <= 0 || a.N <= 0) return cudaSuccess;

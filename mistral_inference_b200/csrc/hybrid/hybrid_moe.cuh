@@ -4,7 +4,7 @@
 //                     experts: output = input); choice = s + correction; the n outputs form `groups` equal groups of
 //                     neighbours, a group scores its largest choice (or the sum of its two largest), only the best `keep` groups stay eligible; the `top`
 //                     largest eligible choices are taken, each weighted by its s, optionally divided by the sum of the chosen ones' s.  Ties go to the lower index.
-//                     Writes the dense weights [T, n] (0 where not chosen) and the chosen (index, weight) pairs [T, top].
+//                     One more output may gate a shared expert (its sigmoid, not routed).  Writes the dense weights [T, n] (0 where not chosen) and the chosen (index, weight) pairs [T, top].
 //   moe_gateup_sparse / moe_down_sparse   few tokens (decode): one CTA column per (token, chosen expert) streams only that
 //                     expert's rows: act = silu(W_gate h) * (W_up h), then y = sum_k w_k W_down[e_k] act_k + (identity weights) h
 //   rows_axpy         y[t] += (sum of the identity weights of t) * h[t]       (after the dense, masked form for prompts)
@@ -29,6 +29,8 @@ struct MoeRouteArgs {
     float scale;              // the weights (dense and wsel) are the chosen scores times this
     int group_two;            // a group scores the sum of its two largest choices instead of its largest
     int renorm;               // the weights are divided by (the sum of the chosen scores + 1e-20)
+    const void* w_gate;       // [width] or null: one more output whose sigmoid gates a shared expert ...
+    float* gate;              // [T] ... goes here; it takes no part in the routing
 };
 
 // (value, index) argmax over a warp; the lower index wins a tie
@@ -73,9 +75,12 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     const T* h = static_cast<const T*>(a.h) + (size_t)t * a.width;
     const T* W = static_cast<const T*>(a.w_router);
-    for (int e = warp; e < a.n; e += nw) {
-        const float acc = warp_dot<T>(W + (size_t)e * a.width, h, a.width, lane);
-        if (lane == 0) z[e] = acc;
+    for (int e = warp; e < a.n + (a.w_gate ? 1 : 0); e += nw) {
+        const float acc = warp_dot<T>(e < a.n ? W + (size_t)e * a.width : static_cast<const T*>(a.w_gate), h, a.width, lane);
+        if (lane == 0) {
+            if (e < a.n) z[e] = acc;
+            else a.gate[t] = sigmoid_exact(acc);
+        }
     }
     __syncthreads();
     if (warp != 0) return;

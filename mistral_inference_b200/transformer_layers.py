@@ -1243,16 +1243,14 @@ class GroupedMoe(nn.Module):
     def run(self, hn: torch.Tensor, x32: torch.Tensor, post=None, scale: float = 1.0) -> None:
         assert post is None, "a norm after this feed-forward is not built"
         a = self.a
-        dense, idx, wsel = _h.moe_route(hn, self.router, self.correction, a.groups, a.keep, a.top, score=1, scale=a.router_scale * scale, group_two=True,
-                                        renorm=True)
+        dense, idx, wsel, *gate = _h.moe_route(hn, self.router, self.correction, a.groups, a.keep, a.top, score=1, scale=a.router_scale * scale,
+                                               group_two=True, renorm=True, w_gate=self.shared_gate)
         if hn.shape[0] <= self.sparse_max_tokens:
             _h.moe_sparse(hn, self.w13, self.w2, idx, wsel, a.experts, a.ff, add_to=x32)
         else:
             _h.linear(_h.linear_swiglu(hn, self.w13, rowscale=dense, group=a.ff), self.w2, epi=_h.EPI_RESIDUAL, residual=x32)
         if self.shared is not None:
-            # a router over one output: its sigmoid is the shared expert's gate
-            gate, _, _ = _h.moe_route(hn, self.shared_gate, None, 1, 1, 1, score=1)
-            self.shared.run(hn, x32, None, scale, rowscale=gate)
+            self.shared.run(hn, x32, None, scale, rowscale=gate[0])
 
     def checkpoint_names(self) -> List[str]:
         names = ["router", "correction"] + [f"e{e}.{n}" for e in range(self.a.experts) for n in ("gate", "up", "down")]
