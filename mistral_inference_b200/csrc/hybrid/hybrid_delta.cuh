@@ -149,7 +149,8 @@ struct DeltaConvWalk {
             float acc = w[u][TAPS - 1] * x[u];
 #pragma unroll
             for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(w[u][j], win[j][u], acc);
-            out[u] = silu_exact(acc);
+            // bf16 storage: fast exponential and division (relative error about 1e-6, far below the storage type of the inputs)
+            out[u] = sizeof(T) == 2 ? __fdividef(acc, 1.f + __expf(-acc)) : silu_exact(acc);
 #pragma unroll
             for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][u] = win[j + 1][u];
             if (TAPS > 1) win[TAPS > 1 ? TAPS - 2 : 0][u] = x[u];

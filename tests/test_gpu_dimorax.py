@@ -148,6 +148,36 @@ def test_gelu_feed_forward(dtype, T):
     _close(x32 - x0.to(DEV), 0.7 * O.gated(hs.float(), f32(w), "l0.mlp.", O.gelu_tanh), dtype, f"T={T}")
 
 
+@pytest.mark.parametrize("bias", [False, True])
+@pytest.mark.parametrize("N,K", [(128, 64), (640, 128)])
+def test_prompt_linear_epilogues(monkeypatch, bias, N, K):
+    """Every epilogue behind the prompt GEMM against the Linear kernels that apply it to their accumulators, groups of the row scale that eight
+    columns straddle included, most of its entries 0."""
+    from mistral_inference_b200 import _abi_hybrid as h
+
+    T = 200
+    g = torch.Generator().manual_seed(N)
+    x, w = torch.randn(T, K, generator=g).to(torch.bfloat16).to(DEV), (torch.randn(N, K, generator=g) * 0.2).to(torch.bfloat16).to(DEV)
+    b = torch.randn(N, generator=g).to(torch.bfloat16).to(DEV) if bias else None
+    base = torch.randn(T, N, generator=g).to(DEV)
+    scale = torch.rand(T, 64, generator=g).to(DEV) * (torch.rand(T, 64, generator=g) < 0.3).to(DEV)
+    calls = {"store": lambda: h.linear(x, w, b, n_act=N // 2 + 3), "f32": lambda: h.linear(x, w, b, epi=h.EPI_F32), "capped": lambda: h.linear(x, w, b, epi=h.EPI_F32, limit=2.0),
+             "residual": lambda: h.linear(x, w, b, epi=h.EPI_RESIDUAL, residual=base.clone()),
+             "scaled": lambda: h.linear(x, w, b, epi=h.EPI_RESIDUAL_SCALED, residual=base.clone(), alpha=0.3), "glu": lambda: h.linear(x, w, b, epi=h.EPI_GLU, limit=1.5, alpha=1.7)}
+    if not bias:
+        for group in (5, 10, 12, 64):
+            for name, fn in (("silu", lambda gr: h.linear_swiglu(x, w, scale, gr)), ("gelu", lambda gr: h.linear_swiglu(x, w, scale, gr, gelu=True)),
+                             ("scaled glu", lambda gr: h.linear_glu(x, w, 1.5, 1.7, scale, gr))):
+                if N // 2 <= 64 * group:
+                    calls[f"{name} by {group}"] = lambda fn=fn, group=group: fn(group)
+    for name, fn in calls.items():
+        monkeypatch.setenv("MB200_HYBRID_GEMM", "1")
+        assert h._prompt_gemm_ok(x, T, N, K)
+        got = fn()
+        monkeypatch.setenv("MB200_HYBRID_GEMM", "0")
+        torch.testing.assert_close(got.float(), fn().float(), rtol=2e-2, atol=2e-2, msg=lambda m: f"{name}: {m}")
+
+
 @pytest.mark.parametrize("E,groups,keep,top,scale", [(6, 3, 2, 2, 1.7), (12, 4, 3, 5, 1.0), (8, 8, 3, 2, 0.5), (40, 5, 1, 6, 2.0), (7, 1, 1, 3, 1.0), (1, 1, 1, 1, 3.0)])
 def test_grouped_router(E, groups, keep, top, scale):
     """Choice scores on both sides of zero (an expert outside the kept groups must stay out though its 0 would win), groups of one expert."""
