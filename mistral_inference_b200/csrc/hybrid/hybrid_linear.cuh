@@ -20,7 +20,8 @@
 //
 // Kernels: `linear_tiled_mma` (bf16) and `linear_tiled_fma` (fp32) for prompts, any shape; `linear_skinny` (M <= 8 rows, FMA,
 // one warp per pair of weight rows) and `linear_skinny_mma` (bf16, 3..8 rows, tensor cores) for decode: every weight byte is read
-// once with 16-byte loads; `linear_epilogue_kernel` applies the epilogues to the output of another GEMM (the main library's
+// once with 16-byte loads; `linear_decay_mma` for decays from a low rank; `linear_epilogue8_kernel` (bf16, eight columns per thread) and
+// `linear_epilogue_kernel` apply the epilogues to the output of another GEMM (the main library's
 // tcgen05 GEMM takes the large aligned bf16 Linears of prompts, see _abi_hybrid.linear).
 #pragma once
 #include "hybrid_common.cuh"
