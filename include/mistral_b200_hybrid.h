@@ -13,7 +13,7 @@
 extern "C" {
 #endif
 
-#define MBH_ABI_VERSION 5
+#define MBH_ABI_VERSION 6
 
 int mbh_abi_version(void);
 const char* mbh_last_error(void);
@@ -30,7 +30,7 @@ int mbh_rmsnorm(const void* x32, const void* w, const void* w2, void* y, void* y
  *   1  out32[M, N] += .        in-place add into the fp32 residual stream
  *   2  out[M, N/2]             rows of W interleaved (2c gate, 2c+1 up): g = min(gate, limit), u = clamp(up, -limit, limit),
  *                              out = g * sigmoid(alpha * g) * (u + 1)
- *   3  out32[M, N] = .         fp32 result (logits); with limit > 0: limit * tanh(. / limit)
+ *   3  out32[M, N] = .         fp32 result (logits); with limit > 0: limit * tanh(. / limit); with alpha != 0 times alpha
  *   5  out32[M, N] += alpha * .  the residual add of epilogue 1 with a fixed weight
  * Any M, N, K.  M <= 8 runs the weight-streaming kernel, larger M the tiled one (tensor cores for bf16). */
 int mbh_linear(const void* x, int64_t ldx, const void* w, const void* bias, void* out, void* out32, int64_t M, int64_t N, int64_t K, int epi, int64_t n_act,
@@ -127,9 +127,12 @@ int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_
 /* Router of a mixture of experts, fp32: s = softmax(W_r h) over n outputs (score 0) or sigmoid of each output (score 1), choice = s + correction (null: none); the outputs form
  * `groups` equal groups of neighbours and only those of the `keep` groups with the largest choice (group_two: the largest sum of the two largest
  * choices) stay eligible; the `top` largest eligible choices are taken, weighted by s * scale (renorm: s / (sum of the chosen s + 1e-20) * scale).  w_gate [width], gate fp32 [T] (both or null): gate =
- * sigmoid(w_gate . h), beside the routing.  dense: fp32 [T, n] (0 where not chosen); idx int32 / wsel fp32 [T, top]. */
+ * sigmoid(w_gate . h), beside the routing.  score 2: the largest `top` of z = W_r h are chosen and weighted by the softmax over the chosen z alone
+ * (no groups, correction or renorm).  w_bias [n] or null: added to W_r h first.  always: so many further experts (n, n + 1, ...) go to every token with weight 1, beside the
+ * routing.  dense: fp32 [T, n + always] (0 where not chosen); idx int32 / wsel fp32 [T, top + always]. */
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate, int dt, void* stream);
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate,
+                  const void* w_bias, int64_t always, int dt, void* stream);
 
 /* The chosen experts of few tokens: y32 [T, width] = sum_k wsel[t, k] * expert(idx[t, k])(h[t]); an index >= E is an identity
  * expert (output = h[t]).  w13 [E * 2 * ff, width] (gate and up rows interleaved), w2 [width, E * ff]; act: scratch [T * top, ff].
@@ -151,11 +154,18 @@ int mbh_rows_axpy(void* y32, const void* h, const void* dense, int64_t T, int64_
  * 4 * chunk keys per round, so a short ring read by few tokens is spread over splits = ceil(W / (4 * chunk)) CTAs.
  * weights 0: softmax over the visible keys.  weights 1: every visible key weighs sigmoid(score) and nothing is normalised (bias_tab with
  * n_tab = 1 is then a number per head inside the sigmoid).
- * softcap > 0: score <- softcap * tanh(score / softcap).  sink (fp32 [H] or null): the softmax denominator of head h also holds exp(sink[h]). */
+ * softcap > 0: score <- softcap * tanh(score / softcap).  sink (fp32 [H] or null): the softmax denominator of head h also holds exp(sink[h]).
+ * chunked 1: `window` is the size of chunks counted from position 0, and the token at position p sees keys p - p % window .. p only.
+ * gate (storage type, or null; softmax weights): head h's output is multiplied by sigmoid(gate[t * gate_pitch + h]), or with gate_entry 1 its
+ * entry c by sigmoid(gate[t * gate_pitch + h*e + c]), before it is rounded to the storage type.
+ * maps 2 (differential attention): q is [T, H, 2, d], key rows are [G, 2, d] (ring and own_k), values [G, e]; the head's output is
+ * unit_rms(a_1 - lambda[0] * a_2; norm_eps) * out_scale over its e entries, a_m the softmax average under map m (lambda fp32 on the device; scratch fp32
+ * [T*H*2, splits, 2 + e] also for splits = 1). */
 int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, const void* bias_tab, int64_t n_tab, const void* positions,
                     const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
-                    float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, const void* own_k, const void* own_v,
-                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, int dt, void* stream);
+                    float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, int chunked, const void* own_k, const void* own_v,
+                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, const void* gate, int64_t gate_pitch, int gate_entry,
+                    int64_t maps, const void* lambda, float out_scale, float norm_eps, int dt, void* stream);
 
 /* Linear with interleaved gate/up rows and the clamped gated unit of mbh_linear's epilogue 2; gate and up of column c are multiplied by
  * rowscale[m, c / rs_group] (fp32 [M, rs_pitch]; null: 1) BEFORE the clamps.  mbh_glu_epilogue applies the same to y[M, N] of another GEMM. */
@@ -168,13 +178,14 @@ int mbh_glu_epilogue(const void* y, void* out, int64_t M, int64_t N, float limit
 int mbh_embed_pos(const void* tokens, const void* positions, const void* table, const void* pos_table, float scale, void* x32, int64_t T, int64_t D,
                   int dt, void* stream);
 
-/* Splits qkv[T, H*d + G*d + G*e]; rotates the first rot_dims entries of every q and k head as interleaved pairs (2i, 2i + 1), or as pairs
+/* Splits rows qkv[T, pitch] = q (H*d) | k (G*d) | ..., whose values are the Nv entries at column v_off (v_off = H*d: the unrotated keys are the
+ * values); rotates the first rot_dims entries of every q and k head as interleaved pairs (2i, 2i + 1), or as pairs
  * (i, i + rot_dims / 2) with halves = 1, by the angle positions[t] * freq[i] (freq: float64 [rot_dims / 2]), cos and sin times mag; with unit_norm divides every rotated head by sqrt(mean(x^2) + eps).  Writes
- * q_out [T, H*d]; k_out [T, G*d] and v_out [T, G*e] (both or neither); and, when cache_rows is given, k and v of token t into ring row
+ * q_out [T, H*d]; k_out [T, G*d] and v_out [T, Nv] (both or neither); and, when cache_rows is given, k and v of token t into ring row
  * cache_rows[t] (-1: not cached). */
 int mbh_rot_prep(const void* qkv, const void* freq, const void* positions, const void* cache_rows, void* q_out, void* k_out, void* v_out, void* ring_k,
-                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int halves, float mag, int unit_norm, float eps, int dt,
-                 void* stream);
+                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t Nv, int64_t pitch, int64_t v_off, int64_t rot_dims, int halves, float mag, int unit_norm,
+                 float eps, int dt, void* stream);
 
 /* ring_k[cache_rows[t]] = k[t] (Nk entries), ring_v[cache_rows[t]] = v[t] (Nv entries) for every t with cache_rows[t] >= 0. */
 int mbh_kv_scatter(const void* k, const void* v, const void* cache_rows, void* ring_k, void* ring_v, int64_t T, int64_t Nk, int64_t Nv, int dt,
@@ -217,9 +228,10 @@ int mbh_canon_conv(const void* x32, const void* w, void* state, int64_t state_st
 
 /* acc32[t] += y32[t] / sqrt(mean(y32[t]^2) + eps) * w (fp32 rows [T, D]; w storage type): the norm of a sublayer's output on its way into
  * the residual stream.  With stack: afterwards out32[t] = sum_(j < n - 1) coef[j] * stack[j * stack_stride + t * D ..] + coef[n - 1] *
- * acc32[t], the weighted average over the results of the layers so far (coef [n] storage type; stack_stride in floats). */
+ * acc32[t], the weighted average over the results of the layers so far (coef [n] storage type; stack_stride in floats).  With w_next and y_next (storage
+ * type; no stack): afterwards y_next[t] = acc32[t] / sqrt(mean(acc32[t]^2) + eps) * w_next, what the next sublayer reads. */
 int mbh_rmsnorm_add(const void* y32, const void* w, void* acc32, int64_t T, int64_t D, float eps, const void* stack, int64_t stack_stride,
-                    const void* coef, int64_t n, void* out32, int dt, void* stream);
+                    const void* coef, int64_t n, void* out32, const void* w_next, void* y_next, int dt, void* stream);
 
 /* out32[i] = sum_(j < n) coef[j] * stack[j * stack_stride + i], i < count. */
 int mbh_depth_mix(const void* stack, int64_t stack_stride, const void* coef, int64_t n, void* out32, int64_t count, int dt, void* stream);

@@ -13,7 +13,7 @@ import torch
 from . import _abi, build
 from ._abi import Mb200Error
 
-ABI_VERSION = 5
+ABI_VERSION = 6
 EPI_STORE, EPI_RESIDUAL, EPI_GLU, EPI_F32, EPI_RESIDUAL_SCALED = 0, 1, 2, 3, 5
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 _lib: Optional[ctypes.CDLL] = None
@@ -42,20 +42,20 @@ _SIGNATURES = {
     "mbh_attn_latent": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, I, P, P, P, c_int, P]),
     "mbh_attn_latent_decode": (c_int, [P, P, P, P, P, I, I, I, I, I, F, I, P, I, P, c_int, P]),
     "mbh_latent_vup": (c_int, [P, P, P, I, I, P, I, I, I, I, c_int, P]),
-    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, P, P, c_int, P]),
+    "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, P, P, P, I, c_int, P]),
     "mbh_moe_sparse": (c_int, [P, P, P, P, P, P, P, I, I, I, I, I, c_int, F, F, c_int, c_int, P]),
-    "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, I, c_int, F, P, c_int, P]),
+    "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, c_int, P, P, P, I, c_int, F, P, P, I, c_int, I, P, F, F, c_int, P]),
     "mbh_linear_glu": (c_int, [P, P, P, I, I, I, F, F, P, I, I, c_int, P]),
     "mbh_glu_epilogue": (c_int, [P, P, I, I, F, F, P, I, I, c_int, P]),
     "mbh_embed_pos": (c_int, [P, P, P, P, F, P, I, I, c_int, P]),
-    "mbh_rot_prep": (c_int, [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, F, c_int, P]),
+    "mbh_rot_prep": (c_int, [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, c_int, F, c_int, F, c_int, P]),
     "mbh_kv_scatter": (c_int, [P, P, P, P, P, I, I, I, c_int, P]),
     "mbh_gated_scan": (c_int, [P, P, I, I, P, I, P, P, P, P, P, I, I, I, I, I, c_int, I, I, P, c_int, P]),
     "mbh_hgrn2_gates": (c_int, [P, P, P, I, I, I, c_int, P]),
     "mbh_mlstm_gates": (c_int, [P, P, P, P, P, I, I, P, P, P, I, I, I, I, I, F, F, c_int, P]),
     "mbh_scan_post": (c_int, [P, P, I, P, P, c_int, P, I, I, c_int, P, I, I, I, c_int, F, c_int, P]),
     "mbh_canon_conv": (c_int, [P, P, P, I, I, P, P, P, P, I, I, I, I, c_int, c_int, P]),
-    "mbh_rmsnorm_add": (c_int, [P, P, P, I, I, F, P, I, P, I, P, c_int, P]),
+    "mbh_rmsnorm_add": (c_int, [P, P, P, I, I, F, P, I, P, I, P, P, P, c_int, P]),
     "mbh_depth_mix": (c_int, [P, I, P, I, P, I, c_int, P]),
     "mbh_retention_qab": (c_int, [P, I, P, P, P, P, I, I, I, I, F, c_int, P]),
     "mbh_gla_qab": (c_int, [P, I, P, P, I, I, F, F, c_int, P]),
@@ -158,7 +158,7 @@ def _prompt_gemm_ok(x: torch.Tensor, M: int, N: int, K: int) -> bool:
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, *, epi: int = EPI_STORE, n_act: int = 0,
            residual: Optional[torch.Tensor] = None, limit: float = 0.0, alpha: float = 0.0) -> torch.Tensor:
     """x [M, K] @ w [N, K]^T with the epilogues of include/mistral_b200_hybrid.h.  EPI_RESIDUAL adds into `residual` (fp32, in
-    place; EPI_RESIDUAL_SCALED: times `alpha`) and returns it; EPI_F32 returns fp32 [M, N] (soft-capped at `limit` when positive);
+    place; EPI_RESIDUAL_SCALED: times `alpha`) and returns it; EPI_F32 returns fp32 [M, N] (soft-capped at `limit` when positive, times `alpha` when not 0);
     EPI_GLU returns [M, N/2].  x may be columns of a wider matrix."""
     M, K = x.shape
     N = w.shape[0]
@@ -275,18 +275,21 @@ def linear_swiglu(x: torch.Tensor, w: torch.Tensor, rowscale: Optional[torch.Ten
 
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], groups: int, keep: int, top: int, score: int = 0,
-              scale: float = 1.0, group_two: bool = False, renorm: bool = False, w_gate: Optional[torch.Tensor] = None):
+              scale: float = 1.0, group_two: bool = False, renorm: bool = False, w_gate: Optional[torch.Tensor] = None, w_bias: Optional[torch.Tensor] = None,
+              always: int = 0):
     """(dense fp32 [T, n], idx int32 [T, top], wsel fp32 [T, top]) of the fp32 router; score 0: softmax, 1: sigmoid; the weights are the
     chosen scores times `scale` (renorm: first divided by their sum).  group_two: a group of outputs counts the sum of its two largest
-    choices instead of its largest.  With w_gate ([1, width]) a fourth result: sigmoid(w_gate . h), fp32 [T, 1]."""
+    choices instead of its largest.  With w_gate ([1, width]) a fourth result: sigmoid(w_gate . h), fp32 [T, 1].  score 2: the largest outputs
+    (w_bias [n] added) are chosen and weighted by a softmax over the chosen ones alone.  always: so many more experts, numbered from n, are every
+    token's with weight 1 (dense, idx and wsel are that much wider)."""
     T, D = h.shape
     n = w_router.shape[0]
-    dense = torch.empty(T, n, dtype=torch.float32, device=h.device)
-    idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
-    wsel = torch.empty(T, top, dtype=torch.float32, device=h.device)
+    dense = torch.empty(T, n + always, dtype=torch.float32, device=h.device)
+    idx = torch.empty(T, top + always, dtype=torch.int32, device=h.device)
+    wsel = torch.empty(T, top + always, dtype=torch.float32, device=h.device)
     gate = torch.empty(T, 1, dtype=torch.float32, device=h.device) if w_gate is not None else None
     _check(lib().mbh_moe_route(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(dense), _ptr(idx), _ptr(wsel), T, D, n, groups, keep, top, score,
-                               scale, int(group_two), int(renorm), _ptr(w_gate), _ptr(gate), dt_of(h.dtype), _stream()), "mbh_moe_route")
+                               scale, int(group_two), int(renorm), _ptr(w_gate), _ptr(gate), _ptr(w_bias), always, dt_of(h.dtype), _stream()), "mbh_moe_route")
     return (dense, idx, wsel) if gate is None else (dense, idx, wsel, gate)
 
 
@@ -328,6 +331,7 @@ def latent_prep(y, qnorm, cnorm, freq, positions, cache_rows, ring, q_rank: int,
     return cq, rows
 
 
+DIFF_FLASH_SIZES = {(32, 32), (32, 64), (48, 96), (64, 64), (64, 128), (96, 96), (128, 128)}  # of those with two maps per head
 FLASH_SIZES = {(32, 32), (64, 32), (64, 64), (128, 64), (64, 128), (128, 128), (96, 64), (96, 96), (48, 32), (192, 128)}  # (key, value) sizes of the tensor-core prompt kernel
 _iota: dict = {}
 
@@ -410,17 +414,19 @@ def embed_pos(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor
 
 
 def rot_prep(qkv, freq, positions, cache_rows, ring_k, ring_v, H: int, G: int, d: int, e: int, rot_dims: int, unit_norm: bool, eps: float, own: bool,
-             halves: bool = False, mag: float = 1.0):
-    """(q [T, H*d], k [T, G*d] or None, v [T, G*e] or None): rotated (and unit-normed) queries and keys.  `own`: k and v are
+             halves: bool = False, mag: float = 1.0, v_heads: Optional[int] = None, v_off: Optional[int] = None):
+    """(q [T, H*d], k [T, G*d] or None, v [T, v_heads*e] or None): rotated (and unit-normed) queries and keys of rows q | k | v | ... (v_heads:
+    G unless given; v_off: the values' first column, H*d when they are the unrotated keys).  `own`: k and v are
     returned token-major; `cache_rows` given: they are written into the ring rows as well.  halves: pairs (i, i + rot_dims / 2) instead of
     neighbours; mag: factor on cos and sin.  G = 0: queries only."""
     assert freq.dtype == torch.float64 and freq.numel() == rot_dims // 2
     T = qkv.shape[0]
     q = torch.empty(T, H * d, dtype=qkv.dtype, device=qkv.device)
     k = torch.empty(T, G * d, dtype=qkv.dtype, device=qkv.device) if own else None
-    v = torch.empty(T, G * e, dtype=qkv.dtype, device=qkv.device) if own else None
+    nv = (G if v_heads is None else v_heads) * e
+    v = torch.empty(T, nv, dtype=qkv.dtype, device=qkv.device) if own else None
     _check(lib().mbh_rot_prep(_ptr(qkv), _ptr(freq), _ptr(positions), _ptr(cache_rows), _ptr(q), _ptr(k), _ptr(v), _ptr(ring_k), _ptr(ring_v), T, H, G,
-                              d, e, rot_dims, int(halves), mag, int(unit_norm), eps, dt_of(qkv.dtype), _stream()), "mbh_rot_prep")
+                              d, nv, qkv.shape[1], (H + G) * d if v_off is None else v_off, rot_dims, int(halves), mag, int(unit_norm), eps, dt_of(qkv.dtype), _stream()), "mbh_rot_prep")
     return q, k, v
 
 
@@ -431,17 +437,27 @@ def kv_scatter(k, v, cache_rows, ring_k, ring_v) -> None:
 
 def attn_window(q, cache_k, cache_v, positions, q_start, slots, out, B: int, W: int, H: int, G: int, d: int, e: int, scale: float, window: int,
                 own_k=None, own_v=None, seqpos=None, n_tiles: int = 0, splits: int = 1, chunk: int = 0, head_bias=None,
-                softcap: float = 0.0, sink=None) -> None:
+                softcap: float = 0.0, sink=None, chunked: bool = False, gate=None, gate_entry: bool = False, lam=None, out_scale: float = 1.0,
+                norm_eps: float = 0.0) -> None:
     """`attn_bias` without a bias, with a sliding window (0: none) and, for prompts, this call's own keys and values beside the ring.
     chunk: keys per warp and step of the exact kernel (0: 128), see `window_decode_plan`.  head_bias (fp32 [H]): sigmoid weights instead
     of the softmax, every visible key weighing sigmoid(score + head_bias[h]), not normalised.  softcap > 0: scores softcap * tanh(. / softcap); sink
-    (fp32 [H]): one more term exp(sink[h]) in the softmax denominator."""
-    scratch = torch.empty(q.shape[0] * H * splits * (2 + e), dtype=torch.float32, device=q.device) if splits > 1 and n_tiles == 0 else None
+    (fp32 [H]): one more term exp(sink[h]) in the softmax denominator.  chunked: `window` is the size of chunks.  gate: columns of a matrix
+    [T, .] whose sigmoid multiplies the output, one per head or (gate_entry) one per entry.  lam (fp32 [1]): differential attention, q holds
+    [T, H, 2, d] and keys [., G, 2, d]; out = unit_rms(a_1 - lam a_2; norm_eps) * out_scale per head."""
+    maps = 1 if lam is None else 2
+    flash = n_tiles > 0 and q.dtype == torch.bfloat16 and (d, e) in DIFF_FLASH_SIZES
+    scratch = (torch.empty(q.shape[0] * H * maps * splits * (2 + e), dtype=torch.float32, device=q.device)
+               if (splits > 1 and n_tiles == 0) or (maps > 1 and not flash) else None)
+    gp, g_pitch = _rows(gate) if gate is not None else (None, 0)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], H * e if gate_entry else H))
+    assert lam is None or (lam.dtype == torch.float32 and q.shape[1] == 2 * H * d)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
     assert head_bias is None or (head_bias.dtype == torch.float32 and head_bias.numel() == H)
     _check(lib().mbh_attn_window(_ptr(q), _ptr(cache_k), _ptr(cache_v), _ptr(head_bias), int(head_bias is not None), _ptr(positions), _ptr(q_start),
-                                 _ptr(slots), _ptr(out), q.shape[0], B, W, H, G, d, e, scale, n_tiles, splits, _ptr(scratch), window, _ptr(own_k),
-                                 _ptr(own_v), _ptr(seqpos), chunk, int(head_bias is not None), softcap, _ptr(sink), dt_of(q.dtype), _stream()), "mbh_attn_window")
+                                 _ptr(slots), _ptr(out), q.shape[0], B, W, H, G, d, e, scale, n_tiles, splits, _ptr(scratch), window, int(chunked), _ptr(own_k),
+                                 _ptr(own_v), _ptr(seqpos), chunk, int(head_bias is not None), softcap, _ptr(sink), gp, g_pitch, int(gate_entry), maps, _ptr(lam),
+                                 out_scale, norm_eps, dt_of(q.dtype), _stream()), "mbh_attn_window")
 
 
 def window_decode_plan(T: int, H: int, W: int):
@@ -541,16 +557,19 @@ def canon_conv(x32: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor]
 
 
 def rmsnorm_add(y32: torch.Tensor, w: torch.Tensor, acc32: torch.Tensor, eps: float, stack: Optional[torch.Tensor] = None, n: int = 0,
-                coef: Optional[torch.Tensor] = None, out32: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """acc32 += rms_norm(y32) * w.  With stack (fp32 [>= n, T, D], whose row n - 1 is acc32): out32 = sum_j coef[j] * stack[j]."""
+                coef: Optional[torch.Tensor] = None, out32: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """acc32 += rms_norm(y32) * w.  With stack (fp32 [>= n, T, D], whose row n - 1 is acc32): out32 = sum_j coef[j] * stack[j].  With w_next: returns
+    rms_norm(acc32) * w_next in the weights' dtype instead of acc32."""
     T, D = y32.shape
     assert y32.dtype == torch.float32 and acc32.dtype == torch.float32 and acc32.shape == y32.shape
     if stack is not None:
         assert stack.dtype == torch.float32 and coef.numel() == n and coef.dtype == w.dtype and out32.shape == y32.shape
         assert stack[n - 1].data_ptr() == acc32.data_ptr(), "the last averaged result is the stream that was just updated"
-    _check(lib().mbh_rmsnorm_add(_ptr(y32), _ptr(w), _ptr(acc32), T, D, eps, _ptr(stack), T * D, _ptr(coef), n, _ptr(out32), dt_of(w.dtype), _stream()),
-           "mbh_rmsnorm_add")
-    return acc32
+    y_next = torch.empty(T, D, dtype=w.dtype, device=y32.device) if w_next is not None else None
+    assert w_next is None or (w_next.shape == w.shape and w_next.dtype == w.dtype)
+    _check(lib().mbh_rmsnorm_add(_ptr(y32), _ptr(w), _ptr(acc32), T, D, eps, _ptr(stack), T * D, _ptr(coef), n, _ptr(out32), _ptr(w_next), _ptr(y_next), dt_of(w.dtype),
+                                 _stream()), "mbh_rmsnorm_add")
+    return acc32 if y_next is None else y_next
 
 
 def depth_mix(stack: torch.Tensor, n: int, coef: torch.Tensor, out32: torch.Tensor) -> torch.Tensor:

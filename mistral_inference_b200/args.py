@@ -207,7 +207,9 @@ class RotaryAttentionArgs:
     """Softmax attention with rotary positions on the first `rot_dims` entries of every query and key head (interleaved pairs
     (2i, 2i + 1), angle position * rot_base^(-2i / rot_dims) / rot_factor), optionally a unit RMS norm of every rotated head, grouped
     key/value heads with separate key and value sizes, and optionally a sliding window of `window` positions (the token itself
-    included; None: the whole sequence)."""
+    included; None: the whole sequence) or, with `chunked`, chunks of `window` positions counted from the sequence's start (a token sees
+    the keys of its own chunk).  With `maps` 2 every head has two query/key maps over one set of values and its output is
+    unit_rms(a_1 - lambda a_2) * (1 - diff), lambda learned around `diff`."""
     heads: int
     kv_heads: int
     dim: int
@@ -224,6 +226,12 @@ class RotaryAttentionArgs:
     softcap: float = 0.0       # > 0: score <- softcap * tanh(score / softcap)
     sink: bool = False         # a learned term per head in the softmax denominator
     kv_from: Optional[int] = None  # the layer has queries only and attends to the keys and values that this earlier layer cached
+    chunked: bool = False      # `window` is the size of chunks instead of a sliding window's
+    maps: int = 1              # 2: differential attention
+    diff: float = 0.0
+    values_are_keys: bool = False  # no value projection: the values are the projected keys before rotation and norm
+    out_gate: Optional[str] = None  # sigmoid gate on the output, read from the mixer's input: "head" (one number per head), "entry"
+    out_bias: bool = False     # a bias on the output projection
 
     @classmethod
     def from_dict(cls, d: dict) -> "RotaryAttentionArgs":
@@ -249,6 +257,30 @@ class CappedAttentionArgs(RotaryAttentionArgs):
         a.unit_norm, a.rot_halves, a.qkv_bias, a.sink = False, True, True, True
         a.softcap = float(d.get("softcap") or 0.0)
         a.kv_from = int(d["kv_from"]) if d.get("kv_from") is not None else None
+        return a
+
+
+class DifferentialAttentionArgs(RotaryAttentionArgs):
+    """Differential rotary attention inside chunks: two maps per head over one set of values, biases on all four projections, neighbouring
+    pairs rotated, no unit norm of q and k, a sigmoid gate per head on the output."""
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "DifferentialAttentionArgs":
+        a = super().from_dict(d)
+        a.chunked, a.maps, a.diff = True, 2, float(d["diff"])
+        a.unit_norm, a.qkv_bias, a.out_bias, a.out_gate = False, True, True, "head"
+        return a
+
+
+class KeyValueAttentionArgs(RotaryAttentionArgs):
+    """Rotary attention inside chunks whose values are the projected keys themselves: rotated halves (linearly scaled frequencies), unit
+    norms of the rotated q and k, a sigmoid gate per output entry, no biases."""
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "KeyValueAttentionArgs":
+        a = super().from_dict(d)
+        assert a.vdim == a.dim, "values that are the keys have their size"
+        a.chunked, a.rot_halves, a.values_are_keys, a.out_gate = True, True, True, "entry"
         return a
 
 
@@ -447,6 +479,33 @@ class GroupedMoeArgs:
         return a
 
 
+@dataclass
+class SiluGluArgs:
+    """Dense feed-forward W_down (silu(W_gate h) * (W_up h))."""
+    ff: int
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "SiluGluArgs":
+        return cls(ff=int(d["ff"]))
+
+
+@dataclass
+class ChosenSoftmaxMoeArgs:
+    """Mixture of gated (SiLU) experts with an fp32 router with biases: the `top` largest logits are chosen and weighted by a softmax over
+    the chosen ones alone; an optional shared expert of size `shared_ff` runs for every token."""
+    ff: int
+    experts: int
+    top: int
+    shared_ff: int = 0
+
+    @classmethod
+    def from_dict(cls, d: dict) -> "ChosenSoftmaxMoeArgs":
+        r, sh = d["router"], d.get("shared")
+        a = cls(ff=int(d["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), shared_ff=int(sh["ff"]) if sh else 0)
+        assert 1 <= a.top <= a.experts, "top must be between 1 and the number of experts"
+        return a
+
+
 MLP_ARGS = {"dense": ClampedGluArgs, "moe": MoeFfArgs}
 
 
@@ -454,8 +513,8 @@ MLP_ARGS = {"dense": ClampedGluArgs, "moe": MoeFfArgs}
 class LayerArgs:
     type: str                                             # a key of MIXER_ARGS
     mixer: Union[BiasedAttentionArgs, LightningArgs, LatentAttentionArgs, SideBySideArgs, MlstmArgs, RetentionArgs, GlaArgs, SigmoidAttentionArgs,
-                 CappedAttentionArgs, SinkLatentAttentionArgs, DeltaArgs]
-    mlp: Union[None, ClampedGluArgs, MoeFfArgs, ScaledInputMoeArgs, Relu2MoeArgs, GeluGluArgs, GroupedMoeArgs]
+                 CappedAttentionArgs, SinkLatentAttentionArgs, DeltaArgs, DifferentialAttentionArgs, KeyValueAttentionArgs]
+    mlp: Union[None, ClampedGluArgs, MoeFfArgs, ScaledInputMoeArgs, Relu2MoeArgs, GeluGluArgs, GroupedMoeArgs, SiluGluArgs, ChosenSoftmaxMoeArgs]
 
 
 MIXER_ARGS = {"attention": BiasedAttentionArgs, "lightning": LightningArgs, "latent_attention": LatentAttentionArgs,
@@ -464,8 +523,8 @@ MIXER_ARGS = {"attention": BiasedAttentionArgs, "lightning": LightningArgs, "lat
 
 @dataclass
 class LoopArgs:
-    """Layers start .. stop-1 run `times` times in a row with the same weights (each pass with a cache of its own); before every
-    pass but the first the embedding output is added to the residual stream."""
+    """Layers start .. stop-1 run `times` times in a row with the same weights (each pass with a cache of its own); in a design with
+    `loop_adds_embedding` the embedding output is added to the residual stream before every pass but the first."""
     start: int
     stop: int
     times: int
@@ -477,17 +536,20 @@ class LoopArgs:
 # "pre_norm": False -- the sublayers read the stream itself and norm1 / norm2 act on their OUTPUTS; "canon" -- what a sublayer reads
 # is first replaced by itself plus a causal convolution over time (taps from config "canon"); "depth_average" -- what goes on to the
 # next layer is a learned weighted average of the embedding output and every layer result so far; "tied_head" -- the logits use the
-# embedding table.  DESIGN_MIXER_ARGS: which mixer a type names in a design (default: MIXER_ARGS).
+# embedding table; "loop_adds_embedding": False -- nothing happens between the passes of looped layers.  DESIGN_MIXER_ARGS: which mixer a type names in a design (default: MIXER_ARGS).
 DESIGNS = {
     "Fesenex": {"norm": "rms", "post_norm": False},
     "Taruvik": {"norm": "layer", "post_norm": True},
     "Lotazen": {"norm": "rms_scalar", "post_norm": False, "parallel_block": True, "learned_positions": True},
     "Viladra": {"norm": "rms", "post_norm": True, "pre_norm": False, "canon": True, "depth_average": True, "tied_head": True},
     "Dimorax": {"norm": "rms_around_one", "post_norm": False, "parallel_block": True, "parallel_norms": 2},
+    "Pukarax": {"norm": "rms", "post_norm": True, "tied_head": True, "loop_adds_embedding": False},
 }
-DESIGN_MLP_ARGS = {"Lotazen": {"moe": ScaledInputMoeArgs}, "Viladra": {"moe": Relu2MoeArgs}, "Dimorax": {"dense": GeluGluArgs, "moe": GroupedMoeArgs}}
+DESIGN_MLP_ARGS = {"Lotazen": {"moe": ScaledInputMoeArgs}, "Viladra": {"moe": Relu2MoeArgs}, "Dimorax": {"dense": GeluGluArgs, "moe": GroupedMoeArgs},
+                   "Pukarax": {"dense": SiluGluArgs, "moe": ChosenSoftmaxMoeArgs}}
 DESIGN_MIXER_ARGS = {"Viladra": {"attention": SigmoidAttentionArgs, "retention": RetentionArgs, "gla": GlaArgs},
-                     "Dimorax": {"attention": CappedAttentionArgs, "latent_attention": SinkLatentAttentionArgs, "channel_delta": DeltaArgs}}
+                     "Dimorax": {"attention": CappedAttentionArgs, "latent_attention": SinkLatentAttentionArgs, "channel_delta": DeltaArgs},
+                     "Pukarax": {"attention": DifferentialAttentionArgs, "attention_2": KeyValueAttentionArgs}}
 
 
 @dataclass
@@ -515,6 +577,8 @@ class LayeredArgs:
     canon_taps: int = 0
     depth_average: bool = False      # the next layer reads sum_j dwa[j] X_j over the embedding output and the layer results so far
     tied_head: bool = False          # logits = embed x (the table without its scale)
+    logit_scale: float = 1.0         # logits are multiplied by it
+    loop_adds_embedding: bool = True  # before every pass but the first of looped layers the embedding output is added to the stream
 
     def layer_runs(self) -> List[int]:
         """The layer index of every layer run, in order (a looped layer appears once per pass)."""
@@ -569,4 +633,5 @@ class LayeredArgs:
         return cls(architecture=d["architecture"], vocab=int(d["vocab"]), width=int(d["width"]),
                    embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)), norm_eps=float(d["norm"]["eps"]), layers=layers,
                    loop=loop, max_positions=int(d.get("max_positions", 0)), logit_softcap=float(d.get("logit_softcap") or 0.0),
+                   logit_scale=float(d["logit_scale"]) if d.get("logit_scale") is not None else 1.0,
                    **design)

@@ -118,8 +118,11 @@ template <typename T> static void run_epilogue(const LinearArgs& a, const void* 
 }
 template <typename T> static void run_prep(const AttnPrepArgs& a, int64_t T_, cudaStream_t st) { attn_prep_kernel<T><<<(unsigned)T_, 128, 0, st>>>(a); }
 template <typename T> static void run_attn(const AttnArgs& a, size_t smem, cudaStream_t st) {
-    attn_bias_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
-    if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H);
+    attn_bias_kernel<T><<<dim3((unsigned)(a.T * a.H * a.maps), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
+    if (a.maps > 1) attn_diff_merge_kernel<T><<<(unsigned)(a.T * a.H), AD_THREADS, 0, st>>>(a);
+    else if (a.splits > 1)
+        attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H, a.gate,
+                                                                                                    a.gate_pitch, a.gate_entry);
 }
 template <typename T> static void run_headnorm(const void* o32, const void* w, const void* g, int64_t g_pitch, int64_t g_off, void* y, int64_t T_,
                                                int64_t N, float eps, cudaStream_t st) {
@@ -216,13 +219,14 @@ int mbh_attn_bias(const void* q, const void* cache_k, const void* cache_v, const
                   const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
                   float scale, int64_t n_tiles, int64_t splits, void* scratch, int dt, void* stream) {
     return mbh_attn_window(q, cache_k, cache_v, bias_tab, n_tab, positions, q_start, slots, out, T, B, W, H, G, d, e, scale, n_tiles, splits, scratch,
-                           0, nullptr, nullptr, nullptr, 0, 0, 0.f, nullptr, dt, stream);
+                           0, 0, nullptr, nullptr, nullptr, 0, 0, 0.f, nullptr, nullptr, 0, 0, 1, nullptr, 0.f, 0.f, dt, stream);
 }
 
 int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, const void* bias_tab, int64_t n_tab, const void* positions,
                     const void* q_start, const void* slots, void* out, int64_t T, int64_t B, int64_t W, int64_t H, int64_t G, int64_t d, int64_t e,
-                    float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, const void* own_k, const void* own_v,
-                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, int dt, void* stream) {
+                    float scale, int64_t n_tiles, int64_t splits, void* scratch, int64_t window, int chunked, const void* own_k, const void* own_v,
+                    const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, const void* gate, int64_t gate_pitch, int gate_entry,
+                    int64_t maps, const void* lambda, float out_scale, float norm_eps, int dt, void* stream) {
     if (T == 0) return 0;
     if (weights != 0 && weights != 1) return bad("mbh_attn_window: weights are 0 (softmax) or 1 (sigmoid)");
     if (weights == 1 && (softcap > 0.f || sink)) return bad("mbh_attn_window: a soft cap and sinks belong to the softmax");
@@ -230,17 +234,24 @@ int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, con
     if (e > 32 * AT_MAXR) return bad("mbh_attn_bias: value size above 256");
     if (H % G) return bad("mbh_attn_bias: heads must be a multiple of kv heads");
     if (splits > AT_MAX_SPLITS) return bad("mbh_attn_bias: at most 64 splits");
+    if (chunked && window < 1) return bad("mbh_attn_window: chunks have a size");
+    if (maps != 1 && maps != 2) return bad("mbh_attn_window: one map per head or two");
+    if (maps == 2 && (weights || softcap > 0.f || sink || bias_tab || !lambda))
+        return bad("mbh_attn_window: two maps take lambda and neither a bias, sigmoid weights, a soft cap nor sinks");
+    if (gate && (weights || gate_pitch < (gate_entry ? H * e : H))) return bad("mbh_attn_window: a gate goes with softmax weights; its rows must not overlap");
     if (window < 0 || (!own_k != !own_v) || (own_k && !seqpos)) return bad("mbh_attn_window: window >= 0; own keys, own values and seqpos come together");
     AttnArgs a{q, cache_k, cache_v, (const float*)bias_tab, (int)n_tab, (const int*)positions, (const int*)q_start, (const int*)slots, out,
                (int)T, (int)B, (int)W, (int)H, (int)G, (int)d, (int)e, scale, (int)(splits > 1 && scratch ? splits : 1), (float*)scratch, 0, 0,
-               (int)window, own_k, own_v, (const int*)seqpos, (int)chunk, softcap, (const float*)sink, 0, 0, weights};
+               (int)window, own_k, own_v, (const int*)seqpos, (int)chunk, softcap, (const float*)sink, 0, 0, weights,
+               chunked, gate, (int)gate_pitch, gate_entry, (int)maps, (const float*)lambda, out_scale, norm_eps};
     const size_t smem = sizeof(float) * ((size_t)d + AT_WARPS * AT_CHUNK + AT_WARPS * (2 + 32 * AT_MAXR));
     cudaStream_t st = (cudaStream_t)stream;
     // prompts in bf16: the tensor-core kernel, when the caller counted the 64-query tiles and the sizes are instantiated
-    if (dt == 0 && n_tiles > 0 && launch_attn_flash(a, (int)n_tiles, st)) {
-        cudaError_t ferr = cudaGetLastError();
+    cudaError_t ferr = cudaSuccess;
+    if (dt == 0 && n_tiles > 0 && launch_attn_flash(a, (int)n_tiles, st, ferr)) {
         return ferr ? fail(ferr, "mbh_attn_bias (flash)") : 0;
     }
+    if (maps == 2 && !scratch) return bad("mbh_attn_window: two maps need scratch outside the tensor-core prompt kernel");
     DISPATCH(dt, run_attn<ST>(a, smem, st));
     cudaError_t err = cudaGetLastError();
     return err ? fail(err, "mbh_attn_bias") : 0;
@@ -395,15 +406,18 @@ int mbh_latent_vup(const void* o_lat, const void* w_uv, const void* gate, int64_
 }
 
 int mbh_moe_route(const void* h, const void* w_router, const void* correction, void* dense, void* idx, void* wsel, int64_t T, int64_t width,
-                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate, int dt, void* stream) {
+                  int64_t n, int64_t groups, int64_t keep, int64_t top, int score, float scale, int group_two, int renorm, const void* w_gate, void* gate,
+                  const void* w_bias, int64_t always, int dt, void* stream) {
     if (T == 0) return 0;
     if (!w_gate != !gate) return bad("mbh_moe_route: a gate needs its weight and its output");
     if (groups < 1 || n % groups || keep < 1 || keep > groups) return bad("mbh_moe_route: groups must divide the routed outputs, 1 <= keep <= groups");
     if (top < 1 || top > n / groups * keep) return bad("mbh_moe_route: top exceeds the eligible outputs");
     const size_t smem = sizeof(float) * (size_t)(2 * n + 2 * groups);
     if (smem > 48 * 1024) return bad("mbh_moe_route: too many routed outputs");
-    if (score != 0 && score != 1) return bad("mbh_moe_route: score is 0 (softmax) or 1 (sigmoid)");
-    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, scale, group_two, renorm, w_gate, (float*)gate};
+    if (score < 0 || score > 2) return bad("mbh_moe_route: score is 0 (softmax), 1 (sigmoid) or 2 (softmax over the chosen outputs)");
+    if (score == 2 && (groups != 1 || correction || renorm)) return bad("mbh_moe_route: a softmax over the chosen outputs has no groups, correction or renormalisation");
+    MoeRouteArgs a{h, w_router, correction, (float*)dense, (int*)idx, (float*)wsel, (int)width, (int)n, (int)groups, (int)keep, (int)top, score, w_bias, scale,
+                   group_two, renorm, w_gate, (float*)gate, (int)always};
     cudaStream_t st = (cudaStream_t)stream;
     DISPATCH(dt, moe_route_kernel<ST><<<(unsigned)T, MOE_ROUTE_THREADS, smem, st>>>(a));
     cudaError_t e = cudaGetLastError();
@@ -461,14 +475,16 @@ int mbh_embed_pos(const void* tokens, const void* positions, const void* table, 
 }
 
 int mbh_rot_prep(const void* qkv, const void* freq, const void* positions, const void* cache_rows, void* q_out, void* k_out, void* v_out, void* ring_k,
-                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t e, int64_t rot_dims, int halves, float mag, int unit_norm, float eps, int dt, void* stream) {
+                 void* ring_v, int64_t T, int64_t H, int64_t G, int64_t d, int64_t Nv, int64_t pitch, int64_t v_off, int64_t rot_dims, int halves, float mag, int unit_norm,
+                 float eps, int dt, void* stream) {
     if (T == 0) return 0;
     if (d > 64 * RP_MAXP) return bad("mbh_rot_prep: head size above 256");
     if (rot_dims > d || (rot_dims & 1)) return bad("mbh_rot_prep: rot_dims must be even and at most the head size");
     if (!k_out != !v_out) return bad("mbh_rot_prep: k_out and v_out come together");
+    if (pitch < (H + G) * d || v_off < 0 || v_off + Nv > pitch) return bad("mbh_rot_prep: queries, keys and values lie inside a row");
     if (cache_rows && (!ring_k || !ring_v)) return bad("mbh_rot_prep: ring rows without a ring");
     RotPrepArgs a{qkv, (const double*)freq, (const int*)positions, (const int*)cache_rows, q_out, k_out, v_out, ring_k, ring_v,
-                  (int)H, (int)G, (int)d, (int)e, (int)rot_dims, unit_norm, eps, halves, mag};
+                  (int)H, (int)G, (int)d, (int)Nv, (int)pitch, (int)v_off, (int)rot_dims, unit_norm, eps, halves, mag};
     cudaStream_t st = (cudaStream_t)stream;
     // few tokens (decode): the heads of a token are spread over CTAs; prompts: one CTA per token
     const unsigned hb = T < 512 ? (unsigned)((H + G + 3) / 4) : 1u;
@@ -572,9 +588,17 @@ int mbh_canon_conv(const void* x32, const void* w, void* state, int64_t state_st
 }
 
 int mbh_rmsnorm_add(const void* y32, const void* w, void* acc32, int64_t T, int64_t D, float eps, const void* stack, int64_t stack_stride,
-                    const void* coef, int64_t n, void* out32, int dt, void* stream) {
+                    const void* coef, int64_t n, void* out32, const void* w_next, void* y_next, int dt, void* stream) {
     if (T == 0) return 0;
     if (stack && (!coef || !out32 || n < 1)) return bad("mbh_rmsnorm_add: the depth average needs coefficients and an output");
+    if (!w_next != !y_next || (w_next && stack)) return bad("mbh_rmsnorm_add: the next norm has its weight and its output, and follows no depth average");
+    if (w_next) {
+        NormAddNormArgs f{(const float*)y32, w, (float*)acc32, w_next, y_next, (int)D, eps};
+        const unsigned nt = D > 2048 ? 512u : D > 512 ? 256u : 128u;
+        DISPATCH(dt, rmsnorm_add_norm_kernel<ST><<<(unsigned)T, nt, 0, (cudaStream_t)stream>>>(f));
+        cudaError_t fe = cudaGetLastError();
+        return fe ? fail(fe, "mbh_rmsnorm_add") : 0;
+    }
     NormAddArgs a{(const float*)y32, w, (float*)acc32, (int)D, eps, (const float*)stack, (size_t)stack_stride, coef, (int)n, (float*)out32};
     cudaStream_t st = (cudaStream_t)stream;
     const int threads = D >= 1024 ? 256 : 128;

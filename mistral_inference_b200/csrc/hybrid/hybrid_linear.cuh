@@ -6,7 +6,8 @@
 //                 g = min(gate, limit), u = clamp(up, +-limit), out = g * sigmoid(alpha * g) * (u + 1); with rowscale (as for
 //                 EPI_SWIGLU) gate and up are multiplied by rowscale[m, c / rs_group] BEFORE the clamps: experts whose INPUT is
 //                 scaled by the routing weight, run densely (weight 0 gives exactly 0)
-//   EPI_F32       out32[M, N]  = acc + b        (logits); with limit > 0: limit * tanh((acc + b) / limit), a soft cap
+//   EPI_F32       out32[M, N]  = acc + b        (logits); with limit > 0: limit * tanh((acc + b) / limit), a soft cap; with alpha != 0
+//                 times alpha
 //   EPI_RESIDUAL_SCALED  resid[M, N] += alpha * (acc + b)    (one of several sublayers that are summed with fixed weights)
 //   EPI_SWIGLU    out[M, N/2]: interleaved rows as for EPI_GLU: out = silu(gate) * up * rowscale[m, c / rs_group]
 //                 (rowscale fp32 [M, rs_pitch] or null: a mixture of experts run densely, every expert's hidden units scaled by
@@ -101,6 +102,7 @@ __device__ __forceinline__ void epilogue_pair(const LinearArgs& a, int m, int n,
     default: {
         float* o = a.out32 + (size_t)m * a.N + n;
         if (a.limit > 0.f) { v0 = a.limit * tanhf(v0 / a.limit); v1 = a.limit * tanhf(v1 / a.limit); }
+        if (a.alpha != 0.f) { v0 *= a.alpha; v1 *= a.alpha; }
         o[0] = v0;
         if (has1) o[1] = v1;
         break; }
@@ -495,6 +497,10 @@ __global__ void __launch_bounds__(256) linear_epilogue8_kernel(LinearArgs a, con
         if (a.limit > 0.f) {
 #pragma unroll
             for (int u = 0; u < 8; ++u) v[u] = a.limit * tanhf(v[u] / a.limit);
+        }
+        if (a.alpha != 0.f) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) v[u] *= a.alpha;
         }
         o[0] = make_float4(v[0], v[1], v[2], v[3]);
         o[1] = make_float4(v[4], v[5], v[6], v[7]);

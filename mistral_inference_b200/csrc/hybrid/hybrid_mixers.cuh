@@ -10,7 +10,8 @@
 //   attn_bias         causal softmax attention over the ring with a per-(distance, head) additive bias, GQA, separate
 //                     key and value sizes; one kernel for prompts, prompt portions and decode; optionally a sliding window and
 //                     sigmoid weights instead of the softmax (every visible key weighs sigmoid(score), nothing is normalised), soft-capped
-//                     scores, a learned sink per head in the softmax denominator
+//                     scores, a learned sink per head in the softmax denominator, chunks instead of a window, a sigmoid gate on the output
+//   attn_diff_merge   differential attention: unit_rms(a_1 - lambda a_2) of a head's two softmax maps over the same values
 //   lightning_scan    decayed linear attention S <- a S + k v^T, o = S^T q with the fp32 state carried in the cache
 //   gated_headnorm    y = rms(o over all heads) * w * sigmoid(g)
 #pragma once
@@ -233,7 +234,26 @@ struct AttnArgs {
     int own_k_pitch, own_v_pitch;  // elements per row of own_k / own_v; 0: G*d / G*e
     int sigmoid;            // 1: the weight of a visible key is sigmoid(score), not normalised over the keys (no softmax): partial results
                             // simply add, so the running maximum stays 0 and the sum is never divided by
+    int chunked;            // 1: `window` is the size of chunks counted from position 0; a token sees the keys of its own chunk up to itself
+    const void* gate;       // storage type, or null: the output of token t, head h, entry c is multiplied by sigmoid(gate[t * gate_pitch + h])
+    int gate_pitch;         //   or, with gate_entry, by sigmoid(gate[t * gate_pitch + h*e + c])
+    int gate_entry;
+    int maps = 1;           // 2: differential attention.  q is [T, H, 2, d], key rows are [G, 2, d]; the two maps of a head share its values
+    const float* lambda;    // [1]: out = unit_rms(a_1 - lambda a_2) * out_scale, the root mean square over the head's e entries
+    float out_scale, norm_eps;
 };
+
+// the first key that the token at position p sees
+__device__ __forceinline__ int first_key(const AttnArgs& a, int p) {
+    if (a.window <= 0) return 0;
+    return a.chunked ? p - p % a.window : max(0, p - a.window + 1);
+}
+
+// factor on output entry c of head h
+template <typename T>
+__device__ __forceinline__ float out_gate(const void* gate, int pitch, int entry, int t, int h, int e, int c) {
+    return gate ? sigmoid_exact(to_f(static_cast<const T*>(gate)[(size_t)t * pitch + (entry ? h * e + c : h)])) : 1.f;
+}
 
 // where key / value j of a sequence lives: this call's own rows, or the ring
 template <typename T>
@@ -256,7 +276,8 @@ constexpr int AT_WARPS = 4, AT_CHUNK = 128, AT_MAXR = 8, AT_MAXR_WIDE = 16;  // 
 template <typename T, int MAXR = AT_MAXR>
 __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
     extern __shared__ __align__(16) float sm[];
-    const int t = blockIdx.x / a.H, h = blockIdx.x % a.H, g = h / (a.H / a.G);
+    const int Hm = a.H * a.maps, t = blockIdx.x / Hm, hm = blockIdx.x % Hm, h = hm / a.maps, g = h / (a.H / a.G);
+    const int gk = g * a.maps + hm % a.maps;         // key head: one per map
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* qs = sm;                                  // [d]
     float* sc = sm + a.d + warp * AT_CHUNK;          // [AT_CHUNK] per warp
@@ -264,22 +285,22 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
     int b = 0;
     while (b + 1 < a.B && a.q_start[b + 1] <= t) ++b;
     const int pos = a.positions[t], n = pos + 1;
-    const T* q = static_cast<const T*>(a.q) + ((size_t)t * a.H + h) * a.d;
+    const T* q = static_cast<const T*>(a.q) + (size_t)blockIdx.x * a.d;
     for (int i = threadIdx.x; i < a.d; i += blockDim.x) qs[i] = to_f(q[i]) * a.scale;
     __syncthreads();
     const size_t base = (size_t)a.slots[b] * a.W;
-    const size_t ks = a.k_pitch ? (size_t)a.k_pitch : (size_t)a.G * a.d, vs = a.v_pitch ? (size_t)a.v_pitch : (size_t)a.G * a.e;
+    const size_t ks = a.k_pitch ? (size_t)a.k_pitch : (size_t)a.G * a.maps * a.d, vs = a.v_pitch ? (size_t)a.v_pitch : (size_t)a.G * a.e;
     const int own_from = a.own_k ? a.seqpos[b] : 0x7fffffff;
     const size_t own_row = a.own_k ? (size_t)a.q_start[b] : 0;
-    const size_t oks = a.own_k_pitch ? (size_t)a.own_k_pitch : (size_t)a.G * a.d, ovs = a.own_v_pitch ? (size_t)a.own_v_pitch : (size_t)a.G * a.e;
-    const KeySource<T> Ksrc{static_cast<const T*>(a.cache_k) + base * ks + (size_t)g * a.d,
-                            static_cast<const T*>(a.own_k) + own_row * oks + (size_t)g * a.d, ks, oks, a.W, own_from};
+    const size_t oks = a.own_k_pitch ? (size_t)a.own_k_pitch : (size_t)a.G * a.maps * a.d, ovs = a.own_v_pitch ? (size_t)a.own_v_pitch : (size_t)a.G * a.e;
+    const KeySource<T> Ksrc{static_cast<const T*>(a.cache_k) + base * ks + (size_t)gk * a.d,
+                            static_cast<const T*>(a.own_k) + own_row * oks + (size_t)gk * a.d, ks, oks, a.W, own_from};
     const KeySource<T> Vsrc{static_cast<const T*>(a.cache_v) + base * vs + (size_t)g * a.e,
                             static_cast<const T*>(a.own_v) + own_row * ovs + (size_t)g * a.e, vs, ovs, a.W, own_from};
     constexpr int V = Vec<T>::N;
     const bool vec_ok = (a.d % V == 0) && (ks % V == 0) && (oks % V == 0) && (reinterpret_cast<uintptr_t>(a.cache_k) % 16 == 0)
                         && (!a.own_k || reinterpret_cast<uintptr_t>(a.own_k) % 16 == 0);
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;  // first visible key
+    const int lo = first_key(a, pos);
     float m = a.sigmoid ? 0.f : -INFINITY, l = 0.f, acc[MAXR];
 #pragma unroll
     for (int r = 0; r < MAXR; ++r) acc[r] = 0.f;
@@ -365,7 +386,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
 #pragma unroll
             for (int r = 0; r < MAXR; ++r) o[r] = fmaf(p[2 + r * 32 + lane], f, o[r]);
         }
-        if (a.splits > 1) {
+        if (a.splits > 1 || a.maps > 1) {
             float* part = a.scratch + ((size_t)blockIdx.x * a.splits + blockIdx.y) * (2 + a.e);
             if (lane == 0) { part[0] = M; part[1] = L; }
 #pragma unroll
@@ -376,7 +397,8 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
             if (a.sink) L = sink_denominator(M, L, a.sink[h]);
 #pragma unroll
             for (int r = 0; r < MAXR; ++r)
-                if (r < cpl && lane * cpl + r < a.e) out[lane * cpl + r] = from_f<T>(a.sigmoid ? o[r] : o[r] / L);
+                if (r < cpl && lane * cpl + r < a.e)
+                    out[lane * cpl + r] = from_f<T>((a.sigmoid ? o[r] : o[r] / L) * out_gate<T>(a.gate, a.gate_pitch, a.gate_entry, t, h, a.e, lane * cpl + r));
         }
     }
 }
@@ -387,7 +409,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(AttnArgs a) {
 constexpr int AT_MAX_SPLITS = 64;
 template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restrict__ out, int splits, int e, int sigmoid = 0, const float* __restrict__ sink = nullptr,
-                                  int H = 1) {
+                                  int H = 1, const void* gate = nullptr, int gate_pitch = 0, int gate_entry = 0) {
     __shared__ float f[AT_MAX_SPLITS];
     __shared__ float red[32];
     const float* part = scratch + (size_t)blockIdx.x * splits * (2 + e);
@@ -415,7 +437,59 @@ __global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restri
         o3 = fmaf(col[(size_t)(s + 3) * (2 + e)], f[s + 3], o3);
     }
     for (; s < splits; ++s) o0 = fmaf(col[(size_t)s * (2 + e)], f[s], o0);
-    out[(size_t)blockIdx.x * e + c] = from_f<T>(((o0 + o1) + (o2 + o3)) / L);
+    out[(size_t)blockIdx.x * e + c] = from_f<T>(((o0 + o1) + (o2 + o3)) / L * out_gate<T>(gate, gate_pitch, gate_entry, blockIdx.x / H, blockIdx.x % H, e, c));
+}
+
+// Differential attention: the two maps' partial results of attn_bias_kernel (scratch [T*H, 2, splits, 2 + e]) become
+// unit_rms(a_1 - lambda a_2) * out_scale * gate.  grid (token * head), a thread per ceil(e / 256) value columns
+constexpr int AD_THREADS = 128, AD_COLS = 2;  // e <= 256
+template <typename T>
+__global__ void __launch_bounds__(AD_THREADS) attn_diff_merge_kernel(AttnArgs a) {
+    __shared__ float f[2][AT_MAX_SPLITS];
+    __shared__ float den[2];
+    __shared__ float red[32];
+    const int t = blockIdx.x / a.H, h = blockIdx.x % a.H, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pitch = 2 + a.e;
+    const float* part = a.scratch + (size_t)blockIdx.x * 2 * a.splits * pitch;
+    if (warp < 2) {  // a warp per map: the splits' weights exp(m_s - M) and the denominator
+        const float* p = part + (size_t)warp * a.splits * pitch;
+        float M = -INFINITY, L = 0.f;
+        for (int s = lane; s < a.splits; s += 32) M = fmaxf(M, p[(size_t)s * pitch]);
+        M = warp_max(M);
+        for (int s = lane; s < a.splits; s += 32) {
+            const float m = p[(size_t)s * pitch], w = (m == -INFINITY) ? 0.f : expf(m - M);
+            f[warp][s] = w;
+            L += w * p[(size_t)s * pitch + 1];
+        }
+        L = warp_sum(L);
+        if (lane == 0) den[warp] = L;
+    }
+    __syncthreads();
+    const float l1 = den[0], l2 = den[1], lam = *a.lambda;
+    float v[AD_COLS], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < AD_COLS; ++k) {
+        const int c = k * AD_THREADS + threadIdx.x;
+        v[k] = 0.f;
+        if (c < a.e) {
+            const float* p1 = part + 2 + c;
+            const float* p2 = p1 + (size_t)a.splits * pitch;
+            float a1 = 0.f, a2 = 0.f;
+            for (int s = 0; s < a.splits; ++s) {
+                a1 = fmaf(p1[(size_t)s * pitch], f[0][s], a1);
+                a2 = fmaf(p2[(size_t)s * pitch], f[1][s], a2);
+            }
+            v[k] = a1 / l1 - lam * (a2 / l2);
+            ss = fmaf(v[k], v[k], ss);
+        }
+    }
+    ss = block_sum(ss, red);
+    const float inv = a.out_scale / sqrtf(ss / (float)a.e + a.norm_eps);
+    T* out = static_cast<T*>(a.out) + (size_t)blockIdx.x * a.e;
+#pragma unroll
+    for (int k = 0; k < AD_COLS; ++k) {
+        const int c = k * AD_THREADS + threadIdx.x;
+        if (c < a.e) out[c] = from_f<T>(v[k] * inv * out_gate<T>(a.gate, a.gate_pitch, a.gate_entry, t, h, a.e, c));
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ lightning attention

@@ -4,6 +4,7 @@
 //                     experts: output = input); choice = s + correction; the n outputs form `groups` equal groups of
 //                     neighbours, a group scores its largest choice (or the sum of its two largest), only the best `keep` groups stay eligible; the `top`
 //                     largest eligible choices are taken, each weighted by its s, optionally divided by the sum of the chosen ones' s.  Ties go to the lower index.
+//                     Another form chooses by z (+ a bias) itself and weights by the softmax over the chosen z alone.
 //                     One more output may gate a shared expert (its sigmoid, not routed).  Writes the dense weights [T, n] (0 where not chosen) and the chosen (index, weight) pairs [T, top].
 //   moe_gateup_sparse / moe_down_sparse   few tokens (decode): one CTA column per (token, chosen expert) streams only that
 //                     expert's rows: act = silu(W_gate h) * (W_up h), then y = sum_k w_k W_down[e_k] act_k + (identity weights) h
@@ -21,16 +22,19 @@ struct MoeRouteArgs {
     const void* h;            // [T, width]
     const void* w_router;     // [n, width]
     const void* correction;   // [n] or null
-    float* dense;             // [T, n]
-    int* idx;                 // [T, top]
-    float* wsel;              // [T, top]
+    float* dense;             // [T, n + always]
+    int* idx;                 // [T, top + always]
+    float* wsel;              // [T, top + always]
     int width, n, groups, keep, top;
-    int score;                // 0: softmax over the outputs; 1: sigmoid of each output
+    int score;                // 0: softmax over the outputs; 1: sigmoid of each output; 2: the outputs themselves decide (one group), the
+                              // weights are the softmax over the chosen ones alone
+    const void* w_bias;       // [n] or null: added to the outputs before anything else
     float scale;              // the weights (dense and wsel) are the chosen scores times this
     int group_two;            // a group scores the sum of its two largest choices instead of its largest
     int renorm;               // the weights are divided by (the sum of the chosen scores + 1e-20)
     const void* w_gate;       // [width] or null: one more output whose sigmoid gates a shared expert ...
     float* gate;              // [T] ... goes here; it takes no part in the routing
+    int always;               // experts n .. n + always - 1 take no part in the routing either: every token has them, with weight 1
 };
 
 // (value, index) argmax over a warp; the lower index wins a tie
@@ -78,13 +82,43 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
     for (int e = warp; e < a.n + (a.w_gate ? 1 : 0); e += nw) {
         const float acc = warp_dot<T>(e < a.n ? W + (size_t)e * a.width : static_cast<const T*>(a.w_gate), h, a.width, lane);
         if (lane == 0) {
-            if (e < a.n) z[e] = acc;
+            if (e < a.n) z[e] = acc + (a.w_bias ? to_f(static_cast<const T*>(a.w_bias)[e]) : 0.f);
             else a.gate[t] = sigmoid_exact(acc);
         }
     }
     __syncthreads();
     if (warp != 0) return;
+    const int dn = a.n + a.always, tk = a.top + a.always;
+    for (int s = lane; s < a.always; s += 32) {
+        a.dense[(size_t)t * dn + a.n + s] = 1.f;
+        a.idx[(size_t)t * tk + a.top + s] = a.n + s;
+        a.wsel[(size_t)t * tk + a.top + s] = 1.f;
+    }
     float sum = 1.f;
+    if (a.score == 2) {
+        float mx = -INFINITY;  // the largest output is always chosen: it keeps the exponentials of the chosen ones in range
+        for (int e = lane; e < a.n; e += 32) { mx = fmaxf(mx, z[e]); ch[e] = z[e]; a.dense[(size_t)t * dn + e] = 0.f; }
+        mx = warp_max(mx);
+        __syncwarp();
+        float den = 0.f;
+        for (int k = 0; k < a.top; ++k) {
+            float v = -INFINITY; int ei = 0x7fffffff;
+            for (int e = lane; e < a.n; e += 32)
+                if (ch[e] > v) { v = ch[e]; ei = e; }
+            warp_argmax(v, ei);
+            if (ei == 0x7fffffff) ei = 0;
+            den += expf(v - mx);
+            if (lane == 0) { a.idx[(size_t)t * tk + k] = ei; ch[ei] = -INFINITY; }
+            __syncwarp();
+        }
+        for (int k = lane; k < a.top; k += 32) {
+            const int ei = a.idx[(size_t)t * tk + k];
+            const float w = expf(z[ei] - mx) / den * a.scale;
+            a.wsel[(size_t)t * tk + k] = w;
+            a.dense[(size_t)t * dn + ei] = w;
+        }
+        return;
+    }
     if (a.score == 1) {
         for (int e = lane; e < a.n; e += 32) z[e] = sigmoid_exact(z[e]);
     } else {
@@ -100,7 +134,7 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
         const float s = z[e] / sum;
         z[e] = s;
         ch[e] = s + (corr ? to_f(corr[e]) : 0.f);
-        a.dense[(size_t)t * a.n + e] = 0.f;
+        a.dense[(size_t)t * dn + e] = 0.f;
     }
     __syncwarp();
     if (a.groups > 1 && a.keep < a.groups) {
@@ -138,19 +172,19 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(MoeRouteAr
         const float w = (v == -INFINITY) ? 0.f : z[ei];
         total += w;
         if (lane == 0) {
-            a.idx[(size_t)t * a.top + k] = ei;
-            a.wsel[(size_t)t * a.top + k] = w * a.scale;
-            if (v != -INFINITY) { a.dense[(size_t)t * a.n + ei] = w * a.scale; ch[ei] = -INFINITY; }
+            a.idx[(size_t)t * tk + k] = ei;
+            a.wsel[(size_t)t * tk + k] = w * a.scale;
+            if (v != -INFINITY) { a.dense[(size_t)t * dn + ei] = w * a.scale; ch[ei] = -INFINITY; }
         }
         __syncwarp();
     }
     if (a.renorm) {  // every value was written by this warp; the barrier above ordered the writes
         const float den = total + 1e-20f;
         for (int k = lane; k < a.top; k += 32) {
-            const int ei = a.idx[(size_t)t * a.top + k];
+            const int ei = a.idx[(size_t)t * tk + k];
             const float w = z[ei] / den * a.scale;
-            a.wsel[(size_t)t * a.top + k] = w;
-            a.dense[(size_t)t * a.n + ei] = w;
+            a.wsel[(size_t)t * tk + k] = w;
+            a.dense[(size_t)t * dn + ei] = w;
         }
     }
 }

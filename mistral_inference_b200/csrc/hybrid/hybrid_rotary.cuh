@@ -1,9 +1,9 @@
 // Rotary attention inputs and the embedding with learned positions.
 //
 //   embed_pos        x[t] = E[token[t]] * scale + P[position[t]]            -> fp32 residual stream
-//   rot_prep         splits qkv[T, H*d + G*d + G*e]; rotates the first rot_dims entries of every q and k head as interleaved pairs
+//   rot_prep         splits qkv[T, H*d | G*d | Nv | ...] (the values may be the unrotated keys themselves); rotates the first rot_dims entries of every q and k head as interleaved pairs
 //                    (2i, 2i + 1), or as pairs (i, i + rot_dims / 2), by position * freq[i], cos and sin times `mag`; optionally divides each head by its root mean square (no weight);
-//                    writes q[T, H*d], k[T, G*d], v[T, G*e] token-major and, for tokens with a ring row, k and v into the ring
+//                    writes q[T, H*d], k[T, G*d], v[T, Nv] token-major and, for tokens with a ring row, k and v into the ring
 //   kv_scatter       k[T, G*d], v[T, G*e] -> ring rows cache_rows[t] (after a prompt's attention has read the old ring)
 //
 // The angle is position * freq[i] in double precision (frequencies come from the host in float64): an fp32 product at
@@ -23,14 +23,14 @@ __global__ void embed_pos_kernel(const int64_t* __restrict__ tok, const int* __r
 }
 
 struct RotPrepArgs {
-    const void* qkv;        // [T, H*d + G*d + G*e]
+    const void* qkv;        // [T, pitch] = q (H*d) | k (G*d) | ...; values (Nv entries) at column v_off
     const double* freq;     // [rot_dims / 2] angle per position step of pair i
     const int* positions;   // [T]
     const int* cache_rows;  // [T] ring row or -1; null: nothing goes to the ring in this call
     void* q_out;            // [T, H*d]
-    void* k_out; void* v_out;   // [T, G*d] / [T, G*e], or null
-    void* ring_k; void* ring_v; // [rows, G, d] / [rows, G, e]
-    int H, G, d, e, rot_dims;
+    void* k_out; void* v_out;   // [T, G*d] / [T, Nv], or null
+    void* ring_k; void* ring_v; // [rows, G*d] / [rows, Nv]
+    int H, G, d, Nv, pitch, v_off, rot_dims;
     int unit_norm;          // divide every rotated q and k head by sqrt(mean(x^2) + eps)
     float eps;
     int halves;             // pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)
@@ -43,8 +43,8 @@ constexpr int RP_MAXP = 4;  // pairs per lane: head sizes up to 256
 template <typename T>
 __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    const int Nq = a.H * a.d, Nk = a.G * a.d, Nv = a.G * a.e;
-    const T* row = static_cast<const T*>(a.qkv) + (size_t)t * (Nq + Nk + Nv);
+    const int Nq = a.H * a.d, Nk = a.G * a.d, Nv = a.Nv;
+    const T* row = static_cast<const T*>(a.qkv) + (size_t)t * a.pitch;
     const int pos = a.positions[t];
     const int crow = a.cache_rows ? a.cache_rows[t] : -1;
     const int half = a.d >> 1;  // pairs; an odd last entry passes unchanged
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
             if (dst1) dst1[a.d - 1] = from_f<T>(last * inv);
         }
     }
-    const T* vsrc = row + Nq + Nk;
+    const T* vsrc = row + a.v_off;
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < Nv; i += gridDim.y * blockDim.x) {
         if (a.v_out) static_cast<T*>(a.v_out)[(size_t)t * Nv + i] = vsrc[i];
         if (crow >= 0) static_cast<T*>(a.ring_v)[(size_t)crow * Nv + i] = vsrc[i];

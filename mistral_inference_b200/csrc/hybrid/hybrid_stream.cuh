@@ -8,6 +8,7 @@
 //   rmsnorm_add       acc[t] += y[t] / sqrt(mean(y[t]^2) + eps) * w: the norm of a sublayer's OUTPUT, added to the stream in fp32;
 //                     optionally followed by the depth average: out[t] = sum_j c[j] * X_j[t] over the layer results X_0 .. X_(n-1)
 //                     kept one after the other (X_(n-1) is acc itself, just updated)
+//   rmsnorm_add_norm  rmsnorm_add, then the RMS norm of the updated stream that the next sublayer reads, in the storage type
 //   depth_mix         the depth average alone
 #pragma once
 #include "hybrid_common.cuh"
@@ -179,6 +180,80 @@ __global__ void rmsnorm_add_kernel(NormAddArgs a) {
             a.out[row + i] = fmaf(to_f(cf[a.n - 1]), v, m);
         }
     }
+}
+
+struct NormAddNormArgs {
+    const float* y;        // [T, D] sublayer output
+    const void* w;         // [D] its norm's weight
+    float* acc;            // [T, D] the stream, updated in place
+    const void* w_next;    // [D] weight of the norm that reads the stream next
+    void* y_next;          // [T, D]
+    int D;
+    float eps;
+};
+
+// One row per CTA.  The quads of the row that a thread owns stay in its registers (up to KEEP of them) from the first pass to the last
+template <typename T>
+__global__ void __launch_bounds__(512) rmsnorm_add_norm_kernel(NormAddNormArgs a) {
+    __shared__ float red[32];
+    constexpr int KEEP = 4;
+    const size_t row = (size_t)blockIdx.x * a.D;
+    const float* y = a.y + row;
+    float* acc = a.acc + row;
+    T* o = static_cast<T*>(a.y_next) + row;
+    const T* w = static_cast<const T*>(a.w);
+    const T* wn = static_cast<const T*>(a.w_next);
+    const bool quads = a.D % 4 == 0 && a.D <= KEEP * 4 * (int)blockDim.x &&
+                       (reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.acc) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.w_next) |
+                        reinterpret_cast<uintptr_t>(a.y_next)) % 16 == 0;
+    float ss = 0.f;
+    if (quads) {
+        float v[KEEP][4], x[KEEP][4];
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (k * blockDim.x + threadIdx.x) * 4;
+            if (i < a.D) { load4(y + i, v[k]); load4(acc + i, x[k]); }
+            else
+#pragma unroll
+                for (int u = 0; u < 4; ++u) v[k][u] = x[k][u] = 0.f;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) ss = fmaf(v[k][u], v[k][u], ss);
+        }
+        const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+        ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (k * blockDim.x + threadIdx.x) * 4;
+            if (i >= a.D) continue;
+            float wv[4];
+            load4(w + i, wv);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) { x[k][u] += v[k][u] * inv * wv[u]; ss = fmaf(x[k][u], x[k][u], ss); }
+            store4<float>(acc + i, x[k]);
+        }
+        const float inv2 = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) {
+            const int i = (k * blockDim.x + threadIdx.x) * 4;
+            if (i >= a.D) continue;
+            float wv[4];
+            load4(wn + i, wv);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) wv[u] *= x[k][u] * inv2;
+            store4<T>(o + i, wv);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < a.D; i += blockDim.x) ss = fmaf(y[i], y[i], ss);
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+    ss = 0.f;
+    for (int i = threadIdx.x; i < a.D; i += blockDim.x) {
+        const float v = acc[i] + y[i] * inv * to_f(w[i]);
+        acc[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float inv2 = 1.f / sqrtf(block_sum(ss, red) / (float)a.D + a.eps);
+    for (int i = threadIdx.x; i < a.D; i += blockDim.x) o[i] = from_f<T>(acc[i] * inv2 * to_f(wn[i]));  // the thread's own writes
 }
 
 // out[i] = sum_j coef[j] * stack[j * stride + i], i < count

@@ -1,7 +1,7 @@
 """Layered decoder: a model given as a list of layers, each with its own kind of token mixer (softmax attention with a
 distance bias, lightning attention with a recurrent state, latent attention, ...) and an optional feed-forward (gated, or a
 mixture of experts), optionally with a span of layers that runs several times (args.LayeredArgs; architectures "Fesenex",
-"Taruvik", "Lotazen", "Viladra", "Dimorax").  It plugs into the same places as `Transformer`: `from_folder`, `forward(input_ids, seqlens, cache)` over ragged
+"Taruvik", "Lotazen", "Viladra", "Dimorax", "Pukarax").  It plugs into the same places as `Transformer`: `from_folder`, `forward(input_ids, seqlens, cache)` over ragged
 batches, `BufferCache` (per-layer rings and states, `make_cache`), `forward_logprobs` / `next_token_logits` for `generate()`.
 
 On disk: config.json + model.safetensors with tensors `embed`, `l<i>.norm1|norm2` (and `norm1b|norm2b` with norms after the
@@ -49,6 +49,8 @@ class LayeredTransformer(nn.Module):
                                        pre_norm=args.pre_norm, canon_taps=args.canon_taps if args.canon else 0,
                                        depth_results=li + 2 if args.depth_average else 0))
         self.layers = nn.ModuleList(blocks)
+        # norms handed on from layer to layer, unless something is added to the stream in between
+        self._chained = all(b.chains() for b in blocks) and (args.loop is None or not args.loop_adds_embedding)
         self.pos = nn.Parameter(torch.empty(args.max_positions, args.width), requires_grad=False) if args.learned_positions else None
         self.final_norm = Norm(args.width, args.norm_eps, args.norm)
         # a tied head is the embedding table itself (without the embedding's scale): no parameter of its own
@@ -115,12 +117,16 @@ class LayeredTransformer(nn.Module):
             return self._run_layers_averaged(x, md, cache, ctx)
         lp = self.args.loop
         first_pass = True
+        hn: Optional[torch.Tensor] = None  # the stream behind the norm that the next layer reads it through, when the layer before left it
         for r, i in enumerate(self.runs):
-            if lp is not None and i == lp.start:
+            if lp is not None and i == lp.start and self.args.loop_adds_embedding:
                 if not first_pass:  # every pass but the first starts from the stream plus the embedding output
                     _h.embed_add(input_ids, self.embed, self.args.embedding_scale, x)
                 first_pass = False
-            self.layers[i](x, cache.get_view(r, md[r]), ctx)
+            if self._chained:
+                hn = self.layers[i].chained(x, cache.get_view(r, md[r]), ctx, hn, self.layers[self.runs[r + 1]].norm1 if r + 1 < len(self.runs) else None)
+            else:
+                self.layers[i](x, cache.get_view(r, md[r]), ctx)
             if self._tap is not None:
                 self._tap(r, x)
         return x
@@ -144,7 +150,8 @@ class LayeredTransformer(nn.Module):
 
     def logits_of(self, x32: torch.Tensor) -> torch.Tensor:
         """Final norm + head, fp32 [rows, vocab]."""
-        return _h.linear(self.final_norm(x32), self.head if self.head is not None else self.embed, epi=_h.EPI_F32, limit=self.args.logit_softcap)
+        return _h.linear(self.final_norm(x32), self.head if self.head is not None else self.embed, epi=_h.EPI_F32, limit=self.args.logit_softcap,
+                         alpha=self.args.logit_scale if self.args.logit_scale != 1.0 else 0.0)
 
     def _graph_decode_ok(self, seqlens: List[int], cache: Optional[BufferCache]) -> bool:
         if cache is None or self._tap is not None or os.environ.get("MB200_DECODE_GRAPH", "1") == "0":

@@ -31,6 +31,7 @@ register("Taruvik", _layered)
 register("Lotazen", _layered)
 register("Viladra", _layered)
 register("Dimorax", _layered)
+register("Pukarax", _layered)
 register("transformer", _reference_format)
 
 

@@ -191,9 +191,9 @@ import math  # noqa: E402
 from typing import Dict  # noqa: E402
 
 from . import _abi_hybrid as _h  # noqa: E402
-from .args import (BiasedAttentionArgs, CappedAttentionArgs, ClampedGluArgs, DeltaArgs, GeluGluArgs, GlaArgs, GroupedMoeArgs, Hgrn2Args, LatentAttentionArgs, LightningArgs, MlstmArgs, MoeFfArgs,  # noqa: E402
-                   Relu2FfArgs, Relu2MoeArgs, RetentionArgs, RotaryAttentionArgs, ScaledInputMoeArgs, SideBySideArgs, SigmoidAttentionArgs,
-                   SinkLatentAttentionArgs)
+from .args import (BiasedAttentionArgs, CappedAttentionArgs, ChosenSoftmaxMoeArgs, ClampedGluArgs, DeltaArgs, DifferentialAttentionArgs, GeluGluArgs, GlaArgs, GroupedMoeArgs,  # noqa: E402
+                   Hgrn2Args, KeyValueAttentionArgs, LatentAttentionArgs, LightningArgs, MlstmArgs, MoeFfArgs, Relu2FfArgs, Relu2MoeArgs, RetentionArgs,
+                   RotaryAttentionArgs, ScaledInputMoeArgs, SideBySideArgs, SigmoidAttentionArgs, SiluGluArgs, SinkLatentAttentionArgs)
 from .rope import scaled_frequencies  # noqa: E402
 from .cache import LayerCacheSpec  # noqa: E402
 
@@ -207,7 +207,8 @@ class Norm(nn.Module):
     same kernel serves it) or "layer" (mean removed; weight and bias).  Reads the fp32 residual stream (or an fp32 sublayer output)
     and either returns the normed rows in the model dtype or adds them, in fp32, to `add_to`.  `mix` = (stack, n, coef, out), with an
     rms norm that adds: the depth average out = sum_j coef[j] * stack[j] over the n layer results so far follows in the same kernel
-    (stack[n - 1] is `add_to`)."""
+    (stack[n - 1] is `add_to`).  `then`, with an rms norm that adds: the norm of the updated stream that the next sublayer reads follows in the same
+    kernel and is returned."""
 
     def __init__(self, width: int, eps: float, kind: str):
         super().__init__()
@@ -216,7 +217,10 @@ class Norm(nn.Module):
         self.weight = nn.Parameter(torch.empty(width), requires_grad=False)
         self.bias = nn.Parameter(torch.empty(width), requires_grad=False) if kind == "layer" else None
 
-    def forward(self, x32: torch.Tensor, add_to: Optional[torch.Tensor] = None, mix: Optional[tuple] = None) -> torch.Tensor:
+    def forward(self, x32: torch.Tensor, add_to: Optional[torch.Tensor] = None, mix: Optional[tuple] = None, then: Optional["Norm"] = None) -> torch.Tensor:
+        if then is not None:
+            assert add_to is not None and mix is None and self.kind == then.kind == "rms" and self.eps == then.eps
+            return _h.rmsnorm_add(x32, self.weight, add_to, self.eps, w_next=then.weight)
         if self.kind == "layer":
             assert mix is None, "a depth average after a layer norm is not built"
             return _h.layernorm(x32, self.weight, self.bias, self.eps, add_to=add_to)
@@ -565,30 +569,43 @@ class MoeFeedForward(nn.Module):
 
 class RotaryWindowAttention(nn.Module):
     """Causal softmax attention with rotary positions, grouped key/value heads and, as the arguments say (args.RotaryAttentionArgs), a unit RMS
-    norm of the rotated q and k heads, a sliding window, biases on q, k and v, soft-capped scores, a sink per head in the softmax denominator.
+    norm of the rotated q and k heads, a sliding window or chunks, biases on q, k and v (and the output), soft-capped scores, a sink per head in the
+    softmax denominator, two maps per head (differential attention), values that are the unrotated keys, a sigmoid gate on the output.
     The ring holds min(window, longest sequence) rows per sequence.  A decode step writes its key and value into the ring, then attends over
     it; a prompt (portion) attends over the OLD ring plus its own keys and values, and writes the ring afterwards, so a prompt longer than
     the ring still finds every key inside each token's window.  With `kv_from` the layer has queries only and attends over the ring of an
-    earlier layer (whole sequence, no window), which that layer has just brought up to date.  Packed weights: wqkv = q ++ k ++ v rows."""
+    earlier layer (whole sequence, no window), which that layer has just brought up to date.  Two maps per head are kept as heads of their own in q
+    and k ([map 1, map 2] head by head), so rotation and ring know nothing of them; attention, difference, norm and gate are one call.  Packed
+    weights: wqkv = q ++ k ++ v ++ g rows (padded when there is a gate)."""
 
     def __init__(self, width: int, a: RotaryAttentionArgs, eps: float):
         super().__init__()
         self.a, self.eps = a, eps
         own_kv = a.kv_from is None
-        self.nq, self.nk, self.nv = a.heads * a.dim, a.kv_heads * a.dim * own_kv, a.kv_heads * a.vdim * own_kv
-        n = self.nq + self.nk + self.nv
+        assert a.maps == 1 or not (a.sink or a.softcap > 0.0), "soft-capped scores and sinks under two maps are not built"
+        assert not a.values_are_keys or (a.maps == 1 and own_kv and a.vdim == a.dim), "values that are the keys: one map, a key projection of their size"
+        assert a.out_gate in (None, "head", "entry"), a.out_gate
+        self.nq, self.nk = a.heads * a.maps * a.dim, a.kv_heads * a.maps * a.dim * own_kv
+        self.nv = a.kv_heads * a.vdim * (own_kv and not a.values_are_keys)
+        self.ng = {None: 0, "head": a.heads, "entry": a.heads * a.vdim}[a.out_gate]
+        self.g_off = self.nq + self.nk + self.nv
+        n = padded_rows(self.g_off + self.ng) if self.ng else self.g_off
         self.wqkv = nn.Parameter(torch.empty(n, width), requires_grad=False)
         self.bqkv = nn.Parameter(torch.empty(n), requires_grad=False) if a.qkv_bias else None
         self.sink = nn.Parameter(torch.empty(a.heads), requires_grad=False) if a.sink else None
+        self.lambdas = nn.Parameter(torch.empty(4, a.dim), requires_grad=False) if a.maps == 2 else None  # rows lq1, lk1, lq2, lk2
         self.wo = nn.Parameter(torch.empty(width, a.heads * a.vdim), requires_grad=False)
+        self.bo = nn.Parameter(torch.empty(width), requires_grad=False) if a.out_bias else None
         self._freq: Optional[torch.Tensor] = None
         self._sink32: Optional[torch.Tensor] = None
+        self._lam32: Optional[torch.Tensor] = None
         self._mag = 1.0
 
     def cache_spec(self) -> LayerCacheSpec:
+        # chunks need no more rows than a window of their size: a token's chunk is among the last `window` positions
         if self.a.kv_from is not None:
             return LayerCacheSpec(kind="shared", source=self.a.kv_from)
-        return LayerCacheSpec(kind="ring", n_kv_heads=self.a.kv_heads, k_dim=self.a.dim, v_dim=self.a.vdim, window=self.a.window)
+        return LayerCacheSpec(kind="ring", n_kv_heads=self.a.kv_heads, k_dim=self.a.maps * self.a.dim, v_dim=self.a.vdim, window=self.a.window)
 
     def frequencies(self) -> torch.Tensor:
         """float64 [rot_dims / 2]: rot_base^(-2i / rot_dims) under the frequency scaling, evaluated on the host in double precision."""
@@ -603,6 +620,13 @@ class RotaryWindowAttention(nn.Module):
             self._sink32 = self.sink.detach().float().contiguous()
         return self._sink32
 
+    def difference_weight(self) -> Optional[torch.Tensor]:
+        """fp32 [1]: lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, evaluated once in double precision."""
+        if self.lambdas is not None and (self._lam32 is None or self._lam32.device != self.lambdas.device):
+            t = self.lambdas.detach().double().cpu()
+            self._lam32 = (torch.exp((t[0] * t[1]).sum()) - torch.exp((t[2] * t[3]).sum()) + self.a.diff).float().reshape(1).to(self.lambdas.device)
+        return self._lam32
+
     def run(self, hn: torch.Tensor, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], post: Optional[Norm] = None,
             scale: float = 1.0) -> None:
         a, md = self.a, view.metadata
@@ -612,34 +636,48 @@ class RotaryWindowAttention(nn.Module):
         window, own_kv, freq, sink = a.window or 0, a.kv_from is None, self.frequencies(), self.sinks()
         own = md.prefill and own_kv
         rows = None if (own or not own_kv) else md.cache_rows
-        q, k, v = _h.rot_prep(qkv, freq, md.positions, rows, view.cache_k if rows is not None else None, view.cache_v if rows is not None else None, a.heads,
-                              a.kv_heads if own_kv else 0, a.dim, a.vdim, a.rot_dims, a.unit_norm, self.eps, own=own, halves=a.rot_halves, mag=self._mag)
+        q, k, v = _h.rot_prep(qkv, freq, md.positions, rows, view.cache_k if rows is not None else None, view.cache_v if rows is not None else None,
+                              a.heads * a.maps, a.kv_heads * a.maps if own_kv else 0, a.dim, a.vdim, a.rot_dims, a.unit_norm, self.eps, own=own,
+                              halves=a.rot_halves, mag=self._mag, v_heads=a.kv_heads if own_kv else 0, v_off=self.nq if a.values_are_keys else None)
         if md.prefill:
             plan = dict(n_tiles=query_tiles(md))
         else:
-            splits, chunk = _h.window_decode_plan(T, a.heads, W)
+            splits, chunk = _h.window_decode_plan(T, a.heads * a.maps, W)
             plan = dict(splits=splits, chunk=chunk)
+        if self.ng:
+            plan.update(gate=qkv[:, self.g_off: self.g_off + self.ng], gate_entry=a.out_gate == "entry")
+        if a.maps == 2:
+            plan.update(lam=self.difference_weight(), out_scale=1.0 - a.diff, norm_eps=self.eps)
         _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, window,
-                       own_k=k, own_v=v, seqpos=md.seqpos if own else None, softcap=a.softcap, sink=sink, **plan)
+                       own_k=k, own_v=v, seqpos=md.seqpos if own else None, softcap=a.softcap, sink=sink, chunked=a.chunked, **plan)
         if own:
             _h.kv_scatter(k, v, md.cache_rows, view.cache_k, view.cache_v)
-        project_out(out, self.wo, x32, post, scale)
+        project_out(out, self.wo, x32, post, scale, bias=self.bo)
 
     def checkpoint_names(self) -> List[str]:
-        proj = ["q", "k", "v"] if self.a.kv_from is None else ["q"]
-        return proj + ([n + ".b" for n in proj] if self.a.qkv_bias else []) + (["sink"] if self.a.sink else []) + ["o"]
+        a = self.a
+        proj = ["q"] if a.kv_from is not None else ["q", "k"] if a.values_are_keys else ["q", "k", "v"]
+        return (proj + ([n + ".b" for n in proj] if a.qkv_bias else []) + (["sink"] if a.sink else []) + (["lq1", "lk1", "lq2", "lk2"] if a.maps == 2 else [])
+                + (["g"] if self.ng else []) + ["o"] + (["o.b"] if a.out_bias else []))
 
     def assign(self, name: str, put) -> bool:
         if name not in self.checkpoint_names():
             return False
-        spans = {"q": (0, self.nq), "k": (self.nq, self.nq + self.nk), "v": (self.nq + self.nk, self.nq + self.nk + self.nv)}
+        spans = {"q": (0, self.nq), "k": (self.nq, self.nq + self.nk), "v": (self.nq + self.nk, self.g_off), "g": (self.g_off, self.g_off + self.ng)}
         if name in spans:
+            self.wqkv[self.g_off + self.ng:].zero_()
             put(self.wqkv[spans[name][0]: spans[name][1]])
+        elif name == "o.b":
+            put(self.bo)
         elif name.endswith(".b"):
+            self.bqkv[self.g_off:].zero_()  # the gate has no bias
             put(self.bqkv[spans[name[:-2]][0]: spans[name[:-2]][1]])
         elif name == "sink":
             put(self.sink)
             self._sink32 = None
+        elif name[0] == "l":
+            put(self.lambdas[("lq1", "lk1", "lq2", "lk2").index(name)])
+            self._lam32 = None
         else:
             put(self.wo)
         return True
@@ -1223,6 +1261,11 @@ class GeluGlu(GatedFeedForward):
         super().__init__(width, a.ff, gelu=True)
 
 
+class SiluGlu(GatedFeedForward):
+    def __init__(self, width: int, a: SiluGluArgs):
+        super().__init__(width, a.ff, gelu=False)
+
+
 class GroupedMoe(nn.Module):
     """Mixture of SiLU-gated experts with an fp32 sigmoid router limited to groups and renormalised weights (args.GroupedMoeArgs), plus a shared
     expert times sigmoid(W_sg h).  Packed like MoeFeedForward.  Few tokens (decode) stream the chosen experts only; prompts run all experts as
@@ -1274,6 +1317,60 @@ class GroupedMoe(nn.Module):
         return True
 
 
+class ChosenSoftmaxMoe(nn.Module):
+    """Mixture of SiLU-gated experts with an fp32 router with biases whose weights are the softmax over the chosen logits (args.ChosenSoftmaxMoeArgs),
+    plus a shared expert for every token.  Packed like MoeFeedForward.  A shared expert whose size is a multiple of the experts' is packed behind
+    them as that many more experts (a gated unit is a sum over its hidden units), which the router gives every token with weight 1: one pair of
+    Linears for a prompt, one pair of kernels for a decode step.  Another size runs beside them and adds into the same fp32 sum."""
+
+    def __init__(self, width: int, a: ChosenSoftmaxMoeArgs):
+        super().__init__()
+        self.a, self.width = a, width
+        self.always = a.shared_ff // a.ff if a.shared_ff % a.ff == 0 else 0
+        self.total = a.experts + self.always
+        self.router = nn.Parameter(torch.empty(a.experts, width), requires_grad=False)
+        self.router_bias = nn.Parameter(torch.empty(a.experts), requires_grad=False)
+        self.w13 = nn.Parameter(torch.empty(self.total * 2 * a.ff, width), requires_grad=False)
+        self.w2 = nn.Parameter(torch.empty(width, self.total * a.ff), requires_grad=False)
+        self.shared = GatedFeedForward(width, a.shared_ff, gelu=False) if a.shared_ff and not self.always else None
+        self.sparse_max_tokens = MOE_SPARSE_MAX_TOKENS
+
+    def run(self, hn: torch.Tensor, x32: torch.Tensor, post=None) -> None:
+        a = self.a
+        dense, idx, wsel = _h.moe_route(hn, self.router, None, 1, 1, a.top, score=2, w_bias=self.router_bias, always=self.always)
+        if hn.shape[0] <= self.sparse_max_tokens:
+            y32 = _h.moe_sparse(hn, self.w13, self.w2, idx, wsel, self.total, a.ff, add_to=x32 if post is None else None)
+        elif post is None:
+            y32 = _h.linear(_h.linear_swiglu(hn, self.w13, rowscale=dense, group=a.ff), self.w2, epi=_h.EPI_RESIDUAL, residual=x32)
+        else:
+            y32 = _h.linear(_h.linear_swiglu(hn, self.w13, rowscale=dense, group=a.ff), self.w2, epi=_h.EPI_F32)
+        if self.shared is not None:
+            self.shared.run(hn, y32)
+        if post is not None:
+            post(y32, add_to=x32)
+
+    def checkpoint_names(self) -> List[str]:
+        names = ["router", "router.b"] + [f"e{e}.{n}" for e in range(self.a.experts) for n in ("gate", "up", "down")]
+        return names + (["shared." + n for n in ("gate", "up", "down")] if self.a.shared_ff else [])
+
+    def assign(self, name: str, put) -> bool:
+        a = self.a
+        head, _, part = name.partition(".")
+        if name == "router":
+            put(self.router)
+        elif name == "router.b":
+            put(self.router_bias)
+        elif head == "shared" and self.shared is not None:
+            return self.shared.assign(part, put)
+        elif part in ("gate", "up", "down") and ((head == "shared" and self.always) or (head[:1] == "e" and head[1:].isdigit() and int(head[1:]) < a.experts)):
+            lo, n = (a.experts, self.always) if head == "shared" else (int(head[1:]), 1)
+            lo, n = lo * a.ff, n * a.ff
+            put(self.w2[:, lo: lo + n] if part == "down" else self.w13.view(-1, 2, self.width)[lo: lo + n, int(part == "up")])
+        else:
+            return False
+        return True
+
+
 class CanonConv(nn.Module):
     """What a sublayer reads, replaced by itself plus a causal convolution over time on every channel: h_t = x_t + sum_j w[:, j]
     x_(t - taps + 1 + j), zeros before the sequence's start.  Reads the fp32 stream, writes the model dtype.  The last taps - 1 inputs
@@ -1294,20 +1391,25 @@ MIXERS = {"attention": BiasedAttention, "lightning": LightningMixer, "latent_att
           "mlstm": MlstmMixer, "mlstm_2": MlstmMixer}
 # mixers that a design names with a type another design uses differently are found by their argument class first
 MIXERS_BY_ARGS = {RetentionArgs: RetentionMixer, GlaArgs: GlaMixer, SigmoidAttentionArgs: SigmoidWindowAttention,
-                  CappedAttentionArgs: RotaryWindowAttention, SinkLatentAttentionArgs: LatentAttention, DeltaArgs: DeltaMixer}
+                  CappedAttentionArgs: RotaryWindowAttention, SinkLatentAttentionArgs: LatentAttention, DeltaArgs: DeltaMixer,
+                  DifferentialAttentionArgs: RotaryWindowAttention, KeyValueAttentionArgs: RotaryWindowAttention}
 FEED_FORWARDS = {ClampedGluArgs: ClampedGLU, MoeFfArgs: MoeFeedForward, ScaledInputMoeArgs: ScaledInputMoe, Relu2MoeArgs: Relu2Moe,
-                 GeluGluArgs: GeluGlu, GroupedMoeArgs: GroupedMoe}
+                 GeluGluArgs: GeluGlu, GroupedMoeArgs: GroupedMoe, SiluGluArgs: SiluGlu, ChosenSoftmaxMoeArgs: ChosenSoftmaxMoe}
 
 
 class _PostNorm:
-    """The norm after a sublayer as the sublayers call it, post(fp32 rows, add_to=stream), with the depth average that follows the
-    layer's last sublayer."""
+    """The norm after a sublayer as the sublayers call it, post(fp32 rows, add_to=stream), with what follows in the same kernel: the depth
+    average after the layer's last sublayer, or the norm that the next sublayer reads the stream through (its rows are left in `normed`)."""
 
-    def __init__(self, norm: Norm, mix: Optional[tuple]):
-        self.norm, self.mix = norm, mix
+    def __init__(self, norm: Norm, mix: Optional[tuple], then: Optional[Norm] = None):
+        self.norm, self.mix, self.then = norm, mix, then
+        self.normed: Optional[torch.Tensor] = None
 
     def __call__(self, y32: torch.Tensor, add_to: torch.Tensor) -> torch.Tensor:
-        return self.norm(y32, add_to=add_to, mix=self.mix)
+        if self.then is None:
+            return self.norm(y32, add_to=add_to, mix=self.mix)
+        self.normed = self.norm(y32, add_to=add_to, then=self.then)
+        return add_to
 
 
 class LayeredBlock(nn.Module):
@@ -1347,6 +1449,21 @@ class LayeredBlock(nn.Module):
         if self.canon1 is None or self.canon1.taps < 2:
             return ()
         return (1 + int(self.canon2 is not None), self.canon1.taps - 1, self.width)
+
+    def chains(self) -> bool:
+        """True for a block whose norms can be handed on from sublayer to sublayer (`chained`)."""
+        return self.norm1b is not None and self.norm1.kind == "rms"
+
+    def chained(self, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], hn: Optional[torch.Tensor], then: Optional[Norm]) -> Optional[torch.Tensor]:
+        """`forward` with each norm before a sublayer computed by the kernel of the norm that was last added: hn = norm1(x32), when the block before
+        has left it; `then` = the norm through which the stream is read next, whose rows are returned."""
+        first = _PostNorm(self.norm1b, None, self.norm2 if self.mlp is not None else then)
+        self.mix.run(self.norm1(x32) if hn is None else hn, x32, view, ctx, first)
+        if self.mlp is None:
+            return first.normed
+        second = _PostNorm(self.norm2b, None, then)
+        self.mlp.run(first.normed, x32, second)
+        return second.normed
 
     def forward(self, x32: torch.Tensor, view: CacheView, ctx: Dict[str, torch.Tensor], mix: Optional[tuple] = None) -> torch.Tensor:
         if not self.pre_norm:
