@@ -267,7 +267,7 @@ class DifferentialAttentionArgs(RotaryAttentionArgs):
     @classmethod
     def from_dict(cls, d: dict) -> "DifferentialAttentionArgs":
         a = super().from_dict(d)
-        a.chunked, a.maps, a.diff = True, 2, float(d["diff"])
+        a.chunked, a.maps, a.diff = a.window is not None, 2, float(d["diff"])
         a.unit_norm, a.qkv_bias, a.out_bias, a.out_gate = False, True, True, "head"
         return a
 
@@ -280,7 +280,7 @@ class KeyValueAttentionArgs(RotaryAttentionArgs):
     def from_dict(cls, d: dict) -> "KeyValueAttentionArgs":
         a = super().from_dict(d)
         assert a.vdim == a.dim, "values that are the keys have their size"
-        a.chunked, a.rot_halves, a.values_are_keys, a.out_gate = True, True, True, "entry"
+        a.chunked, a.rot_halves, a.values_are_keys, a.out_gate = a.window is not None, True, True, "entry"
         return a
 
 
