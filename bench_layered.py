@@ -1,4 +1,4 @@
-"""`bench.py --design fesenex|taruvik|lotazen|viladra|dimorax`: prefill and decode throughput of the layered decoder at layer sizes of real models (random
+"""`bench.py --design fesenex|taruvik|lotazen|viladra|dimorax|pukarax`: prefill and decode throughput of the layered decoder at layer sizes of real models (random
 weights), beside the dense `Transformer` of equal width / heads / feed-forward size / depth / vocabulary, plus the time of each
 hybrid kernel at those shapes against its roofline (bf16 tensor peak or HBM copy bandwidth from MEASURED_PEAKS.json).
 For `taruvik` (latent attention, mixture of experts) the neighbour is the `Transformer` with a mixture of experts of equal
@@ -6,7 +6,8 @@ width / heads / experts / depth; for `lotazen` (rotary window attention beside a
 input) it is the Fesenex design at equal width / heads / depth, and every new kernel is timed next to the like kernel at the same shape;
 for `viladra` (convolution on the stream, norms after the sublayers with a depth average, retention, gated linear attention,
 sigmoid-weight window attention, ungated experts) the neighbour is the Lotazen design at equal width / heads / experts / depth; for
-`dimorax` (gated delta rule, soft-capped attention with sinks, windowed latent attention, group-limited experts) too.  Timed with CUDA events after warm-up; the prompt batch and the weights exceed L2 at the larger size, and L2 is flushed between
+`dimorax` (gated delta rule, soft-capped attention with sinks, windowed latent attention, group-limited experts) too; for `pukarax` (differential attention and attention
+with keys as values, both inside chunks, softmax over the chosen experts) it is the Dimorax design with rotary attention in every layer.  Timed with CUDA events after warm-up; the prompt batch and the weights exceed L2 at the larger size, and L2 is flushed between
 timed kernel launches.  Prints one JSON line."""
 import json
 import math
@@ -953,7 +954,195 @@ def run_dimorax(a, peaks: dict) -> dict:
     return res
 
 
+# ----------------------------------------------------------------------------------------------- Pukarax
+PUKARAX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, map_dim=64, chunk_a=2048, chunk_b=1024, experts=16, top=2, ff=1408, shared_ff=2816, dense_ff=5632, vocab=32768,
+                  order="kdkd", loop=(1, 3, 2)),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, map_dim=64, chunk_a=4096, chunk_b=2048, experts=8, top=2, ff=3584, shared_ff=7168, dense_ff=14336, vocab=32768,
+                  order="dkd", loop=None),
+}
+
+
+def pukarax_config(s: dict) -> dict:
+    d = s["dim"]
+    mixers = {
+        "d": {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["map_dim"], "vdim": d, "scale": s["map_dim"] ** -0.5, "diff": 0.5,
+                                             "mask": {"size": s["chunk_a"]}, "rot": {"base": 500000.0, "dims": s["map_dim"]}}},
+        "k": {"type": "attention_2", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": s["chunk_b"]},
+                                               "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 8.0}}}},
+    }
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}, "shared": {"ff": s["shared_ff"]}}
+    cfg = {"architecture": "Pukarax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 4.0}, "logit_scale": 0.5,
+           "layers": [{**mixers[c], "mlp": moe if i % 3 != 2 else {"kind": "dense", "ff": s["dense_ff"]}} for i, c in enumerate(s["order"])]}
+    if s["loop"]:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), s["loop"]))
+    return cfg
+
+
+def build_pukarax(s: dict, dev):
+    from mistral_inference_b200.args import LayeredArgs
+    from mistral_inference_b200.layered import LayeredTransformer
+
+    m = LayeredTransformer.empty(LayeredArgs.from_dict(pukarax_config(s)), dev, torch.bfloat16)
+    g = torch.Generator(device=dev).manual_seed(0)
+    with torch.no_grad():
+        for n, p in m.named_parameters():
+            if "norm" in n:
+                p.fill_(1.0)
+            elif p.dim() >= 2:
+                p.copy_(torch.randn(p.shape, generator=g, device=dev, dtype=torch.float32) / math.sqrt(p.shape[-1]))
+            else:
+                p.copy_(torch.randn(p.shape, generator=g, device=dev, dtype=torch.float32) * 0.1)
+    return m.eval()
+
+
+def dimorax_like_pukarax(s: dict) -> dict:
+    """The closest existing design at equal size: rotary softmax attention (over the whole sequence, one map of the value size per head) in every
+    layer run, silu-gated experts with a shared expert and dense layers of the same sizes in the same places."""
+    n = len(s["order"]) + ((s["loop"][1] - s["loop"][0]) * (s["loop"][2] - 1) if s["loop"] else 0)
+    return dict(width=s["width"], heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"], lat_heads=1, lat_dim=64, rot_dim=32, kv_rank=64, window=64, rec_heads=1, rec_kv_heads=1,
+                taps=1, rank=1, experts=s["experts"], top=s["top"], groups=1, keep=1, ff=s["ff"], shared_ff=s["shared_ff"], dense_ff=s["dense_ff"], vocab=s["vocab"], order="a" * n)
+
+
+def pukarax_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
+    """Every kernel the design added or extended, alone at this size, each next to the like kernel of an existing design at the same shape."""
+    from mistral_inference_b200 import _abi_hybrid as h
+    from mistral_inference_b200.cache import BufferCache, LayerCacheSpec
+    from mistral_inference_b200.rope import scaled_frequencies
+
+    bf = torch.bfloat16
+    W, H, G, d, dm, E, ff, sff, top, ca, cb = (s[k] for k in ("width", "heads", "kv_heads", "dim", "map_dim", "experts", "ff", "shared_ff", "top", "chunk_a", "chunk_b"))
+    flush = torch.zeros(160 << 20, dtype=torch.float32, device=dev)
+    rows = {}
+
+    def rec(name, fn, flops=0.0, bytes_=0.0, note=None, n=(3, 8)):
+        ms = _time(fn, n[0], n[1], flush)
+        r = {"ms": round(ms, 4)}
+        if flops:
+            r["tflops"] = round(flops / ms / 1e9, 2)
+            r["of_bf16_peak"] = round(flops / ms / 1e9 / peaks["bf16_tflops"], 4)
+        if bytes_:
+            r["gb_s"] = round(bytes_ / ms / 1e6, 1)
+            r["of_hbm_peak"] = round(bytes_ / ms / 1e6 / peaks["hbm_gbs"], 3)
+        if note:
+            r["note"] = note
+        rows[name] = r
+
+    def rnd(*shape, scale=1.0):
+        return (torch.randn(*shape, device=dev) * scale).to(bf)
+
+    B, nt = 8, (T + 63) // 64
+    # ---- norms
+    x32, y32, nw = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev), torch.ones(W, device=dev).to(bf)
+    rec("rmsnorm_add_norm prompt (add, then the next norm)", lambda: h.rmsnorm_add(y32, nw, x32, 1e-5, w_next=nw), bytes_=T * W * 14.0)
+    rec("like: rmsnorm_add prompt", lambda: h.rmsnorm_add(y32, nw, x32, 1e-5), bytes_=T * W * 12.0)
+    yB, xB = y32[:B].contiguous(), x32[:B].contiguous()
+    rec(f"rmsnorm_add_norm decode B={B}", lambda: h.rmsnorm_add(yB, nw, xB, 1e-5, w_next=nw), bytes_=B * W * 14.0, note="latency")
+    rec(f"like: rmsnorm_add, then rmsnorm, decode B={B}", lambda: (h.rmsnorm_add(yB, nw, xB, 1e-5), h.rmsnorm(xB, nw, 1e-5)), bytes_=B * W * 18.0, note="latency, two launches")
+    # ---- rotation
+    specs = {"diff": LayerCacheSpec(kind="ring", n_kv_heads=G, k_dim=2 * dm, v_dim=d, window=ca), "keyval": LayerCacheSpec(kind="ring", n_kv_heads=G, k_dim=d, v_dim=d, window=cb),
+             "like": LayerCacheSpec(kind="ring", n_kv_heads=G, k_dim=d, v_dim=d, window=ca), "like_b": LayerCacheSpec(kind="ring", n_kv_heads=G, k_dim=d, v_dim=d, window=cb)}
+    ring = BufferCache(4, B, ctx + 8, 0, 0, None, layer_specs=list(specs.values())).to(dev, bf)
+    for i in range(4):
+        ring.cache_k[i].normal_()
+        ring.cache_v[i].normal_()
+    mds = dict(zip(specs, ring.get_input_metadata([T])))
+    md = mds["like"]
+    fm, fd = scaled_frequencies(dm, 5e5, None)[0].to(dev), scaled_frequencies(d, 1e4, None)[0].to(dev)
+    qkv_d, qkv_k, qkv = rnd(T, (2 * H + 2 * G) * dm + G * d + 64), rnd(T, (H + G) * d + H * d), rnd(T, (H + 2 * G) * d)
+    rot_d = lambda: h.rot_prep(qkv_d, fm, md.positions, None, None, None, 2 * H, 2 * G, dm, d, dm, False, 0.0, own=True, v_heads=G)  # noqa: E731
+    rot_k = lambda: h.rot_prep(qkv_k, fd, md.positions, None, None, None, H, G, d, d, d, True, 1e-5, own=True, halves=True, v_off=H * d)  # noqa: E731
+    rec("rot_prep prompt (two maps, neighbours)", rot_d, bytes_=T * 4.0 * ((2 * H + 2 * G) * dm + G * d))
+    rec("rot_prep prompt (keys as values, halves, unit norm)", rot_k, bytes_=T * 2.0 * ((H + G) * d + (H + 2 * G) * d))
+    rec("like: rot_prep prompt (neighbours, unit norm)", lambda: h.rot_prep(qkv, fd, md.positions, None, None, None, H, G, d, d, d, True, 1e-5, own=True), bytes_=4.0 * qkv.numel())
+    # ---- attention
+    qd, kd, vd = rot_d()
+    qk, kk, vk = rot_k()
+    ql, kl, vl = h.rot_prep(qkv, fd, md.positions, None, None, None, H, G, d, d, d, True, 1e-5, own=True)
+    o, lam, gates = torch.empty(T, H * d, device=dev, dtype=bf), torch.full((1,), 0.5, device=dev), rnd(T, H * d)
+    diff = dict(lam=lam, out_scale=0.5, norm_eps=1e-5)
+    pairs_chunk = lambda c: sum(p % c + 1 for p in range(T))  # noqa: E731
+    pairs_win = lambda c: sum(min(p + 1, c) for p in range(T))  # noqa: E731
+
+    def prompt(name, q, k, v, key, dk, c, flops, **kw):
+        m_, i = mds[key], list(specs).index(key)
+        rec(name, lambda: h.attn_window(q, ring.cache_k[i], ring.cache_v[i], m_.positions, m_.q_start, m_.slots, o, 1, m_.window, H, G, dk, d, 0.09, c, own_k=k, own_v=v,
+                                        seqpos=m_.seqpos, n_tiles=nt, **kw), flops=flops, n=(2, 5))
+
+    prompt(f"differential attention prompt, chunks of {ca}, head gate", qd, kd, vd, "diff", dm, ca, 4.0 * H * (dm + d) * pairs_chunk(ca), chunked=True, gate=gates[:, :H], **diff)
+    prompt(f"like: softmax attention prompt, window {ca}", ql, kl, vl, "like", d, ca, 4.0 * H * d * pairs_win(ca))
+    prompt(f"attention prompt, chunks of {cb}, entry gate", qk, kk, vk, "keyval", d, cb, 4.0 * H * d * pairs_chunk(cb), chunked=True, gate=gates, gate_entry=True)
+    prompt(f"like: softmax attention prompt, window {cb}", ql, kl, vl, "like_b", d, cb, 4.0 * H * d * pairs_win(cb))
+    at = ca - 1 if ca - 1 <= ctx else ctx  # the last token of a chunk: it sees the whole chunk
+    ring.reset(); ring.init_kvseqlens(B); ring.update_seqlens([at] * B)
+    md2 = dict(zip(specs, ring.get_input_metadata([1] * B)))
+    oB = torch.empty(B, H * d, device=dev, dtype=bf)
+
+    def decode(name, q, key, dk, c, **kw):
+        m_, i, qB = md2[key], list(specs).index(key), q[:B].contiguous()
+        sp, ch = h.window_decode_plan(B, H * (2 if "lam" in kw else 1), m_.window)
+        rec(f"{name} B={B}", lambda: h.attn_window(qB, ring.cache_k[i], ring.cache_v[i], m_.positions, m_.q_start, m_.slots, oB, B, m_.window, H, G, dk, d, 0.09, c, splits=sp, chunk=ch, **kw),
+            bytes_=B * min(at + 1, c) * G * 2.0 * (d + dk * (2 if "lam" in kw else 1)))
+
+    decode(f"differential attention decode, chunks of {ca}, head gate", qd, "diff", dm, ca, chunked=True, gate=gates[:B, :H], **diff)
+    decode(f"like: softmax attention decode, window {ca}", ql, "like", d, ca)
+    decode(f"attention decode, chunks of {cb}, entry gate", qk, "keyval", d, cb, chunked=True, gate=gates[:B], gate_entry=True)
+    decode(f"like: softmax attention decode, window {cb}", ql, "like_b", d, cb)
+    # ---- feed-forward
+    x = rnd(T, W)
+    al = sff // ff
+    w13, w2, wr, wb = rnd((E + al) * 2 * ff, W, scale=0.02), rnd(W, (E + al) * ff, scale=0.02), rnd(E, W, scale=4 / math.sqrt(W)), torch.zeros(E, device=dev).to(bf)
+    route = lambda t: h.moe_route(t, wr, None, 1, 1, top, score=2, w_bias=wb, always=al)  # noqa: E731
+    rec("moe_route prompt (softmax over the chosen)", lambda: route(x), bytes_=T * W * 2.0)
+    rec("like: moe_route prompt (sigmoid)", lambda: h.moe_route(x, wr, None, 1, 1, top, score=1), bytes_=T * W * 2.0)
+    dense, idx, wsel = route(x)
+    l13, l2, s13, s2 = w13[: E * 2 * ff], w2[:, : E * ff].contiguous(), w13[E * 2 * ff:], w2[:, E * ff:].contiguous()
+    d_like, i_like, w_like = h.moe_route(x, wr, None, 1, 1, top, score=1)
+    ones = torch.ones(T, 1, device=dev)
+    fl = 6.0 * T * (top * ff + sff) * W
+
+    def like_prompt():
+        y = h.linear(h.linear_swiglu(x, l13, rowscale=d_like, group=ff), l2, epi=h.EPI_F32)
+        return h.linear(h.linear_swiglu(x, s13, rowscale=ones, group=sff), s2, epi=h.EPI_RESIDUAL, residual=y)
+
+    rec("experts prompt (shared expert among them)", lambda: h.linear(h.linear_swiglu(x, w13, rowscale=dense, group=ff), w2, epi=h.EPI_F32), flops=fl, n=(2, 5),
+        note=f"useful FLOPs (top {top} of {E} + shared); the kernels compute all {E} experts")
+    rec("like: experts prompt, shared expert of its own", like_prompt, flops=fl, n=(2, 5))
+    for M in (1, B):
+        xs, ii, ww, il, wl = (t[:M].contiguous() for t in (x, idx, wsel, i_like, w_like))
+
+        def like_decode():
+            y = h.moe_sparse(xs, l13, l2, il, wl, E, ff)
+            return h.linear(h.linear_swiglu(xs, s13), s2, epi=h.EPI_RESIDUAL, residual=y)
+
+        by = 3.0 * W * 2 * ff * (len(set(ii[:, :top].flatten().tolist())) + al)
+        rec(f"experts decode (chosen and shared) M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E + al, ff), bytes_=by, note="bytes: every weight that is used, once")
+        rec(f"like: experts decode, shared expert of its own M={M}", like_decode, bytes_=by)
+    return rows
+
+
+def run_pukarax(a, peaks: dict) -> dict:
+    dev = torch.device("cuda", torch.cuda.current_device())
+    T, ctx = a.prefill, a.prefill - 128  # decode steps near the end of a chunk, where they read most of it (both models at the same place)
+    res = {"design": "Pukarax", "dtype": "bf16", "data": "synthetic", "prompt_tokens": T, "peaks": {k: peaks.get(k) for k in ("hbm_gbs", "bf16_tflops")}, "sizes": {}}
+    for name, s in PUKARAX_SIZES.items():
+        t0 = time.time()
+        m = build_pukarax(s, dev)
+        new = end_to_end(m, s["vocab"], T, ctx, (1, 8), a.warmup, a.steps, dev)
+        del m
+        torch.cuda.empty_cache()
+        d = build_dimorax(dimorax_like_pukarax(s), dev)
+        old = end_to_end(d, s["vocab"], T, ctx, (1, 8), a.warmup, a.steps, dev)
+        del d
+        torch.cuda.empty_cache()
+        res["sizes"][name] = {"config": s, "layered": new, "dimorax_equal_size": old, "kernels": pukarax_kernel_table(s, T, ctx, peaks, dev),
+                              "seconds": round(time.time() - t0, 1)}
+    return res
+
+
 def run(a, peaks: dict) -> dict:
+    if a.design == "pukarax":
+        return run_pukarax(a, peaks)
     if a.design == "dimorax":
         return run_dimorax(a, peaks)
     if a.design == "viladra":
