@@ -1080,14 +1080,18 @@ def pukarax_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
 
     def decode(name, q, key, dk, c, **kw):
         m_, i, qB = md2[key], list(specs).index(key), q[:B].contiguous()
-        sp, ch = h.window_decode_plan(B, H * (2 if "lam" in kw else 1), m_.window)
-        rec(f"{name} B={B}", lambda: h.attn_window(qB, ring.cache_k[i], ring.cache_v[i], m_.positions, m_.q_start, m_.slots, oB, B, m_.window, H, G, dk, d, 0.09, c, splits=sp, chunk=ch, **kw),
+        rec(f"{name} B={B}", lambda: h.attn_decode(qB, ring.cache_k[i], ring.cache_v[i], m_.positions, m_.slots, oB, B, m_.window, H, G, dk, d, 0.09, c, **kw),
             bytes_=B * min(at + 1, c) * G * 2.0 * (d + dk * (2 if "lam" in kw else 1)))
 
     decode(f"differential attention decode, chunks of {ca}, head gate", qd, "diff", dm, ca, chunked=True, gate=gates[:B, :H], **diff)
     decode(f"like: softmax attention decode, window {ca}", ql, "like", d, ca)
     decode(f"attention decode, chunks of {cb}, entry gate", qk, "keyval", d, cb, chunked=True, gate=gates[:B], gate_entry=True)
     decode(f"like: softmax attention decode, window {cb}", ql, "like_b", d, cb)
+    m_, sp_ch = md2["like"], h.window_decode_plan(B, H, md2["like"].window)
+    qB = ql[:B].contiguous()
+    rec(f"like: softmax attention decode, window {ca}, a CTA per query head B={B}",
+        lambda: h.attn_window(qB, ring.cache_k[2], ring.cache_v[2], m_.positions, m_.q_start, m_.slots, oB, B, m_.window, H, G, d, d, 0.09, ca, splits=sp_ch[0], chunk=sp_ch[1]),
+        bytes_=B * min(at + 1, ca) * G * 4.0 * d)
     # ---- feed-forward
     x = rnd(T, W)
     al = sff // ff

@@ -167,6 +167,13 @@ int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, con
                     const void* seqpos, int64_t chunk, int weights, float softcap, const void* sink, const void* gate, int64_t gate_pitch, int gate_entry,
                     int64_t maps, const void* lambda, float out_scale, float norm_eps, int dt, void* stream);
 
+/* mbh_attn_window's softmax attention for one token per sequence (token b belongs to sequence b, its own key and value are in the ring) on tensor cores, bf16
+ * storage: every ring row is read once for all H / G <= 16 query heads of its group.  Head sizes (d, e) with a kernel: (32,32) (64,32) (64,64) (64,128)
+ * (128,64) (128,128) (96,64) (96,96); with two maps (32,32) (32,64) (48,96) (64,64) (64,128) (96,96) (128,128).  scratch fp32 [B*H*maps, splits, 2 + e]. */
+int mbh_attn_decode(const void* q, const void* ring_k, const void* ring_v, const void* positions, const void* slots, void* out, int64_t B, int64_t W, int64_t H,
+                    int64_t G, int64_t d, int64_t e, float scale, int64_t splits, void* scratch, int64_t window, int chunked, float softcap, const void* sink,
+                    const void* gate, int64_t gate_pitch, int gate_entry, int64_t maps, const void* lambda, float out_scale, float norm_eps, int dt, void* stream);
+
 /* Linear with interleaved gate/up rows and the clamped gated unit of mbh_linear's epilogue 2; gate and up of column c are multiplied by
  * rowscale[m, c / rs_group] (fp32 [M, rs_pitch]; null: 1) BEFORE the clamps.  mbh_glu_epilogue applies the same to y[M, N] of another GEMM. */
 int mbh_linear_glu(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, float limit, float alpha, const void* rowscale,

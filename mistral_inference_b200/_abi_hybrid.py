@@ -45,6 +45,7 @@ _SIGNATURES = {
     "mbh_moe_route": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, c_int, F, c_int, c_int, P, P, P, I, c_int, P]),
     "mbh_moe_sparse": (c_int, [P, P, P, P, P, P, P, I, I, I, I, I, c_int, F, F, c_int, c_int, P]),
     "mbh_attn_window": (c_int, [P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, I, c_int, P, P, P, I, c_int, F, P, P, I, c_int, I, P, F, F, c_int, P]),
+    "mbh_attn_decode": (c_int, [P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, I, c_int, F, P, P, I, c_int, I, P, F, F, c_int, P]),
     "mbh_linear_glu": (c_int, [P, P, P, I, I, I, F, F, P, I, I, c_int, P]),
     "mbh_glu_epilogue": (c_int, [P, P, I, I, F, F, P, I, I, c_int, P]),
     "mbh_embed_pos": (c_int, [P, P, P, P, F, P, I, I, c_int, P]),
@@ -458,6 +459,35 @@ def attn_window(q, cache_k, cache_v, positions, q_start, slots, out, B: int, W: 
                                  _ptr(slots), _ptr(out), q.shape[0], B, W, H, G, d, e, scale, n_tiles, splits, _ptr(scratch), window, int(chunked), _ptr(own_k),
                                  _ptr(own_v), _ptr(seqpos), chunk, int(head_bias is not None), softcap, _ptr(sink), gp, g_pitch, int(gate_entry), maps, _ptr(lam),
                                  out_scale, norm_eps, dt_of(q.dtype), _stream()), "mbh_attn_window")
+
+
+DECODE_SIZES = {1: {(32, 32), (64, 32), (64, 64), (64, 128), (128, 64), (128, 128), (96, 64), (96, 96)}, 2: DIFF_FLASH_SIZES}  # by maps per head
+DECODE_MAX_GROUP = 16
+
+
+def attn_decode_ok(q: torch.Tensor, H: int, G: int, d: int, e: int, maps: int = 1) -> bool:
+    return q.dtype == torch.bfloat16 and H // G <= DECODE_MAX_GROUP and (d, e) in DECODE_SIZES[maps] and os.environ.get("MB200_ATTN_DECODE", "1") != "0"
+
+
+def attn_decode_splits(B: int, G: int, W: int, n_sm: int = 148) -> int:
+    """CTAs per (sequence, key/value head) along the keys: two per SM over the batch, at least one round of 64 ring rows each (batch and ring size
+    only, so a captured decode graph stays valid as the context grows)."""
+    return int(max(1, min((2 * n_sm + B * G - 1) // (B * G), (W + 63) // 64, 64)))
+
+
+def attn_decode(q, cache_k, cache_v, positions, slots, out, B: int, W: int, H: int, G: int, d: int, e: int, scale: float, window: int, softcap: float = 0.0, sink=None,
+                chunked: bool = False, gate=None, gate_entry: bool = False, lam=None, out_scale: float = 1.0, norm_eps: float = 0.0, splits: int = 0) -> None:
+    """`attn_window` for one token per sequence on tensor cores (attn_decode_ok says when)."""
+    maps = 1 if lam is None else 2
+    splits = splits or attn_decode_splits(B, G, W)
+    scratch = torch.empty(B * H * maps * splits * (2 + e), dtype=torch.float32, device=q.device)
+    gp, g_pitch = _rows(gate) if gate is not None else (None, 0)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (B, H * e if gate_entry else H))
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
+    assert q.shape == (B, maps * H * d) and (lam is None or lam.dtype == torch.float32)
+    _check(lib().mbh_attn_decode(_ptr(q), _ptr(cache_k), _ptr(cache_v), _ptr(positions), _ptr(slots), _ptr(out), B, W, H, G, d, e, scale, splits, _ptr(scratch), window,
+                                 int(chunked), softcap, _ptr(sink), gp, g_pitch, int(gate_entry), maps, _ptr(lam), out_scale, norm_eps, dt_of(q.dtype), _stream()),
+           "mbh_attn_decode")
 
 
 def window_decode_plan(T: int, H: int, W: int):

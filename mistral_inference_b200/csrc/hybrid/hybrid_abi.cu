@@ -4,6 +4,7 @@
 #include "hybrid_linear.cuh"
 #include "hybrid_mixers.cuh"
 #include "hybrid_attn_flash.cuh"
+#include "hybrid_attn_decode.cuh"
 #include "hybrid_latent.cuh"
 #include "hybrid_moe.cuh"
 #include "hybrid_rotary.cuh"
@@ -102,6 +103,9 @@ template <typename T> static void run_attn_wide(const AttnArgs& a, size_t smem, 
     if (a.splits > 1) attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H);
 }
 template <typename T> static void run_moe_sparse(const MoeSparseArgs& a, int64_t T_, cudaStream_t st) {
+    if constexpr (sizeof(T) == 2) {
+        if (launch_moe_mma(a, T_, st)) return;
+    }
     moe_gateup_sparse_kernel<T><<<dim3((unsigned)((a.ff + MOE_WARPS - 1) / MOE_WARPS), (unsigned)(T_ * a.top)), MOE_WARPS * 32, 0, st>>>(a);
     moe_down_sparse_kernel<T><<<dim3((unsigned)((a.width + MOE_WARPS - 1) / MOE_WARPS), (unsigned)T_), MOE_WARPS * 32, 0, st>>>(a);
 }
@@ -117,12 +121,16 @@ template <typename T> static void run_epilogue(const LinearArgs& a, const void* 
     linear_epilogue_kernel<T><<<(unsigned)((pairs + 255) / 256), 256, 0, st>>>(a, (const T*)y);
 }
 template <typename T> static void run_prep(const AttnPrepArgs& a, int64_t T_, cudaStream_t st) { attn_prep_kernel<T><<<(unsigned)T_, 128, 0, st>>>(a); }
-template <typename T> static void run_attn(const AttnArgs& a, size_t smem, cudaStream_t st) {
-    attn_bias_kernel<T><<<dim3((unsigned)(a.T * a.H * a.maps), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
+// the partial results in a.scratch -> a.out
+template <typename T> static void run_attn_merge(const AttnArgs& a, cudaStream_t st) {
     if (a.maps > 1) attn_diff_merge_kernel<T><<<(unsigned)(a.T * a.H), AD_THREADS, 0, st>>>(a);
-    else if (a.splits > 1)
+    else
         attn_merge_kernel<T><<<dim3((unsigned)(a.T * a.H), (unsigned)((a.e + 127) / 128)), 128, 0, st>>>(a.scratch, (T*)a.out, a.splits, a.e, a.sigmoid, a.sink, a.H, a.gate,
                                                                                                     a.gate_pitch, a.gate_entry);
+}
+template <typename T> static void run_attn(const AttnArgs& a, size_t smem, cudaStream_t st) {
+    attn_bias_kernel<T><<<dim3((unsigned)(a.T * a.H * a.maps), (unsigned)a.splits), AT_WARPS * 32, smem, st>>>(a);
+    if (a.maps > 1 || a.splits > 1) run_attn_merge<T>(a, st);
 }
 template <typename T> static void run_headnorm(const void* o32, const void* w, const void* g, int64_t g_pitch, int64_t g_off, void* y, int64_t T_,
                                                int64_t N, float eps, cudaStream_t st) {
@@ -255,6 +263,31 @@ int mbh_attn_window(const void* q, const void* cache_k, const void* cache_v, con
     DISPATCH(dt, run_attn<ST>(a, smem, st));
     cudaError_t err = cudaGetLastError();
     return err ? fail(err, "mbh_attn_bias") : 0;
+}
+
+int mbh_attn_decode(const void* q, const void* ring_k, const void* ring_v, const void* positions, const void* slots, void* out, int64_t B, int64_t W, int64_t H,
+                    int64_t G, int64_t d, int64_t e, float scale, int64_t splits, void* scratch, int64_t window, int chunked, float softcap, const void* sink,
+                    const void* gate, int64_t gate_pitch, int gate_entry, int64_t maps, const void* lambda, float out_scale, float norm_eps, int dt, void* stream) {
+    if (B == 0) return 0;
+    if (dt != 0) return bad("mbh_attn_decode: bf16 storage only");
+    if (H % G) return bad("mbh_attn_decode: heads must be a multiple of kv heads");
+    if (window < 0 || (chunked && window < 1)) return bad("mbh_attn_decode: window >= 0, chunks have a size");
+    if (maps != 1 && maps != 2) return bad("mbh_attn_decode: one map per head or two");
+    if (maps == 2 && (softcap > 0.f || sink || !lambda)) return bad("mbh_attn_decode: two maps take lambda and neither a soft cap nor sinks");
+    if (gate && gate_pitch < (gate_entry ? H * e : H)) return bad("mbh_attn_decode: the gate's rows must not overlap");
+    if (splits < 1 || splits > AT_MAX_SPLITS || !scratch) return bad("mbh_attn_decode: 1 to 64 splits, with scratch");
+    AttnArgs a{};
+    a.q = q; a.cache_k = ring_k; a.cache_v = ring_v; a.positions = (const int*)positions; a.slots = (const int*)slots; a.out = out;
+    a.T = (int)B; a.B = (int)B; a.W = (int)W; a.H = (int)H; a.G = (int)G; a.d = (int)d; a.e = (int)e; a.scale = scale; a.splits = (int)splits; a.scratch = (float*)scratch;
+    a.window = (int)window; a.chunked = chunked; a.softcap = softcap; a.sink = (const float*)sink; a.gate = gate; a.gate_pitch = (int)gate_pitch; a.gate_entry = gate_entry;
+    a.maps = (int)maps; a.lambda = (const float*)lambda; a.out_scale = out_scale; a.norm_eps = norm_eps;
+    cudaStream_t st = (cudaStream_t)stream;
+    cudaError_t err = cudaSuccess;
+    if (!launch_attn_decode(a, st, err)) return bad("mbh_attn_decode: head sizes without a kernel");
+    if (err) return fail(err, "mbh_attn_decode");
+    run_attn_merge<__nv_bfloat16>(a, st);
+    err = cudaGetLastError();
+    return err ? fail(err, "mbh_attn_decode") : 0;
 }
 
 int mbh_lightning_scan(const void* qkvg, void* state, const void* decay, const void* q_start, const void* seqpos, const void* slots, void* o32,

@@ -639,17 +639,17 @@ class RotaryWindowAttention(nn.Module):
         q, k, v = _h.rot_prep(qkv, freq, md.positions, rows, view.cache_k if rows is not None else None, view.cache_v if rows is not None else None,
                               a.heads * a.maps, a.kv_heads * a.maps if own_kv else 0, a.dim, a.vdim, a.rot_dims, a.unit_norm, self.eps, own=own,
                               halves=a.rot_halves, mag=self._mag, v_heads=a.kv_heads if own_kv else 0, v_off=self.nq if a.values_are_keys else None)
-        if md.prefill:
-            plan = dict(n_tiles=query_tiles(md))
-        else:
-            splits, chunk = _h.window_decode_plan(T, a.heads * a.maps, W)
-            plan = dict(splits=splits, chunk=chunk)
+        kind = dict(softcap=a.softcap, sink=sink, chunked=a.chunked)
         if self.ng:
-            plan.update(gate=qkv[:, self.g_off: self.g_off + self.ng], gate_entry=a.out_gate == "entry")
+            kind.update(gate=qkv[:, self.g_off: self.g_off + self.ng], gate_entry=a.out_gate == "entry")
         if a.maps == 2:
-            plan.update(lam=self.difference_weight(), out_scale=1.0 - a.diff, norm_eps=self.eps)
-        _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, window,
-                       own_k=k, own_v=v, seqpos=md.seqpos if own else None, softcap=a.softcap, sink=sink, chunked=a.chunked, **plan)
+            kind.update(lam=self.difference_weight(), out_scale=1.0 - a.diff, norm_eps=self.eps)
+        if not md.prefill and _h.attn_decode_ok(q, a.heads, a.kv_heads, a.dim, a.vdim, a.maps):
+            _h.attn_decode(q, view.cache_k, view.cache_v, md.positions, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, window, **kind)
+        else:
+            splits, chunk = _h.window_decode_plan(T, a.heads * a.maps, W) if not md.prefill else (1, 0)
+            _h.attn_window(q, view.cache_k, view.cache_v, md.positions, md.q_start, md.slots, out, B, W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, window,
+                           own_k=k, own_v=v, seqpos=md.seqpos if own else None, n_tiles=query_tiles(md) if md.prefill else 0, splits=splits, chunk=chunk, **kind)
         if own:
             _h.kv_scatter(k, v, md.cache_rows, view.cache_k, view.cache_v)
         project_out(out, self.wo, x32, post, scale, bias=self.bo)

@@ -171,6 +171,28 @@ def test_experts(dtype, T, f):
     _close(x32 - x0.to(DEV), O.norm(want, w["l0.norm2b"].float(), 1e-3), dtype, f"T={T}, normed")
 
 
+@pytest.mark.parametrize("glu", [0, 1, 2])
+@pytest.mark.parametrize("T", [2, 3, 8, 9, 16])
+@pytest.mark.parametrize("E,top,ff,width,identity", [(4, 2, 24, 40, 0), (3, 3, 8, 304, 0), (40, 2, 16, 72, 2), (1, 1, 72, 24, 0)])
+def test_experts_of_several_tokens(glu, T, E, top, ff, width, identity):
+    """Expert by expert on tensor cores against one token at a time: experts that nobody, one or all tokens chose, identity experts, results stored
+    and added."""
+    from mistral_inference_b200 import _abi_hybrid as h
+
+    g = torch.Generator().manual_seed(T * E)
+    bf = lambda *sh: torch.randn(*sh, generator=g).to(torch.bfloat16).to(DEV)  # noqa: E731
+    x, w13, w2 = bf(T, width), bf(E * ff * (1 if glu == 2 else 2), width) * 0.2, bf(width, E * ff) * 0.2
+    idx = torch.stack([torch.randperm(E + identity, generator=g)[:top] for _ in range(T)]).to(torch.int32).to(DEV)
+    wsel, base = torch.rand(T, top, generator=g).to(DEV), torch.randn(T, width, generator=g).to(DEV)
+    kw = dict(glu=glu, limit=1.5, alpha=1.7)
+    for add in (False, True):
+        got = h.moe_sparse(x, w13, w2, idx, wsel, E, ff, add_to=base.clone() if add else None, **kw)
+        one = torch.cat([h.moe_sparse(x[t:t + 1], w13, w2, idx[t:t + 1].contiguous(), wsel[t:t + 1].contiguous(), E, ff, add_to=base[t:t + 1].clone() if add else None, **kw)
+                         for t in range(T)])
+        torch.testing.assert_close(got, one, rtol=3e-2, atol=3e-2 * float(one.abs().max().clamp_min(1.0)))
+        assert (got - one).norm() < 1e-2 * one.norm()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T", [1, 6, 70])
 def test_silu_feed_forward(dtype, T):
@@ -295,6 +317,39 @@ def _attention_core(dtype, maps, gate, d, e, H, G, size):
             h.attn_window(q[n - 1: n].to(DEV), ck, cv, _i32([n - 1]), _i32([0, 1]), slots, out, 1, W, H, G, d, e, scale, size or 0, splits=splits, chunk=chunk,
                           gate=None if gd is None else gd[n - 1: n], **kw)
             _close(out, ref[n - 1: n], dtype, f"decode at {n - 1}, {splits} splits", tol=3e-5)
+        if h.attn_decode_ok(q, H, G, d, e, maps):
+            for splits in (1, 3, 64):
+                out = torch.full((1, H * e), 9.0, dtype=dtype, device=DEV)
+                h.attn_decode(q[n - 1: n].to(DEV), ck, cv, _i32([n - 1]), slots, out, 1, W, H, G, d, e, scale, size or 0, gate=None if gd is None else gd[n - 1: n], splits=splits, **kw)
+                _close(out, ref[n - 1: n], dtype, f"grouped decode at {n - 1}, {splits} splits", tol=3e-5)
+
+
+@pytest.mark.parametrize("H,G,d,e,W,window,chunked,softcap", [(16, 1, 64, 64, 300, 0, False, 0.0), (6, 2, 96, 64, 40, 40, False, 5.0), (4, 4, 32, 32, 7, 7, True, 0.0), (9, 1, 128, 128, 1000, 600, True, 2.0),
+                                                              (8, 1, 64, 32, 5, 3, False, 0.0), (2, 1, 128, 64, 1, 1, True, 0.0)])
+def test_grouped_decode_attention(H, G, d, e, W, window, chunked, softcap):
+    """Sequences of unequal length in scattered rows of a ring against the exact kernel: sliding windows, chunks, soft caps, sinks, rings shorter than
+    a piece of keys, groups of up to 16 query heads; keys outside a window are poisoned."""
+    from mistral_inference_b200 import _abi_hybrid as h
+
+    g = torch.Generator().manual_seed(W)
+    pos, rows = [0, W // 2, W - 1, 3 * W + 1, 7 * W + W // 3], [4, 0, 6, 1, 3]
+    if window == 0:
+        pos = [min(p, W - 1) for p in pos]
+    B = len(pos)
+    ck, cv = torch.full((7, W, G, d), 30.0).to(torch.bfloat16), torch.full((7, W, G, e), 1e4).to(torch.bfloat16)
+    for p, r in zip(pos, rows):
+        lo = 0 if window == 0 else p - p % window if chunked else max(0, p - window + 1)
+        for j in range(lo, p + 1):
+            ck[r, j % W], cv[r, j % W] = torch.randn(G, d, generator=g), torch.randn(G, e, generator=g)
+    q = torch.randn(B, H * d, generator=g).to(torch.bfloat16).to(DEV)
+    sink = None if chunked else torch.randn(H, generator=g).to(DEV)
+    outs = []
+    for fn, extra in ((h.attn_decode, {}), (h.attn_window, dict(splits=3, chunk=32))):
+        out = torch.empty(B, H * e, dtype=torch.bfloat16, device=DEV)
+        pre = (q, ck.to(DEV), cv.to(DEV), _i32(pos)) + (() if fn is h.attn_decode else (_i32(range(B + 1)),))
+        fn(*pre, _i32(rows), out, B, W, H, G, d, e, 2.0 / math.sqrt(d), window, chunked=chunked, softcap=softcap, sink=sink, **extra)
+        outs.append(out)
+    torch.testing.assert_close(outs[0].float(), outs[1].float(), rtol=2e-2, atol=2e-2)
 
 
 def test_attention_rejects():
