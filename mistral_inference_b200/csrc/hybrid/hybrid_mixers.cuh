@@ -414,7 +414,8 @@ __global__ void attn_merge_kernel(const float* __restrict__ scratch, T* __restri
     __shared__ float red[32];
     const float* part = scratch + (size_t)blockIdx.x * splits * (2 + e);
     float M = -INFINITY;
-    for (int s = 0; s < splits; ++s) M = fmaxf(M, part[(size_t)s * (2 + e)]);
+    for (int s = threadIdx.x & 31; s < splits; s += 32) M = fmaxf(M, part[(size_t)s * (2 + e)]);
+    M = warp_max(M);
     float lpart = 0.f;
     for (int s = threadIdx.x; s < splits; s += blockDim.x) {
         const float m = part[(size_t)s * (2 + e)];
@@ -474,7 +475,8 @@ __global__ void __launch_bounds__(AD_THREADS) attn_diff_merge_kernel(AttnArgs a)
             const float* p1 = part + 2 + c;
             const float* p2 = p1 + (size_t)a.splits * pitch;
             float a1 = 0.f, a2 = 0.f;
-            for (int s = 0; s < a.splits; ++s) {
+#pragma unroll 8
+            for (int s = 0; s < a.splits; ++s) {  // the loads of eight splits in flight
                 a1 = fmaf(p1[(size_t)s * pitch], f[0][s], a1);
                 a2 = fmaf(p2[(size_t)s * pitch], f[1][s], a2);
             }

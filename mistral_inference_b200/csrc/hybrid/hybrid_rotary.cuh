@@ -52,6 +52,16 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
     // entries of pair pi: rotated ones by the layout, the rest two neighbours each
     auto first = [&](int pi) { return a.halves && pi < rh ? pi : 2 * pi; };
     auto second = [&](int pi) { return a.halves && pi < rh ? pi + rh : 2 * pi + 1; };
+    float cs[RP_MAXP], sn[RP_MAXP];  // of this lane's pairs: the same for every head
+#pragma unroll
+    for (int r = 0; r < RP_MAXP; ++r) {
+        cs[r] = 1.f; sn[r] = 0.f;
+        if (lane + 32 * r < rh) {
+            double s, c;
+            sincos((double)pos * a.freq[lane + 32 * r], &s, &c);
+            cs[r] = (float)c * a.mag; sn[r] = (float)s * a.mag;
+        }
+    }
     for (int h = blockIdx.y * nw + warp; h < a.H + a.G; h += gridDim.y * nw) {
         const bool is_q = h < a.H;
         const T* src = row + (is_q ? h * a.d : Nq + (h - a.H) * a.d);
@@ -63,10 +73,7 @@ __global__ void __launch_bounds__(128) rot_prep_kernel(RotPrepArgs a) {
             if (pi < half) {
                 float x0 = to_f(src[first(pi)]), x1 = to_f(src[second(pi)]);
                 if (pi < rh) {
-                    double sn, cs;
-                    sincos((double)pos * a.freq[pi], &sn, &cs);
-                    const float c = (float)cs * a.mag, s = (float)sn * a.mag;
-                    const float y0 = x0 * c - x1 * s, y1 = x1 * c + x0 * s;
+                    const float y0 = x0 * cs[r] - x1 * sn[r], y1 = x1 * cs[r] + x0 * sn[r];
                     x0 = y0; x1 = y1;
                 }
                 u[r] = x0; v[r] = x1;
