@@ -89,6 +89,11 @@ def _time(fn, warmup: int, steps: int, flush=None) -> float:
     return ts[len(ts) // 2]
 
 
+def _experts_used(idx) -> int:
+    """Experts that some token of the step chose: each one's weights have to be read once."""
+    return len(set(idx.flatten().tolist()))
+
+
 def end_to_end(model, vocab: int, T: int, ctx: int, batches, warmup: int, steps: int, dev) -> dict:
     out = {}
     ids = torch.randint(0, vocab, (T,), device=dev)
@@ -315,7 +320,7 @@ def taruvik_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
         note=f"useful FLOPs (top {top} of {E}); the kernels compute all {E} experts")
     for M in (1, B):
         xs, ii, ww = x[:M].contiguous(), idx[:M].contiguous(), wsel[:M].contiguous()
-        live = int((ii < E).sum())
+        live = len({e for e in ii.flatten().tolist() if e < E})
         rec(f"experts decode (chosen only) M={M}", _time(lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff), 3, 8, flush), bytes_=live * 3.0 * ff * W * 2)
     return rows
 
@@ -517,9 +522,9 @@ def lotazen_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
     for M in (1, B):
         xs, ii, ww = x[:M].contiguous(), idx[:M].contiguous(), wsel[:M].contiguous()
         rec(f"experts decode (chosen only, scaled input) M={M}", _time(lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, glu=True, limit=7.0, alpha=1.702), 3, 8, flush),
-            bytes_=M * top * 3.0 * ff * W * 2)
+            bytes_=_experts_used(ii) * 3.0 * ff * W * 2)
         rec(f"like: experts decode of the softmax-routed mixture M={M}", _time(lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff), 3, 8, flush),
-            bytes_=M * top * 3.0 * ff * W * 2)
+            bytes_=_experts_used(ii) * 3.0 * ff * W * 2)
     return rows
 
 
@@ -717,9 +722,9 @@ def viladra_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
     for M in (1, B):
         xs, ii, ww = x[:M].contiguous(), idx[:M].contiguous(), wsel[:M].contiguous()
         rec(f"experts decode (chosen only, ungated) M={M}", _time(lambda: h.moe_sparse(xs, w_up, w2, ii, ww, E, ff, glu=2), 3, 8, flush),
-            bytes_=M * top * 2.0 * ff * W * 2)
+            bytes_=_experts_used(ii) * 2.0 * ff * W * 2)
         rec(f"like: experts decode of the scaled-input gated mixture M={M}", _time(lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, glu=1, limit=7.0, alpha=1.702), 3, 8, flush),
-            bytes_=M * top * 3.0 * ff * W * 2)
+            bytes_=_experts_used(ii) * 3.0 * ff * W * 2)
     # ---- one decode step's convolution and norms
     xB = x32[:B].contiguous()
     rec(f"canon_conv decode B={B}", _time(lambda: h.canon_conv(xB, cw, cstate, 0, md2.q_start, one, md2.slots, B, True), 3, 8, flush),
@@ -926,9 +931,9 @@ def dimorax_kernel_table(s: dict, T: int, ctx: int, peaks: dict, dev) -> dict:
         flops=6.0 * T * top * ff * W, n=(2, 5))
     for M in (1, B):
         xs, ii, ww, xm = x[:M].contiguous(), idx[:M].contiguous(), wsel[:M].contiguous(), xr[:M].contiguous()
-        rec(f"experts decode (chosen only) M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, add_to=xm), bytes_=M * top * 3.0 * ff * W * 2)
+        rec(f"experts decode (chosen only) M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, add_to=xm), bytes_=_experts_used(ii) * 3.0 * ff * W * 2)
         rec(f"like: experts decode of the scaled-input gated mixture M={M}", lambda: h.moe_sparse(xs, w13, w2, ii, ww, E, ff, glu=1, limit=7.0, alpha=1.702, add_to=xm),
-            bytes_=M * top * 3.0 * ff * W * 2)
+            bytes_=_experts_used(ii) * 3.0 * ff * W * 2)
     wd = rnd(2 * s["dense_ff"], W, scale=0.02)
     rec("linear_swiglu prompt (gelu)", lambda: h.linear_swiglu(x, wd, gelu=True), flops=4.0 * T * s["dense_ff"] * W, n=(2, 5))
     rec("like: linear prompt (clamped gated unit)", lambda: h.linear_glu(x, wd, 7.0, 1.702), flops=4.0 * T * s["dense_ff"] * W, n=(2, 5))
